@@ -1,6 +1,8 @@
 // Row-wise kernels around the matrix products: embedding gather, residual-add + RMSNorm,
 // gather of the rows whose logits are wanted, and the SiLU-gated product.
 //
+// At the end: the scaled sum of two deltas with an RMS norm in groups, half the sum of two normed rows, tanh.
+//
 // Reference counterparts: csrc/ops/embedding.cu:18-36, csrc/ops/rms_norm.cu:18-73,
 // csrc/ops/residual_rms_norm_fused.cu:26-110, csrc/ops/residual_add.cu:23-82, csrc/ops/swiglu.cu:34-60.
 // Unlike those, every size is a run-time parameter, the residual stream is kept in 32 bits, and the
@@ -163,18 +165,22 @@ add_rmsnorm_rows_kernel(float* __restrict__ residual, const TD* __restrict__ del
 }
 
 // ---- gather of wanted rows ------------------------------------------------------------------------
-// out[s, :] = residual[idx[s], :] (+ delta[idx[s], :]) in 32 bits.
+// out[s, :] = residual[idx[s], :] (+ scale * (delta[idx[s], :] (+ delta2[idx[s], :]))) in 32 bits.
 template <typename TD>
 __global__ void gather_rows_kernel(const float* __restrict__ residual, const TD* __restrict__ delta,
-                                   const int* __restrict__ idx, float* __restrict__ out, int hidden,
-                                   int num_rows) {
+                                   const TD* __restrict__ delta2, float scale, const int* __restrict__ idx,
+                                   float* __restrict__ out, int hidden, int num_rows) {
     const int s = blockIdx.x;
     int r = idx[s];
     if (r < 0 || r >= num_rows) r = 0;
     const size_t src = (size_t)r * hidden;
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
         float v = residual[src + i];
-        if (delta) v += to_f32(delta[src + i]);
+        if (delta) {
+            float d = to_f32(delta[src + i]);
+            if (delta2) d += to_f32(delta2[src + i]);
+            v = fmaf(scale, d, v);
+        }
         out[(size_t)s * hidden + i] = v;
     }
 }
@@ -321,13 +327,14 @@ extern "C" int cib_add_rmsnorm(float* residual, const void* delta, int delta_dty
     return 0;
 }
 
-extern "C" int cib_gather_rows(const float* residual, const void* delta, int delta_dtype, const int* idx,
-                               float* out, int num_out, int hidden, int num_rows, cudaStream_t stream) {
+extern "C" int cib_gather_rows(const float* residual, const void* delta, const void* delta2, int delta_dtype, float scale,
+                               const int* idx, float* out, int num_out, int hidden, int num_rows, cudaStream_t stream) {
     CIB_REQUIRE(num_out >= 0 && hidden > 0, "gather_rows: bad sizes");
+    CIB_REQUIRE(delta || !delta2, "gather_rows: a second delta needs a first one");
     if (num_out == 0) return 0;
     const int threads = hidden >= 256 ? 256 : 64;
-    if (!delta || delta_dtype == kF32) gather_rows_kernel<float><<<num_out, threads, 0, stream>>>(residual, (const float*)delta, idx, out, hidden, num_rows);
-    else if (delta_dtype == kBF16) gather_rows_kernel<__nv_bfloat16><<<num_out, threads, 0, stream>>>(residual, (const __nv_bfloat16*)delta, idx, out, hidden, num_rows);
+    if (!delta || delta_dtype == kF32) gather_rows_kernel<float><<<num_out, threads, 0, stream>>>(residual, (const float*)delta, (const float*)delta2, scale, idx, out, hidden, num_rows);
+    else if (delta_dtype == kBF16) gather_rows_kernel<__nv_bfloat16><<<num_out, threads, 0, stream>>>(residual, (const __nv_bfloat16*)delta, (const __nv_bfloat16*)delta2, scale, idx, out, hidden, num_rows);
     else CIB_REQUIRE(false, "gather_rows: unsupported delta dtype %d", delta_dtype);
     CIB_LAUNCH_CHECK("gather_rows");
     return 0;
@@ -453,5 +460,239 @@ extern "C" int cib_gelu_tanh(const void* x, const void* table, int table_stride,
     else
         CIB_REQUIRE(false, "gelu_tanh: bad dtype %d", dtype);
     CIB_LAUNCH_CHECK("gelu_tanh");
+    return 0;
+}
+
+// ---- a scaled residual sum of two deltas, and an RMS norm in groups ------------------------------------------------------
+// One pass over the 32-bit residual rows x:
+//   x   += scale * (delta + delta2)                         (either delta may be absent)
+//   out  = part / sqrt(mean(part^2) + eps) * gain           for each of `groups` equal consecutive parts of the row
+// The parts of a row are independent, so the kernels walk rows * groups parts of hidden / groups values whose gains start
+// at (part % groups) * width.  Statistics and sum 32-bit, one rounding at the end.
+namespace cib {
+
+// Few parts: a block per part.
+template <typename TD, typename TO, int V>
+__global__ void group_rms_kernel(float* __restrict__ residual, const TD* __restrict__ delta, const TD* __restrict__ delta2,
+                                 float scale, AnyVec gain, float eps, TO* __restrict__ out, int groups, int width) {
+    __shared__ float scratch[33];
+    griddep_launch();
+    griddep_wait();
+    const size_t at = (size_t)blockIdx.x * width;
+    const int g0 = (int)(blockIdx.x % groups) * width;
+    float ss = 0.f;
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+        float x[V];
+        Vec<float, V>::load(residual + at + i, x);
+        if (delta) {
+            float d[V];
+            Vec<TD, V>::load(delta + at + i, d);
+            if (delta2) {
+                float e[V];
+                Vec<TD, V>::load(delta2 + at + i, e);
+#pragma unroll
+                for (int k = 0; k < V; ++k) d[k] += e[k];
+            }
+#pragma unroll
+            for (int k = 0; k < V; ++k) x[k] = fmaf(scale, d[k], x[k]);
+            Vec<float, V>::store(residual + at + i, x);
+        }
+#pragma unroll
+        for (int k = 0; k < V; ++k) ss += x[k] * x[k];
+    }
+    if (!out) return;
+    ss = block_sum(ss, scratch);
+    const float factor = 1.f / sqrtf(ss / (float)width + eps);
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+        float x[V];
+        Vec<float, V>::load(residual + at + i, x);          // this thread wrote exactly these elements above
+#pragma unroll
+        for (int k = 0; k < V; ++k) x[k] = x[k] * factor * gain[g0 + i + k];
+        Vec<TO, V>::store(out + at + i, x);
+    }
+}
+
+// Many parts of up to CH * 128 values: a warp per part, the part in registers, every load issued before the first use.
+template <typename TD, typename TO, int CH>
+__global__ void __launch_bounds__(256)
+group_rms_rows_kernel(float* __restrict__ residual, const TD* __restrict__ delta, const TD* __restrict__ delta2, float scale,
+                      AnyVec gain, float eps, TO* __restrict__ out, int groups, int width, long long parts) {
+    griddep_launch();
+    griddep_wait();
+    const int lane = threadIdx.x & 31;
+    const long long part = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (part >= parts) return;
+    const size_t at = (size_t)part * width;
+    const int g0 = (int)(part % groups) * width;
+    float x[CH][4], d[CH][4];
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+        const int i = (c * 32 + lane) * 4;
+        if (i < width) Vec<float, 4>::load(residual + at + i, x[c]);
+    }
+    if (delta) {
+#pragma unroll
+        for (int c = 0; c < CH; ++c) {
+            const int i = (c * 32 + lane) * 4;
+            if (i < width) Vec<TD, 4>::load(delta + at + i, d[c]);
+        }
+        if (delta2) {
+#pragma unroll
+            for (int c = 0; c < CH; ++c) {
+                const int i = (c * 32 + lane) * 4;
+                if (i < width) {
+                    float e[4];
+                    Vec<TD, 4>::load(delta2 + at + i, e);
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) d[c][k] += e[k];
+                }
+            }
+        }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+        const int i = (c * 32 + lane) * 4;
+        if (i < width) {
+            if (delta) {
+#pragma unroll
+                for (int k = 0; k < 4; ++k) x[c][k] = fmaf(scale, d[c][k], x[c][k]);
+                Vec<float, 4>::store(residual + at + i, x[c]);
+            }
+#pragma unroll
+            for (int k = 0; k < 4; ++k) ss += x[c][k] * x[c][k];
+        }
+    }
+    if (!out) return;
+    ss = warp_sum(ss);
+    const float factor = 1.f / sqrtf(ss / (float)width + eps);
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+        const int i = (c * 32 + lane) * 4;
+        if (i < width) {
+            float y[4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) y[k] = x[c][k] * factor * gain[g0 + i + k];
+            Vec<TO, 4>::store(out + at + i, y);
+        }
+    }
+}
+
+template <typename TD, typename TO>
+static void launch_group_rms(float* residual, const void* delta, const void* delta2, float scale, AnyVec gain, float eps, void* out,
+                             int rows, int hidden, int groups, cudaStream_t stream) {
+    const int width = hidden / groups;
+    const long long parts = (long long)rows * groups;
+    const bool pdl = prompt_pdl();
+    const TD *d1 = (const TD*)delta, *d2 = (const TD*)delta2;
+    if (width % 4 == 0 && parts >= 256 && width <= 2048) {
+        const int ch = (width + 127) / 128;
+        const dim3 grid((unsigned)((parts + 7) / 8));
+        if (ch <= 4) launch_pdl(group_rms_rows_kernel<TD, TO, 4>, grid, dim3(256), 0, stream, pdl, residual, d1, d2, scale, gain, eps, (TO*)out, groups, width, parts);
+        else if (ch <= 8) launch_pdl(group_rms_rows_kernel<TD, TO, 8>, grid, dim3(256), 0, stream, pdl, residual, d1, d2, scale, gain, eps, (TO*)out, groups, width, parts);
+        else launch_pdl(group_rms_rows_kernel<TD, TO, 16>, grid, dim3(256), 0, stream, pdl, residual, d1, d2, scale, gain, eps, (TO*)out, groups, width, parts);
+    } else if (width % 4 == 0) {
+        launch_pdl(group_rms_kernel<TD, TO, 4>, dim3((unsigned)parts), dim3(norm_threads(width, 4)), 0, stream, pdl, residual, d1, d2, scale, gain, eps, (TO*)out, groups, width);
+    } else {
+        launch_pdl(group_rms_kernel<TD, TO, 1>, dim3((unsigned)parts), dim3(norm_threads(width, 1)), 0, stream, pdl, residual, d1, d2, scale, gain, eps, (TO*)out, groups, width);
+    }
+}
+
+// ---- half the sum of two rows, each RMS-normed over the whole row ------------------------------------------------------------
+// out[t] = 1/2 (a / sqrt(mean(a^2) + eps) * gain_a + b / sqrt(mean(b^2) + eps) * gain_b): a block per row.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+pair_rms_mean_kernel(const T* __restrict__ a, const T* __restrict__ b, AnyVec gain_a, AnyVec gain_b, float eps,
+                     T* __restrict__ out, int hidden) {
+    __shared__ float scratch[33];
+    griddep_launch();
+    griddep_wait();
+    const size_t at = (size_t)blockIdx.x * hidden;
+    float sa = 0.f, sb = 0.f;
+    for (int i = threadIdx.x * V; i < hidden; i += blockDim.x * V) {
+        float x[V], y[V];
+        Vec<T, V>::load(a + at + i, x);
+        Vec<T, V>::load(b + at + i, y);
+#pragma unroll
+        for (int k = 0; k < V; ++k) {
+            sa = fmaf(x[k], x[k], sa);
+            sb = fmaf(y[k], y[k], sb);
+        }
+    }
+    sa = block_sum(sa, scratch);
+    sb = block_sum(sb, scratch);
+    const float fa = 0.5f / sqrtf(sa / (float)hidden + eps), fb = 0.5f / sqrtf(sb / (float)hidden + eps);
+    for (int i = threadIdx.x * V; i < hidden; i += blockDim.x * V) {
+        float x[V], y[V];
+        Vec<T, V>::load(a + at + i, x);
+        Vec<T, V>::load(b + at + i, y);
+#pragma unroll
+        for (int k = 0; k < V; ++k) x[k] = x[k] * fa * gain_a[i + k] + y[k] * fb * gain_b[i + k];
+        Vec<T, V>::store(out + at + i, x);
+    }
+}
+
+// out = tanh(x), 32-bit in with the exact tangent, one rounding at the end.
+template <typename T>
+__global__ void tanh_rows_kernel(const float* __restrict__ x, int x_stride, T* __restrict__ out, int cols, long long total) {
+    for (long long e = (long long)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (long long)gridDim.x * blockDim.x) {
+        const long long t = e / cols;
+        out[e] = from_f32<T>(tanhf(x[t * x_stride + (e - t * cols)]));
+    }
+}
+
+}  // namespace cib
+
+// delta, delta2 (of one type) may be null; out may be null (the sum alone).
+extern "C" int cib_group_rms(float* residual, const void* delta, const void* delta2, int delta_dtype, float scale, const void* gain,
+                             int gain_dtype, float eps, int groups, void* out, int out_dtype, int rows, int hidden,
+                             cudaStream_t stream) {
+    CIB_REQUIRE(rows >= 0 && hidden > 0 && groups > 0 && hidden % groups == 0, "group_rms: bad sizes (%d x %d in %d groups)", rows, hidden, groups);
+    CIB_REQUIRE(delta || !delta2, "group_rms: a second delta needs a first one");
+    CIB_REQUIRE(!out || gain, "group_rms: a norm needs its gain");
+    CIB_REQUIRE((long long)rows * groups < (1ll << 31), "group_rms: too many rows");
+    if (rows == 0 || (!delta && !out)) return 0;
+    AnyVec g{gain, gain_dtype == kBF16};
+    const bool d16 = delta && delta_dtype == kBF16, o16 = out_dtype == kBF16;
+    if (d16 && o16) launch_group_rms<__nv_bfloat16, __nv_bfloat16>(residual, delta, delta2, scale, g, eps, out, rows, hidden, groups, stream);
+    else if (d16) launch_group_rms<__nv_bfloat16, float>(residual, delta, delta2, scale, g, eps, out, rows, hidden, groups, stream);
+    else if (o16) launch_group_rms<float, __nv_bfloat16>(residual, delta, delta2, scale, g, eps, out, rows, hidden, groups, stream);
+    else launch_group_rms<float, float>(residual, delta, delta2, scale, g, eps, out, rows, hidden, groups, stream);
+    CIB_LAUNCH_CHECK("group_rms");
+    return 0;
+}
+
+extern "C" int cib_pair_rms_mean(const void* a, const void* b, int dtype, const void* gain_a, const void* gain_b, int gain_dtype,
+                                 float eps, void* out, int rows, int hidden, cudaStream_t stream) {
+    CIB_REQUIRE(rows >= 0 && hidden > 0, "pair_rms_mean: bad sizes");
+    if (rows == 0) return 0;
+    AnyVec ga{gain_a, gain_dtype == kBF16}, gb{gain_b, gain_dtype == kBF16};
+    const bool pdl = prompt_pdl();
+#define CIB_PAIR(T, V)                                                                                                         \
+    launch_pdl(pair_rms_mean_kernel<T, V>, dim3(rows), dim3(std::min(256, norm_threads(hidden, V))), 0, stream, pdl, (const T*)a,     \
+               (const T*)b, ga, gb, eps, (T*)out, hidden)
+    if (dtype == kF32) {
+        if (hidden % 4 == 0) CIB_PAIR(float, 4);
+        else CIB_PAIR(float, 1);
+    } else if (dtype == kBF16) {
+        if (hidden % 4 == 0) CIB_PAIR(__nv_bfloat16, 4);
+        else CIB_PAIR(__nv_bfloat16, 1);
+    } else {
+        CIB_REQUIRE(false, "pair_rms_mean: bad dtype %d", dtype);
+    }
+#undef CIB_PAIR
+    CIB_LAUNCH_CHECK("pair_rms_mean");
+    return 0;
+}
+
+extern "C" int cib_tanh_rows(const float* x, int x_stride, void* out, int out_dtype, int rows, int cols, cudaStream_t stream) {
+    CIB_REQUIRE(rows >= 0 && cols > 0 && x_stride >= cols, "tanh_rows: bad sizes");
+    const long long total = (long long)rows * cols;
+    if (total == 0) return 0;
+    const int blocks = (int)std::min<long long>((total + 255) / 256, 148 * 16);
+    if (out_dtype == kF32) tanh_rows_kernel<float><<<blocks, 256, 0, stream>>>(x, x_stride, (float*)out, cols, total);
+    else if (out_dtype == kBF16) tanh_rows_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>(x, x_stride, (__nv_bfloat16*)out, cols, total);
+    else CIB_REQUIRE(false, "tanh_rows: bad dtype %d", out_dtype);
+    CIB_LAUNCH_CHECK("tanh_rows");
     return 0;
 }

@@ -11,28 +11,9 @@
 // values each (DP: the key size rounded up to 32, 64, 128 or 256), so a warp holds 32 / (DP / 32) columns; the dot
 // products of a column with the token's key and query are finished by shuffles among its lanes.  The token's key and
 // query are staged in shared memory per warp, and the token after the one being computed is fetched meanwhile.
-#include "common.cuh"
+#include "scan_utils.cuh"
 
 namespace cib {
-
-__device__ __forceinline__ float sigmoidf_(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float softplusf_(float x) { return x > 20.f ? x : log1pf(expf(x)); }
-__device__ __forceinline__ float logsigmoidf_(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
-
-constexpr int kScanWarps = 4;
-constexpr int kScanChunk = 16;          // tokens staged in shared memory at a time
-
-// index of key element i in the staging rows: four floats of padding after every 32, so that the lanes of a column
-// (which read elements 32 apart, four at a time) hit different banks
-__device__ __forceinline__ int pad32(int i) { return i + 4 * (i >> 5); }
-template <int DP> constexpr int padded_len() { return DP + 4 * (DP / 32); }
-
-template <int SPLIT>
-__device__ __forceinline__ float split_sum(float v) {
-#pragma unroll
-    for (int o = SPLIT / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    return v;
-}
 
 // The gates of every token at once, before the scans walk the tokens one by one (in place, 32-bit):
 //   kind 0: z[t, h] -> cap * tanh((z + b0[h]) / cap);  z[t, H + h] -> logsigmoid(cap * tanh((z + b1[h]) / cap))
@@ -174,10 +155,10 @@ constexpr int kConvWarps = 8;
 
 template <typename T>
 __global__ void __launch_bounds__(kConvWarps * 32)
-delta_prep_kernel(const T* __restrict__ x, int stride, const T* __restrict__ taps, int K, const float* __restrict__ conv_state,
+delta_prep_kernel(const T* __restrict__ x, int stride, const T* __restrict__ taps, int K, float* __restrict__ conv_state,
                   const int* __restrict__ query_start_loc, const int* __restrict__ token_request,
                   const int* __restrict__ state_slots, int num_slots, int G, int H, int d, int dv, float unit_eps,
-                  float q_scale, float* __restrict__ out, int num_tokens) {
+                  float q_scale, float* __restrict__ out, int num_tokens, int update) {
     const int lane = threadIdx.x & 31;
     const int vectors = 2 * G + H;
     const long long w = (long long)blockIdx.x * kConvWarps + (threadIdx.x >> 5);
@@ -189,7 +170,7 @@ delta_prep_kernel(const T* __restrict__ x, int stride, const T* __restrict__ tap
     const int r = token_request[t];
     const int start = query_start_loc[r];
     const int slot = state_slots[r];
-    const float* cs = (slot >= 0 && slot < num_slots) ? conv_state + (size_t)slot * (K - 1) * C : nullptr;
+    float* cs = (slot >= 0 && slot < num_slots) ? conv_state + (size_t)slot * (K - 1) * C : nullptr;
     float ss = 0.f;
     for (int i = lane; i < len; i += 32) {
         const int c = c0 + i;
@@ -200,6 +181,10 @@ delta_prep_kernel(const T* __restrict__ x, int stride, const T* __restrict__ tap
             if (tt >= start) xv = to_f32(x[(size_t)tt * stride + c]);
             else if (cs) xv = cs[(size_t)(K - 1 - (start - tt)) * C + c];
             y = fmaf(to_f32(taps[(size_t)c * K + K - 1 - jb]), xv, y);
+        }
+        if (update && cs) {                               // one token a request: this lane alone reads and moves the channel's state
+            for (int i = 0; i + 2 < K; ++i) cs[(size_t)i * C + c] = cs[(size_t)(i + 1) * C + c];
+            if (K > 1) cs[(size_t)(K - 2) * C + c] = to_f32(x[(size_t)t * stride + c]);
         }
         y = y / (1.f + expf(-y));
         out[(size_t)t * C + c] = y;
@@ -213,11 +198,12 @@ delta_prep_kernel(const T* __restrict__ x, int stride, const T* __restrict__ tap
 }
 
 // The conv state after the step: the last K - 1 inputs of (old state ++ the step's rows).  A thread per (request,
-// channel) walks its K - 1 entries oldest first, so an entry is read before it is overwritten.
+// channel) walks its K - 1 entries oldest first, so an entry is read before it is overwritten.  `bias` (may be null) is
+// added to the rows' values.
 template <typename T>
 __global__ void conv_state_update_kernel(const T* __restrict__ x, int stride, int K, float* __restrict__ conv_state,
                                          const int* __restrict__ query_start_loc, const int* __restrict__ state_slots,
-                                         int num_slots, int C) {
+                                         int num_slots, int C, const float* __restrict__ bias) {
     const int r = blockIdx.y;
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
     if (c >= C) return;
@@ -226,9 +212,10 @@ __global__ void conv_state_update_kernel(const T* __restrict__ x, int stride, in
     const int start = query_start_loc[r], n = query_start_loc[r + 1] - start;
     if (n <= 0) return;
     float* cs = conv_state + (size_t)slot * (K - 1) * C;
+    const float b = bias ? bias[c] : 0.f;
     for (int i = 0; i < K - 1; ++i) {
         const int at = n + i;                              // index into old state (K - 1 entries) followed by the rows
-        cs[(size_t)i * C + c] = at < K - 1 ? cs[(size_t)at * C + c] : to_f32(x[(size_t)(start + at - (K - 1)) * stride + c]);
+        cs[(size_t)i * C + c] = at < K - 1 ? cs[(size_t)at * C + c] : to_f32(x[(size_t)(start + at - (K - 1)) * stride + c]) + b;
     }
 }
 
@@ -341,14 +328,6 @@ head_rms_gate_kernel(const float* __restrict__ o, const T* __restrict__ gate, in
 
 using namespace cib;
 
-#define CIB_SCAN_DISPATCH(d, CALL)                         \
-    do {                                                   \
-        if (d <= 32) { constexpr int DP = 32; CALL; }      \
-        else if (d <= 64) { constexpr int DP = 64; CALL; } \
-        else if (d <= 128) { constexpr int DP = 128; CALL; } \
-        else { constexpr int DP = 256; CALL; }             \
-    } while (0)
-
 extern "C" int cib_mlstm_scan(const void* q, const void* k, const void* v, int dtype, int stride, float* gates,
                               int gates_stride, const void* i_bias, const void* f_bias, int bias_dtype, float cap,
                               float q_scale, float floor_, float* state, const int* query_start_loc, const int* state_slots,
@@ -378,10 +357,25 @@ extern "C" int cib_mlstm_scan(const void* q, const void* k, const void* v, int d
     return 0;
 }
 
+// The state of a short convolution after the step, for a kernel that has only read it (see conv_state_update_kernel).
+extern "C" int cib_conv_state_update(const void* x, int dtype, int stride, int K, float* conv_state, const int* query_start_loc,
+                                     const int* state_slots, int num_slots, int num_requests, int C, const float* bias,
+                                     cudaStream_t stream) {
+    CIB_REQUIRE(K >= 2 && C > 0 && num_requests >= 0 && stride >= C, "conv_state_update: bad sizes");
+    if (num_requests == 0) return 0;
+    dim3 grid((C + 127) / 128, num_requests);
+    if (dtype == kF32) conv_state_update_kernel<float><<<grid, 128, 0, stream>>>((const float*)x, stride, K, conv_state, query_start_loc, state_slots, num_slots, C, bias);
+    else if (dtype == kBF16) conv_state_update_kernel<__nv_bfloat16><<<grid, 128, 0, stream>>>((const __nv_bfloat16*)x, stride, K, conv_state, query_start_loc, state_slots, num_slots, C, bias);
+    else CIB_REQUIRE(false, "conv_state_update: bad dtype %d", dtype);
+    CIB_LAUNCH_CHECK("conv_state_update");
+    return 0;
+}
+
+// one_token_each: every request brings one token; the state moves on in the same launch.
 extern "C" int cib_delta_prep(const void* x, int dtype, int stride, const void* taps, int K, float* conv_state,
                               const int* query_start_loc, const int* token_request, const int* state_slots, int num_slots,
                               int num_requests, int G, int H, int d, int dv, float unit_eps, float q_scale, float* out,
-                              int num_tokens, cudaStream_t stream) {
+                              int num_tokens, int one_token_each, cudaStream_t stream) {
     CIB_REQUIRE(G > 0 && H > 0 && H % G == 0 && d > 0 && dv > 0 && K >= 1, "delta_prep: bad sizes");
     if (num_tokens == 0) return 0;
     const long long warps = (long long)num_tokens * (2 * G + H);
@@ -389,13 +383,13 @@ extern "C" int cib_delta_prep(const void* x, int dtype, int stride, const void* 
     const int C = 2 * G * d + H * dv;
     dim3 ugrid((C + 127) / 128, num_requests);
     if (dtype == kF32) {
-        delta_prep_kernel<float><<<blocks, kConvWarps * 32, 0, stream>>>((const float*)x, stride, (const float*)taps, K, conv_state, query_start_loc, token_request, state_slots, num_slots, G, H, d, dv, unit_eps, q_scale, out, num_tokens);
+        delta_prep_kernel<float><<<blocks, kConvWarps * 32, 0, stream>>>((const float*)x, stride, (const float*)taps, K, conv_state, query_start_loc, token_request, state_slots, num_slots, G, H, d, dv, unit_eps, q_scale, out, num_tokens, one_token_each);
         CIB_LAUNCH_CHECK("delta_prep");
-        if (K > 1) conv_state_update_kernel<float><<<ugrid, 128, 0, stream>>>((const float*)x, stride, K, conv_state, query_start_loc, state_slots, num_slots, C);
+        if (K > 1 && !one_token_each) conv_state_update_kernel<float><<<ugrid, 128, 0, stream>>>((const float*)x, stride, K, conv_state, query_start_loc, state_slots, num_slots, C, nullptr);
     } else if (dtype == kBF16) {
-        delta_prep_kernel<__nv_bfloat16><<<blocks, kConvWarps * 32, 0, stream>>>((const __nv_bfloat16*)x, stride, (const __nv_bfloat16*)taps, K, conv_state, query_start_loc, token_request, state_slots, num_slots, G, H, d, dv, unit_eps, q_scale, out, num_tokens);
+        delta_prep_kernel<__nv_bfloat16><<<blocks, kConvWarps * 32, 0, stream>>>((const __nv_bfloat16*)x, stride, (const __nv_bfloat16*)taps, K, conv_state, query_start_loc, token_request, state_slots, num_slots, G, H, d, dv, unit_eps, q_scale, out, num_tokens, one_token_each);
         CIB_LAUNCH_CHECK("delta_prep");
-        if (K > 1) conv_state_update_kernel<__nv_bfloat16><<<ugrid, 128, 0, stream>>>((const __nv_bfloat16*)x, stride, K, conv_state, query_start_loc, state_slots, num_slots, C);
+        if (K > 1 && !one_token_each) conv_state_update_kernel<__nv_bfloat16><<<ugrid, 128, 0, stream>>>((const __nv_bfloat16*)x, stride, K, conv_state, query_start_loc, state_slots, num_slots, C, nullptr);
     } else {
         CIB_REQUIRE(false, "delta_prep: bad dtype %d", dtype);
     }

@@ -3,8 +3,10 @@
 //    over the chosen logits only.
 //  * router_scored_topk: scores s = sigmoid(z); the choice goes by s + correction[e] (a learned number per expert, may be
 //    null), the weights by s alone, times `scale`, not renormalised.  The experts form `groups` equal groups of
-//    neighbours; a group's mark is the sum of its two largest choice scores (of its one, for groups of one), and only
-//    experts of the `keep` groups with the largest marks can be chosen (the lower group wins a tie).
+//    neighbours (with `softmax` the scores are the softmax over ALL of the row's logits instead); a group's mark is the sum of its two largest choice scores (of its one, for groups of one), and only
+//    experts of the `keep` groups with the largest marks can be chosen (the lower group wins a tie).  `identity_weight`,
+//    if given, gets the sum of a token's weights of chosen experts from index `identity_from` on: experts without
+//    matrices whose output is their input, which the caller adds as weight times input.
 #include "common.cuh"
 
 namespace cib {
@@ -62,8 +64,8 @@ constexpr int kScoredWarps = 4;
 // Shared memory per warp: E choice scores, then `groups` marks.
 __global__ void __launch_bounds__(kScoredWarps * 32)
 router_scored_topk_kernel(const float* __restrict__ logits, int stride, int experts, int top, const float* __restrict__ correction,
-                          int groups, int keep, float scale, int* __restrict__ choice, float* __restrict__ weight,
-                          int num_tokens) {
+                          int groups, int keep, float scale, int softmax, int identity_from, int* __restrict__ choice,
+                          float* __restrict__ weight, float* __restrict__ identity_weight, int num_tokens) {
     extern __shared__ float scored_s[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int t = blockIdx.x * kScoredWarps + warp;
@@ -71,8 +73,19 @@ router_scored_topk_kernel(const float* __restrict__ logits, int stride, int expe
     float* cs = scored_s + (size_t)warp * (experts + groups);
     float* mark = cs + experts;
     const float* z = logits + (size_t)t * stride;
+    float z_max = 0.f, z_inv = 1.f;                               // softmax: the row's largest logit and one over the sum
+    if (softmax) {
+        z_max = -INFINITY;
+        for (int e = lane; e < experts; e += 32) z_max = fmaxf(z_max, z[e]);
+        z_max = warp_max(z_max);
+        float sum = 0.f;
+        for (int e = lane; e < experts; e += 32) sum += expf(z[e] - z_max);
+        z_inv = 1.f / warp_sum(sum);
+    }
+    auto score = [&](int e) { return softmax ? expf(z[e] - z_max) * z_inv : 1.f / (1.f + expf(-z[e])); };
+    float identity = 0.f;
     for (int e = lane; e < experts; e += 32) {
-        const float s = 1.f / (1.f + expf(-z[e]));
+        const float s = score(e);
         float c = s + (correction ? correction[e] : 0.f);
         if (c != c) c = -INFINITY;                                // a NaN is never chosen
         cs[e] = c;
@@ -127,18 +140,21 @@ router_scored_topk_kernel(const float* __restrict__ logits, int stride, int expe
         if (at == 0x7fffffff) at = -1;
         if (lane == 0) {
             choice[(size_t)t * top + k] = at;
-            weight[(size_t)t * top + k] = at >= 0 ? scale / (1.f + expf(-z[at])) : 0.f;
+            const float w = at >= 0 ? scale * score(at) : 0.f;
+            weight[(size_t)t * top + k] = w;
+            if (at >= identity_from) identity += w;
             if (at >= 0) cs[at] = -INFINITY;
         }
         __syncwarp();
     }
+    if (identity_weight && lane == 0) identity_weight[t] = identity;
 }
 
 }  // namespace cib
 
 extern "C" int cib_router_scored_topk(const float* logits, int stride, int experts, int top, const float* correction,
-                                      int groups, int keep, float scale, int* choice, float* weight, int num_tokens,
-                                      cudaStream_t stream) {
+                                      int groups, int keep, float scale, int softmax, int identity_from, int* choice,
+                                      float* weight, float* identity_weight, int num_tokens, cudaStream_t stream) {
     using namespace cib;
     CIB_REQUIRE(experts > 0 && top > 0 && top <= experts, "router_scored_topk: top %d of %d experts", top, experts);
     CIB_REQUIRE(groups > 0 && experts % groups == 0 && keep > 0 && keep <= groups, "router_scored_topk: %d groups (%d kept) of %d experts", groups, keep, experts);
@@ -149,7 +165,8 @@ extern "C" int cib_router_scored_topk(const float* logits, int stride, int exper
     static SmemLimit limit;
     if (smem > 48 * 1024 && raise_smem_limit(limit, router_scored_topk_kernel, 200 * 1024, "router_scored_topk") != 0) return -2;
     router_scored_topk_kernel<<<(num_tokens + kScoredWarps - 1) / kScoredWarps, kScoredWarps * 32, smem, stream>>>(
-        logits, stride, experts, top, correction, groups, keep, scale, choice, weight, num_tokens);
+        logits, stride, experts, top, correction, groups, keep, scale, softmax, identity_from, choice, weight, identity_weight,
+        num_tokens);
     CIB_LAUNCH_CHECK("router_scored_topk");
     return 0;
 }

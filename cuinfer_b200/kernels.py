@@ -11,6 +11,7 @@ from __future__ import annotations
 import ctypes
 import os
 import threading
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -79,24 +80,31 @@ def _declare(lib: ctypes.CDLL) -> None:
         "cib_gemm_generic_batched": [_P, _I, ctypes.c_longlong, _P, _I, ctypes.c_longlong, _I, _P, _I, ctypes.c_longlong, _I,
                                      _I, _I, _I, _I, _P],
         "cib_moe_table_gate_up": [_P, _I, _I, _P, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _F, _P],
-        "cib_moe_table_grouped": [_P, _I, _P, _P, _I, _I, _I, _P, _P, _P, _I, _F, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _P],
-        "cib_moe_table_down": [_P, _I, _P, _P, _I, _I, _I, _P, _P, _I, _F, _P, _P, _I, _P, _I, _I, _I, _P],
-        "cib_window_attention_prep": [_P, _I, _I, _P, _P, _P, _I, _F, _I, _I, _I, _I, _P, _I, _P, _I, _P, ctypes.c_longlong, _I, _I,
-                                      _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _F, _P],
-        "cib_window_attention_generic": [_P, _I, _I, _P, _I, _P, _I, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _I, _I, _P, _P, _P],
-        "cib_window_attention_mma": [_P, _I, _P, _I, _P, _I, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I, _I, _I, _P, _I, _I, _I, _P, _P, _P],
+        "cib_moe_table_grouped": [_P, _I, _P, _P, _I, _I, _I, _P, _P, _P, _I, _F, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _P],
+        "cib_moe_table_down": [_P, _I, _P, _P, _I, _I, _I, _P, _P, _I, _F, _P, _P, _I, _I, _P, _I, _I, _I, _P],
+        "cib_window_attention_prep": [_P, _I, _I, _P, _I, _P, _P, _P, _I, _F, _I, _I, _I, _I, _P, _I, _P, _I, _P, ctypes.c_longlong, _I, _I,
+                                      _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _F, _I, _P, _I, _P, _P, _P, _P, _I, _I, _P],
+        "cib_conv_state_update": [_P, _I, _I, _I, _P, _P, _P, _I, _I, _I, _P, _P],
+        "cib_channel_delta_scan": [_P, _I, _I, _P, _I, _P, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _P, _I, _I, _I, _P],
+        "cib_wkv_scan": [_P, _P, _P, _I, _I, _P, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _P, _I, _I, _I, _P],
+        "cib_token_shift": [_P, _I, _I, _P, _I, _P, _P, _P, _P, _I, _P, _I, _I, _P],
+        "cib_group_rms": [_P, _P, _P, _I, _F, _P, _I, _F, _I, _P, _I, _I, _I, _P],
+        "cib_pair_rms_mean": [_P, _P, _I, _P, _P, _I, _F, _P, _I, _I, _P],
+        "cib_tanh_rows": [_P, _I, _P, _I, _I, _I, _P],
+        "cib_window_attention_generic": [_P, _I, _I, _P, _I, _P, _I, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _I, _P],
+        "cib_window_attention_mma": [_P, _I, _P, _I, _P, _I, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I, _I, _I, _P, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _I, _P],
         "cib_hyper_stream": [_P, _P, _I, _P, _P, _P, _P, _I, _F, _P, _I, _P, _I, _I, _I, _P],
         "cib_hyper_gather": [_P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _P],
         "cib_mlstm_scan": [_P, _P, _P, _I, _I, _P, _I, _P, _P, _I, _F, _F, _F, _P, _P, _P, _I, _I, _I, _P, _I, _I, _I, _P],
-        "cib_delta_prep": [_P, _I, _I, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _P, _I, _P],
+        "cib_delta_prep": [_P, _I, _I, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _P, _I, _I, _P],
         "cib_delta_scan": [_P, _I, _P, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _P, _I, _I, _I, _P],
         "cib_head_rms_gate": [_P, _P, _I, _I, _P, _I, _I, _F, _I, _P, _I, _I, _I, _P],
         "cib_router_topk": [_P, _I, _I, _I, _P, _P, _I, _P],
-        "cib_router_scored_topk": [_P, _I, _I, _I, _P, _I, _I, _F, _P, _P, _I, _P],
+        "cib_router_scored_topk": [_P, _I, _I, _I, _P, _I, _I, _F, _I, _I, _P, _P, _P, _I, _P],
         "cib_rms_stream": [_P, _P, _I, _P, _I, _F, _P, _I, _F, _P, _P, _I, _I, _I, _P],
         "cib_gelu_tanh": [_P, _P, _I, _P, _I, _P, _I, _I, _I, _P],
         "cib_add_rmsnorm": [_P, _P, _I, _P, _I, _F, _P, _I, _I, _I, _P],
-        "cib_gather_rows": [_P, _P, _I, _P, _P, _I, _I, _I, _P],
+        "cib_gather_rows": [_P, _P, _P, _I, _F, _P, _P, _I, _I, _I, _P],
         "cib_silu_mul": [_P, _P, _I, _I, _I, _I, _P],
         "cib_qk_norm_rope_kv_write": [_P, _I, _I, _P, _P, _P, _P, _I, _I, _F, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
         "cib_paged_attention_generic": [_P, _I, _I, _P, _I, _P, _I, _I, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _I, _P],
@@ -270,17 +278,71 @@ def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor, out: torch.Tensor) -> None
     _count()
 
 
-def gather_rows(residual: torch.Tensor, delta: torch.Tensor | None, indices: torch.Tensor, out: torch.Tensor) -> None:
-    """out[s] = residual[indices[s]] (+ delta[indices[s]]), float32."""
+def gather_rows(residual: torch.Tensor, delta: torch.Tensor | None, indices: torch.Tensor, out: torch.Tensor,
+                delta2: torch.Tensor | None = None, scale: float = 1.0) -> None:
+    """out[s] = residual[indices[s]] (+ scale * (delta[indices[s]] (+ delta2[indices[s]]))), float32."""
     rows, H = residual.shape
     S = indices.numel()
     if out.shape != (S, H):
         raise KernelError(f"gather_rows: out must be [{S}, {H}]")
     rc = library().cib_gather_rows(
         _cuda(residual, "residual", torch.float32),
-        _cuda(delta, "delta") if delta is not None else None, _code(delta, "delta") if delta is not None else 0,
+        _cuda(delta, "delta") if delta is not None else None, _second_delta(delta, delta2),
+        _code(delta, "delta") if delta is not None else 0, float(scale),
         _cuda(indices, "indices", torch.int32), _cuda(out, "out", torch.float32), S, H, rows, _stream())
     _check(rc, "gather_rows")
+    _count()
+
+
+def _second_delta(delta: torch.Tensor | None, delta2: torch.Tensor | None):
+    if delta2 is None:
+        return None
+    if delta is None or delta2.shape != delta.shape or delta2.dtype != delta.dtype:
+        raise KernelError("a second delta needs a first one of its shape and dtype")
+    return _cuda(delta2, "delta2")
+
+
+def group_rms(residual: torch.Tensor, delta: torch.Tensor | None, delta2: torch.Tensor | None, scale: float,
+              norm: tuple | None, groups: int, out: torch.Tensor | None) -> None:
+    """One pass over the 32-bit residual rows: ``residual += scale * (delta + delta2)`` (either may be None), then, with
+    ``norm = (gain, eps)``, ``out`` gets the rows split into ``groups`` equal parts, each divided by its root mean square
+    (eps inside the root), times the gain."""
+    rows, H = residual.shape
+    for name, t in (("delta", delta), ("out", out)):
+        if t is not None and t.shape != residual.shape:
+            raise KernelError(f"group_rms: {name} {list(t.shape)} does not match residual {list(residual.shape)}")
+    if out is not None and (norm is None or norm[0].numel() != H):
+        raise KernelError(f"group_rms: out needs a gain of {H} values")
+    rc = library().cib_group_rms(
+        _cuda(residual, "residual", torch.float32), _cuda(delta, "delta") if delta is not None else None,
+        _second_delta(delta, delta2), _code(delta, "delta") if delta is not None else 0, float(scale),
+        _cuda(norm[0], "gain") if norm else None, _code(norm[0], "gain") if norm else 0, float(norm[1]) if norm else 0.0,
+        int(groups), _cuda(out, "out") if out is not None else None, _code(out, "out") if out is not None else 0, rows, H, _stream())
+    _check(rc, "group_rms")
+    _count()
+
+
+def pair_rms_mean(a: torch.Tensor, b: torch.Tensor, gain_a: torch.Tensor, gain_b: torch.Tensor, eps: float, out: torch.Tensor) -> None:
+    """out = (rmsnorm(a) * gain_a + rmsnorm(b) * gain_b) / 2, norms over whole rows."""
+    rows, H = a.shape
+    if b.shape != a.shape or out.shape != a.shape or not (a.dtype == b.dtype == out.dtype):
+        raise KernelError("pair_rms_mean: a, b and out must have one shape and dtype")
+    if gain_a.numel() != H or gain_b.numel() != H or gain_a.dtype != gain_b.dtype:
+        raise KernelError(f"pair_rms_mean: gains must have {H} values and one dtype")
+    rc = library().cib_pair_rms_mean(_cuda(a, "a"), _cuda(b, "b"), _code(a, "a"), _cuda(gain_a, "gain_a"), _cuda(gain_b, "gain_b"),
+                                     _code(gain_a, "gain"), float(eps), _cuda(out, "out"), rows, H, _stream())
+    _check(rc, "pair_rms_mean")
+    _count()
+
+
+def tanh_rows(x: torch.Tensor, out: torch.Tensor) -> None:
+    """out = tanh(x) for float32 rows (``out`` may have fewer columns: the first ones), rounded to out's dtype."""
+    rows, cols = out.shape
+    if x.shape[0] != rows or x.shape[1] < cols or x.stride(1) != 1:
+        raise KernelError("tanh_rows: out does not fit x")
+    rc = library().cib_tanh_rows(_cuda(x, "x", torch.float32, contiguous=False), x.stride(0), _cuda(out, "out"), _code(out, "out"),
+                                 rows, cols, _stream())
+    _check(rc, "tanh_rows")
     _count()
 
 
@@ -671,14 +733,15 @@ MOE_GROUPED_MIN_ROWS = 128
 def moe_table_feed_forward(h: torch.Tensor, ids: torch.Tensor | None, table: torch.Tensor, gate_up: torch.Tensor,
                            down: torch.Tensor, base: torch.Tensor | None, out: torch.Tensor,
                            weights: torch.Tensor | None = None, clamp_limit: float | None = None, activation: str | None = None,
-                           base_gate: torch.Tensor | None = None) -> None:
+                           base_gate: torch.Tensor | None = None, base_gate_plain: bool = False) -> None:
     """out[t] = base[t] + (1/top) * sum over k of expert(table[ids[t], k])(h[t]) with gated experts
     (``ids`` None: the table has a row per row of ``h`` — experts chosen by a router; ``weights`` float32 [T, top]:
     a weight per choice instead of 1/top; ``clamp_limit``: the experts' activation is
     ``g * sigmoid(1.702 g) * (u + 1)`` with ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``)
     ``down_e(silu(gate_e h) * up_e h)``; ``gate_up[E, 2 ff, W]`` (gate rows first), ``down[E, W, ff]``, ``table[V, top]``.
     ``activation="relu2"``: experts without a gate, ``down_e(relu(up_e h) ** 2)``, whose first matrix is ``[E, ff, W]``.
-    ``base_gate`` float32 [T] (any stride): ``base[t]`` is multiplied by ``sigmoid(base_gate[t])`` as it is added.
+    ``base_gate`` float32 [T] (any stride): ``base[t]`` is multiplied by ``sigmoid(base_gate[t])`` as it is added, or with
+    ``base_gate_plain`` by ``base_gate[t]`` itself.
     Few rows, 32-bit, or sizes that are not multiples of 32: two launches (a matrix-vector product per token and
     choice).  Many bfloat16 rows: grouped by expert (see ``MOE_GROUPED_MIN_ROWS``)."""
     T, W = h.shape
@@ -704,6 +767,7 @@ def moe_table_feed_forward(h: torch.Tensor, ids: torch.Tensor | None, table: tor
         raise KernelError("moe_table: a gate for base needs base and one number per row")
     p_bg = _cuda(base_gate, "base_gate", torch.float32, contiguous=False) if base_gate is not None else None
     bg_stride = base_gate.stride(0) if base_gate is not None else 0
+    bg_plain = 1 if base_gate_plain else 0
     lib = library()
     if (h.dtype == torch.bfloat16 and T * top >= MOE_GROUPED_MIN_ROWS and h.stride(0) % 8 == 0
             and lib.cib_moe_table_grouped_supports(W, ff, E)):
@@ -714,7 +778,7 @@ def moe_table_feed_forward(h: torch.Tensor, ids: torch.Tensor | None, table: tor
         rc = lib.cib_moe_table_grouped(
             _cuda(h, "h", contiguous=False), h.stride(0), p_ids, _cuda(table, "table", torch.int32), V, top, E,
             _cuda(gate_up, "gate_up"), _cuda(down, "down"), _cuda(base, "base", contiguous=False) if base is not None else None,
-            base.stride(0) if base is not None else 0, 1.0 / top, p_w, p_bg, bg_stride, _cuda(out, "out"), _cuda(act, "act"), _cuda(y, "y"),
+            base.stride(0) if base is not None else 0, 1.0 / top, p_w, p_bg, bg_stride, bg_plain, _cuda(out, "out"), _cuda(act, "act"), _cuda(y, "y"),
             _cuda(ints, "ints"), T, W, ff, act_kind, limit, _stream())
         _check(rc, "moe_table_grouped")
         for _ in range(4):
@@ -727,7 +791,7 @@ def moe_table_feed_forward(h: torch.Tensor, ids: torch.Tensor | None, table: tor
     _check(rc, "moe_table_gate_up")
     rc = lib.cib_moe_table_down(_cuda(act, "act"), _code(act, "act"), p_ids, _cuda(table, "table", torch.int32),
                                 V, top, E, _cuda(down, "down"), _cuda(base, "base", contiguous=False) if base is not None else None,
-                                base.stride(0) if base is not None else 0, 1.0 / top, p_w, p_bg, bg_stride, _cuda(out, "out"), T, W, ff, _stream())
+                                base.stride(0) if base is not None else 0, 1.0 / top, p_w, p_bg, bg_stride, bg_plain, _cuda(out, "out"), T, W, ff, _stream())
     _check(rc, "moe_table_down")
     _count()
     _count()
@@ -1043,20 +1107,26 @@ def router_topk(logits: torch.Tensor, top: int, choice: torch.Tensor, weight: to
 
 
 def router_scored_topk(logits: torch.Tensor, top: int, choice: torch.Tensor, weight: torch.Tensor, *,
-                       correction: torch.Tensor | None = None, groups: int = 1, keep: int = 1, scale: float = 1.0) -> None:
-    """From float32 logits [T, E] with scores ``s = sigmoid(logits)``: ``choice`` int32 [T, top], the experts with the
+                       correction: torch.Tensor | None = None, groups: int = 1, keep: int = 1, scale: float = 1.0,
+                       softmax: bool = False, identity_from: int | None = None, identity_weight: torch.Tensor | None = None) -> None:
+    """From float32 logits [T, E] with scores ``s = sigmoid(logits)`` (``softmax``: the softmax over all E): ``choice`` int32 [T, top], the experts with the
     largest ``s + correction`` (float32 [E], None: no correction; the lower index wins a tie) among the ``keep`` of
     ``groups`` equal groups of neighbouring experts whose two largest ``s + correction`` sum highest; ``weight`` float32
-    [T, top] = ``scale * s`` of the chosen, not renormalised."""
+    [T, top] = ``scale * s`` of the chosen, not renormalised.  ``identity_weight`` float32 [T] gets the sum of a token's
+    weights of chosen experts from index ``identity_from`` on."""
     T, E = logits.shape
     if choice.shape != (T, top) or weight.shape != (T, top) or logits.stride(1) != 1:
         raise KernelError("router_scored_topk: shapes do not fit")
     if correction is not None and (correction.dtype != torch.float32 or correction.numel() != E):
         raise KernelError("router_scored_topk: the correction must be float32 with a number per expert")
+    if identity_weight is not None and (identity_weight.shape != (T,) or identity_from is None):
+        raise KernelError("router_scored_topk: identity_weight must be [tokens] and identity_from given")
     rc = library().cib_router_scored_topk(_cuda(logits, "logits", torch.float32, contiguous=False), logits.stride(0), E, top,
                                           _cuda(correction, "correction") if correction is not None else None, int(groups),
-                                          int(keep), float(scale), _cuda(choice, "choice", torch.int32),
-                                          _cuda(weight, "weight", torch.float32), T, _stream())
+                                          int(keep), float(scale), 1 if softmax else 0, E if identity_from is None else int(identity_from),
+                                          _cuda(choice, "choice", torch.int32), _cuda(weight, "weight", torch.float32),
+                                          _cuda(identity_weight, "identity_weight", torch.float32) if identity_weight is not None else None,
+                                          T, _stream())
     _check(rc, "router_scored_topk")
     _count()
 
@@ -1077,7 +1147,8 @@ def window_attention_prep(qkv: torch.Tensor, positions: torch.Tensor, slot_mappi
                           vdim: int, v_first: torch.Tensor | None, mix: torch.Tensor | None, cache: torch.Tensor | None, *,
                           bias: torch.Tensor | None = None, norm: bool = True, q_gain: torch.Tensor | None = None,
                           k_gain: torch.Tensor | None = None, norm_first: bool = False, rot_half: bool = False,
-                          q_temp: tuple | None = None, value_from_key: bool = False, rot_gain: float = 1.0) -> None:
+                          q_temp: tuple | None = None, value_from_key: bool = False, rot_gain: float = 1.0, q_only: bool = False,
+                          q_out: torch.Tensor | None = None, conv: "ShortConv | None" = None) -> None:
     """On the packed rows ``[q | k | v]``: ``bias`` (float32, one value per column) is added; rotary encoding of the
     first ``rot_dims`` values of every query and key head (32-bit angle ``pos * freq[i]``; neighbouring pairs, or with
     ``rot_half`` the pairs (i, i + rot_dims / 2)); with ``norm`` every query and key head is divided by its root mean
@@ -1085,10 +1156,19 @@ def window_attention_prep(qkv: torch.Tensor, positions: torch.Tensor, slot_mappi
     ``norm_first``, before it; ``q_temp = (coef, every)`` multiplies the queries by
     ``1 + coef * ln(floor((pos + 1) / every) + 1)``.  ``value_from_key``: the rows are ``[q | k]`` and a token's value is
     its key as it stands before norm and rotation (``vdim == dim``).  ``rot_gain``: a factor on the rotation's cosine and
-    sine.  Queries are rewritten in place; keys and values
+    sine.  ``q_only``: the rows hold queries only (keys and values are those another layer has cached).  ``conv``: a short
+    causal convolution over time of every column (biases included in its input) before anything else, whose state is read
+    and, after this launch or in it, moved on; the queries then go to ``q_out`` [T, H * dim].  Queries are otherwise
+    rewritten in place; keys and values
     (``(1 - mix) * v + mix * v_first`` when both are given) go to ``cache[page, 0, kv head, slot, dim + vdim]``."""
     T, stride = qkv.shape
-    columns = (num_heads + num_kv_heads) * dim + (0 if value_from_key else num_kv_heads * vdim)
+    columns = num_heads * dim if q_only else (num_heads + num_kv_heads) * dim + (0 if value_from_key else num_kv_heads * vdim)
+    if conv is not None:
+        conv.check(columns)
+        if q_out is None:
+            raise KernelError("window_attention_prep: with a convolution the queries need rows of their own")
+    if q_out is not None and (q_out.shape != (T, num_heads * dim) or q_out.dtype != qkv.dtype or q_out.stride(1) != 1):
+        raise KernelError("window_attention_prep: q_out must be [tokens, heads * dim] of the rows' dtype")
     if value_from_key and (vdim != dim or v_first is not None):
         raise KernelError("window_attention_prep: values taken from the keys have the keys' size and are not mixed")
     if stride < columns or qkv.stride(1) != 1:
@@ -1103,7 +1183,9 @@ def window_attention_prep(qkv: torch.Tensor, positions: torch.Tensor, slot_mappi
     if v_first is not None and (v_first.shape != (T, num_kv_heads * vdim) or v_first.dtype != qkv.dtype or v_first.stride(1) != 1):
         raise KernelError("window_attention_prep: v_first does not fit")
     rc = library().cib_window_attention_prep(
-        _cuda(qkv, "qkv", contiguous=False), _code(qkv, "qkv"), qkv.stride(0), _cuda(positions, "positions", torch.int32),
+        _cuda(qkv, "qkv", contiguous=False), _code(qkv, "qkv"), qkv.stride(0),
+        _cuda(q_out, "q_out", contiguous=False) if q_out is not None else None, q_out.stride(0) if q_out is not None else 0,
+        _cuda(positions, "positions", torch.int32),
         _cuda(slot_mapping, "slot_mapping", torch.int32) if cache is not None else None,
         _cuda(freq, "freq", torch.float32) if freq is not None and rot_dims else None, rot_dims if freq is not None else 0,
         float(eps), num_heads, num_kv_heads, dim, vdim,
@@ -1113,20 +1195,67 @@ def window_attention_prep(qkv: torch.Tensor, positions: torch.Tensor, slot_mappi
         cache.shape[3] if cache is not None else 1, T,
         _f32_vec(bias, columns, "bias"), _f32_vec(q_gain, dim, "q_gain"), _f32_vec(k_gain, dim, "k_gain"), 1 if norm else 0,
         1 if norm_first else 0, 1 if rot_half else 0, 1 if q_temp else 0, float(q_temp[0]) if q_temp else 0.0,
-        int(q_temp[1]) if q_temp else 1, 1 if value_from_key else 0, float(rot_gain), _stream())
+        int(q_temp[1]) if q_temp else 1, 1 if value_from_key else 0, float(rot_gain), 1 if q_only else 0,
+        *(conv.arguments() if conv is not None else (None, 0, None, None, None, None, 0, 0)), _stream())
     _check(rc, "window_attention_prep")
+    _count()
+    if conv is not None and conv.taps.shape[0] > 1 and not conv.one_token_each:
+        conv_state_update(qkv, conv.taps.shape[0], conv.state, conv.query_start_loc, conv.state_slots, columns, bias)
+
+
+@dataclass
+class ShortConv:
+    """A short causal convolution as ``window_attention_prep`` takes it: ``taps`` float32 [K, columns] (last row: the
+    current token's), ``state`` float32 [slots, max(K - 1, 1), columns] (oldest first), the batch's device arrays, and whether every
+    request brings one token (the state then moves on in the same launch)."""
+
+    taps: torch.Tensor
+    state: torch.Tensor
+    query_start_loc: torch.Tensor
+    token_request: torch.Tensor
+    state_slots: torch.Tensor
+    one_token_each: bool = False
+
+    def check(self, columns: int) -> None:
+        K = self.taps.shape[0]
+        if self.taps.shape != (K, columns) or self.state.shape[1:] != (max(K - 1, 1), columns):
+            raise KernelError(f"short convolution: taps {list(self.taps.shape)} / state {list(self.state.shape)} do not fit {columns} columns")
+
+    def arguments(self) -> tuple:
+        return (_cuda(self.taps, "taps", torch.float32), self.taps.shape[0], _cuda(self.state, "conv_state", torch.float32),
+                _cuda(self.query_start_loc, "query_start_loc", torch.int32), _cuda(self.token_request, "token_request", torch.int32),
+                _cuda(self.state_slots, "state_slots", torch.int32), self.state.shape[0], 1 if self.one_token_each else 0)
+
+
+def conv_state_update(x: torch.Tensor, taps: int, state: torch.Tensor, query_start_loc: torch.Tensor, state_slots: torch.Tensor,
+                      columns: int, bias: torch.Tensor | None = None) -> None:
+    """The last ``taps - 1`` inputs of every request after the step: of its old state followed by its rows
+    ``x[:, :columns] + bias``."""
+    if state.shape[1:] != (max(taps - 1, 1), columns) or x.stride(1) != 1 or x.shape[1] < columns:
+        raise KernelError("conv_state_update: state or rows do not fit")
+    rc = library().cib_conv_state_update(
+        _cuda(x, "x", contiguous=False), _code(x, "x"), x.stride(0), taps, _cuda(state, "state", torch.float32),
+        _cuda(query_start_loc, "query_start_loc", torch.int32), _cuda(state_slots, "state_slots", torch.int32), state.shape[0],
+        state_slots.numel(), columns, _f32_vec(bias, columns, "bias"), _stream())
+    _check(rc, "conv_state_update")
     _count()
 
 
 def window_attention_generic(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor,
                              positions: torch.Tensor, token_request: torch.Tensor, num_heads: int, num_kv_heads: int,
                              dim: int, vdim: int, scale: float, softcap: float, window: int, keep_first: int, *,
-                             chunked: bool = False, slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None) -> None:
+                             chunked: bool = False, slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
+                             sigmoid_bias: torch.Tensor | None = None, log_bias: tuple | None = None,
+                             gate: torch.Tensor | None = None) -> None:
     """Attention of the query rows ``q[:, :H * dim]`` over the paged cache of [key | value] rows; ``out`` [T, H * vdim].
     ``softcap`` 0: no cap; ``window`` 0: every earlier key; ``chunked``: the window is a chunk, key j is seen when
     ``j // window == i // window``; ``slopes`` (float32 [H]): ``score -= slope * (i - j)``; ``sinks`` (float32 [H]): a
-    score per head that joins the softmax's denominator and nothing else."""
+    score per head that joins the softmax's denominator and nothing else.  ``sigmoid_bias`` (float32 [H]): no softmax, the
+    weight of a visible key is ``sigmoid(score + sigmoid_bias)``; ``log_bias = (r1, r2)`` (float32 [H] each):
+    ``score -= r1 * ln(1 + r2 * (i - j))``; ``gate`` (rows' dtype, [T, H * vdim] or [T, H], any row stride): the result is
+    multiplied by its sigmoid, per value or per head."""
     T = q.shape[0]
+    gate_args = _gate_args(gate, q, num_heads, vdim)
     if q.stride(1) != 1 or out.shape != (T, num_heads * vdim) or out.dtype != q.dtype or cache.dtype != q.dtype or not out.is_contiguous():
         raise KernelError("window_attention: out/cache do not fit q")
     rc = library().cib_window_attention_generic(
@@ -1134,9 +1263,25 @@ def window_attention_generic(q: torch.Tensor, out: torch.Tensor, cache: torch.Te
         cache.shape[0], cache.shape[3], _cuda(block_table, "block_table", torch.int32, contiguous=False), block_table.stride(0),
         _cuda(positions, "positions", torch.int32), _cuda(token_request, "token_request", torch.int32), T, num_heads,
         num_kv_heads, dim, vdim, float(scale), float(softcap or 0.0), int(window or 0), int(keep_first or 0),
-        1 if chunked and window else 0, _f32_vec(slopes, num_heads, "slopes"), _f32_vec(sinks, num_heads, "sinks"), _stream())
+        1 if chunked and window else 0, _f32_vec(slopes, num_heads, "slopes"), _f32_vec(sinks, num_heads, "sinks"),
+        _f32_vec(sigmoid_bias, num_heads, "sigmoid_bias"), *_log_bias_args(log_bias, num_heads), *gate_args, _stream())
     _check(rc, "window_attention_generic")
     _count()
+
+
+def _gate_args(gate: torch.Tensor | None, q: torch.Tensor, num_heads: int, vdim: int) -> tuple:
+    if gate is None:
+        return None, 0, 0
+    T = q.shape[0]
+    if gate.dtype != q.dtype or gate.stride(1) != 1 or gate.shape not in ((T, num_heads * vdim), (T, num_heads)):
+        raise KernelError(f"window_attention: the gate must be [{T}, {num_heads * vdim}] or [{T}, {num_heads}] of the rows' dtype")
+    return _cuda(gate, "gate", contiguous=False), gate.stride(0), 1 if gate.shape[1] == num_heads and vdim != 1 else 0
+
+
+def _log_bias_args(log_bias: tuple | None, num_heads: int) -> tuple:
+    if log_bias is None:
+        return None, None
+    return _f32_vec(log_bias[0], num_heads, "r1"), _f32_vec(log_bias[1], num_heads, "r2")
 
 
 def window_attention_mma_supports(dim: int, vdim: int, num_heads: int, num_kv_heads: int) -> bool:
@@ -1146,12 +1291,14 @@ def window_attention_mma_supports(dim: int, vdim: int, num_heads: int, num_kv_he
 def window_attention_mma(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor,
                          query_start_loc: torch.Tensor, seq_lens: torch.Tensor, query_lens, num_heads: int, num_kv_heads: int,
                          dim: int, vdim: int, scale: float, softcap: float, window: int, keep_first: int, splits: int = 1, *,
-                         chunked: bool = False, slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None) -> None:
+                         chunked: bool = False, slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
+                         sigmoid_bias: torch.Tensor | None = None, log_bias: tuple | None = None,
+                         gate: torch.Tensor | None = None) -> None:
     """The same attention on the tensor cores (bfloat16; key sizes 64 or 128, value sizes 32, 64 or 128).  ``query_lens``:
     tokens per request as host integers, or an upper bound that holds for every batch a captured step replays; they size
     the launch only.  ``splits`` > 1: the key tiles of every row tile are shared out to so many CTAs and a second kernel
     merges their partial results (decode steps over long windows, where a request has one row tile per key head).
-    ``chunked``, ``slopes``, ``sinks``: as for the all-sizes kernel."""
+    ``chunked``, ``slopes``, ``sinks``, ``sigmoid_bias``, ``log_bias``, ``gate``: as for the all-sizes kernel."""
     T = q.shape[0]
     if q.dtype != torch.bfloat16 or q.stride(1) != 1 or out.shape != (T, num_heads * vdim) or out.dtype != q.dtype or cache.dtype != q.dtype:
         raise KernelError("window_attention_mma: bfloat16 rows, out [T, H * vdim]")
@@ -1166,7 +1313,8 @@ def window_attention_mma(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor
         _cuda(query_start_loc, "query_start_loc", torch.int32), _cuda(seq_lens, "seq_lens", torch.int32), seq_lens.numel(), tiles,
         num_heads, num_kv_heads, dim, vdim, float(scale), float(softcap or 0.0), int(window or 0), int(keep_first or 0), splits,
         _cuda(partial, "partial") if partial is not None else None, T, 1 if chunked and window else 0, 1 if few_rows else 0,
-        _f32_vec(slopes, num_heads, "slopes"), _f32_vec(sinks, num_heads, "sinks"), _stream())
+        _f32_vec(slopes, num_heads, "slopes"), _f32_vec(sinks, num_heads, "sinks"), _f32_vec(sigmoid_bias, num_heads, "sigmoid_bias"),
+        *_log_bias_args(log_bias, num_heads), *_gate_args(gate, q, num_heads, vdim), _stream())
     _check(rc, "window_attention_mma")
     _count()
     if splits > 1:
@@ -1203,10 +1351,10 @@ def mlstm_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: torch.T
 
 def delta_prep(x: torch.Tensor, taps: torch.Tensor, conv_state: torch.Tensor, query_start_loc: torch.Tensor,
                token_request: torch.Tensor, state_slots: torch.Tensor, num_kv_heads: int, num_heads: int, dim: int, vdim: int,
-               unit_eps: float, q_scale: float, out: torch.Tensor) -> None:
+               unit_eps: float, q_scale: float, out: torch.Tensor, one_token_each: bool = False) -> None:
     """Short causal convolution + SiLU over the channels ``[q | k | v]`` of the packed rows ``x`` (continuing from, and
     updating, each request's ``conv_state`` float32 [slots, taps - 1, C]), then unit q and k heads, q times ``q_scale``;
-    ``out`` float32 [T, C].  Two launches."""
+    ``out`` float32 [T, C].  Two launches, or one when every request brings one token (``one_token_each``)."""
     T = x.shape[0]
     C = 2 * num_kv_heads * dim + num_heads * vdim
     K = taps.shape[1]
@@ -1218,10 +1366,11 @@ def delta_prep(x: torch.Tensor, taps: torch.Tensor, conv_state: torch.Tensor, qu
         _cuda(x, "x", contiguous=False), _code(x, "x"), x.stride(0), _cuda(taps, "taps"), K, _cuda(conv_state, "conv_state", torch.float32),
         _cuda(query_start_loc, "query_start_loc", torch.int32), _cuda(token_request, "token_request", torch.int32),
         _cuda(state_slots, "state_slots", torch.int32), conv_state.shape[0], state_slots.numel(), num_kv_heads, num_heads, dim, vdim,
-        float(unit_eps), float(q_scale), _cuda(out, "out", torch.float32), T, _stream())
+        float(unit_eps), float(q_scale), _cuda(out, "out", torch.float32), T, 1 if one_token_each else 0, _stream())
     _check(rc, "delta_prep")
     _count()
-    _count()
+    if not one_token_each:
+        _count()
 
 
 def delta_scan(qkv: torch.Tensor, gates: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor,
@@ -1258,6 +1407,69 @@ def head_rms_gate(o: torch.Tensor, gate: torch.Tensor, gain: torch.Tensor, eps: 
         _code(gain, "gain"), 1 if gain.numel() != vdim else 0, float(eps), 1 if silu else 0,
         _cuda(out, "out"), num_heads, vdim, T, _stream())
     _check(rc, "head_rms_gate")
+    _count()
+
+
+def channel_delta_scan(qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
+                       state: torch.Tensor, query_start_loc: torch.Tensor, state_slots: torch.Tensor, out: torch.Tensor,
+                       num_kv_heads: int, num_heads: int, dim: int, vdim: int) -> None:
+    """The gated delta rule with a decay per head and key channel.  ``qkv`` float32 [T, C] from ``delta_prep``; ``beta``
+    float32 [T, >= H] and ``decay`` float32 [T, >= H * dim] pre-activations (rows of any stride; the kernel takes
+    ``sigmoid(beta)`` and ``exp(-exp(a_log) * softplus(decay + dt_bias))``); ``state`` float32 [slots, H, dim * vdim]."""
+    T = qkv.shape[0]
+    if state.shape[1:] != (num_heads, dim * vdim) or out.shape != (T, num_heads * vdim) or qkv.shape[1] != 2 * num_kv_heads * dim + num_heads * vdim:
+        raise KernelError("channel_delta_scan: state, rows or out do not fit")
+    if beta.shape[0] != T or decay.shape[0] != T or beta.shape[1] < num_heads or decay.shape[1] < num_heads * dim or beta.stride(1) != 1 or decay.stride(1) != 1:
+        raise KernelError("channel_delta_scan: beta or decay do not fit")
+    if a_log.dtype != dt_bias.dtype or a_log.numel() != num_heads or dt_bias.numel() != num_heads * dim:
+        raise KernelError("channel_delta_scan: a_log has a number per head, dt_bias one per head and channel, in one dtype")
+    rc = library().cib_channel_delta_scan(
+        _cuda(qkv, "qkv", torch.float32), qkv.stride(0), num_kv_heads, _cuda(beta, "beta", torch.float32, contiguous=False), beta.stride(0),
+        _cuda(decay, "decay", torch.float32, contiguous=False), decay.stride(0), _cuda(a_log, "a_log"), _cuda(dt_bias, "dt_bias"),
+        _code(a_log, "a_log"), _cuda(state, "state", torch.float32), _cuda(query_start_loc, "query_start_loc", torch.int32),
+        _cuda(state_slots, "state_slots", torch.int32), state.shape[0], state_slots.numel(), T, _cuda(out, "out", torch.float32),
+        num_heads, dim, vdim, _stream())
+    _check(rc, "channel_delta_scan")
+    _count()
+
+
+def wkv_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, w0: torch.Tensor, bonus: torch.Tensor,
+             state: torch.Tensor, query_start_loc: torch.Tensor, state_slots: torch.Tensor, out: torch.Tensor, num_heads: int,
+             dim: int, vdim: int) -> None:
+    """RWKV-style time mixing over every request's rows.  ``r``, ``k`` [T, H * dim] and ``v`` [T, H * vdim] with one dtype and
+    row stride; ``decay`` float32 [T, >= H * dim] (the kernel takes ``exp(-exp(decay + w0))``); ``bonus`` [H * dim], the
+    weight of the current token's own write in its read-out; ``state`` float32 [slots, H, dim * vdim]; ``out`` float32."""
+    T = out.shape[0]
+    if not (r.stride(0) == k.stride(0) == v.stride(0)) or not (r.dtype == k.dtype == v.dtype) or r.stride(1) != 1:
+        raise KernelError("wkv_scan: r, k and v must have one dtype and row stride")
+    if (state.shape[1:] != (num_heads, dim * vdim) or out.shape != (T, num_heads * vdim) or r.shape != (T, num_heads * dim)
+            or k.shape != r.shape or v.shape != (T, num_heads * vdim)):
+        raise KernelError("wkv_scan: state, rows or out do not fit")
+    if decay.shape[0] != T or decay.shape[1] < num_heads * dim or decay.stride(1) != 1 or w0.dtype != bonus.dtype or w0.numel() != num_heads * dim or bonus.numel() != w0.numel():
+        raise KernelError("wkv_scan: decay, w0 or bonus do not fit")
+    rc = library().cib_wkv_scan(
+        _cuda(r, "r", contiguous=False), _cuda(k, "k", contiguous=False), _cuda(v, "v", contiguous=False), _code(r, "r"), r.stride(0),
+        _cuda(decay, "decay", torch.float32, contiguous=False), decay.stride(0), _cuda(w0, "w0"), _cuda(bonus, "bonus"), _code(w0, "w0"),
+        _cuda(state, "state", torch.float32), _cuda(query_start_loc, "query_start_loc", torch.int32),
+        _cuda(state_slots, "state_slots", torch.int32), state.shape[0], state_slots.numel(), T, _cuda(out, "out", torch.float32),
+        num_heads, dim, vdim, _stream())
+    _check(rc, "wkv_scan")
+    _count()
+
+
+def token_shift(x: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, query_start_loc: torch.Tensor, token_request: torch.Tensor,
+                state_slots: torch.Tensor, out: torch.Tensor) -> None:
+    """``out[s, t] = x[t] + (x[t - 1] - x[t]) * mu[s]`` for every mixing vector ``mu`` (float32 [S, W]); the row before a
+    request's first comes from ``state`` (float32 [slots, W]), which then holds the request's last row."""
+    T, W = x.shape
+    S = mu.shape[0]
+    if mu.shape != (S, W) or state.shape[1:] != (W,) or out.shape != (S, T, W) or out.dtype != x.dtype or x.stride(1) != 1:
+        raise KernelError("token_shift: mu, state or out do not fit")
+    rc = library().cib_token_shift(
+        _cuda(x, "x", contiguous=False), _code(x, "x"), x.stride(0), _cuda(mu, "mu", torch.float32), S, _cuda(state, "state", torch.float32),
+        _cuda(query_start_loc, "query_start_loc", torch.int32), _cuda(token_request, "token_request", torch.int32),
+        _cuda(state_slots, "state_slots", torch.int32), state.shape[0], _cuda(out, "out"), W, T, _stream())
+    _check(rc, "token_shift")
     _count()
 
 

@@ -100,10 +100,13 @@ TCGEN05_DECODE_MIN_CTAS = 48
 
 def window_attention(q: torch.Tensor, out: torch.Tensor, kv: PagedKV, ctx: StepContext, num_heads: int, num_kv_heads: int,
                      dim: int, vdim: int, scale: float, softcap: float, window: int, keep_first: int, *, chunked: bool = False,
-                     slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None) -> None:
+                     slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
+                     sigmoid_bias: torch.Tensor | None = None, log_bias: tuple | None = None,
+                     gate: torch.Tensor | None = None) -> None:
     """Attention over cached [key | value] rows with a capped score and a window that keeps the first tokens (or, with
     ``chunked``, a mask of chunks; ``slopes``: a distance bias per head; ``sinks``: a score per head in the softmax's
-    denominator): bfloat16
+    denominator; ``sigmoid_bias``: weights without a softmax; ``log_bias``: a bias by the logarithm of the distance; ``gate``:
+    gate logits on the result): bfloat16
     steps whose sizes the tensor-core kernel takes run there, decode steps too (the window's 64-key tiles shared out to
     several CTAs, see ``window_decode_splits``; the all-sizes kernel, a warp per token and head with one key per lane,
     measured 16 times slower at a window of 1 024 keys of 128 values); float32 and every other size run the all-sizes kernel.  ``CUINFER_B200_WINDOW_ATTENTION=generic``
@@ -117,6 +120,7 @@ def window_attention(q: torch.Tensor, out: torch.Tensor, kv: PagedKV, ctx: StepC
     if (q.dtype == torch.bfloat16 and not _FORCE_GENERIC_WINDOW and not _FORCE_MMA
             and (not ctx.decode_only or ctx.num_requests * num_kv_heads >= TCGEN05_DECODE_MIN_CTAS)
             and dim == vdim and not softcap and not keep_first and not chunked and slopes is None
+            and sigmoid_bias is None and log_bias is None and gate is None
             and kernels.attention_tcgen05_supports(dim, num_heads, num_kv_heads, kv.group.page_size)
             and q.stride(0) % 8 == 0 and out.stride(0) % 8 == 0 and (sinks is None or sinks.dtype == torch.float32)):
         kernels.attention_tcgen05(q, out, kv.cache, kv.group.block_table, ctx.query_start_loc, ctx.seq_lens,
@@ -127,8 +131,8 @@ def window_attention(q: torch.Tensor, out: torch.Tensor, kv: PagedKV, ctx: StepC
         kernels.window_attention_mma(q, out, kv.cache, kv.group.block_table, ctx.query_start_loc, ctx.seq_lens,
                                      ctx.query_lens_for_launch(), num_heads, num_kv_heads, dim, vdim, scale, softcap, window, keep_first,
                                      splits=window_decode_splits(ctx, num_kv_heads, window, keep_first), chunked=chunked,
-                                     slopes=slopes, sinks=sinks)
+                                     slopes=slopes, sinks=sinks, sigmoid_bias=sigmoid_bias, log_bias=log_bias, gate=gate)
         return
     kernels.window_attention_generic(q, out, kv.cache, kv.group.block_table, ctx.positions, ctx.token_request, num_heads,
                                      num_kv_heads, dim, vdim, scale, softcap, window, keep_first, chunked=chunked,
-                                     slopes=slopes, sinks=sinks)
+                                     slopes=slopes, sinks=sinks, sigmoid_bias=sigmoid_bias, log_bias=log_bias, gate=gate)

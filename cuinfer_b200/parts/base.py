@@ -36,9 +36,13 @@ class ResidualStream:
     A residual of several streams per token (``residual`` is [T, S, W]) is written to by learned coefficients instead of
     a sum: ``pending`` then waits together with ``writer``, the part that knows how it joins the streams; the next read
     of the streams does the write in its own pass, ``settle()`` does it alone.
+
+    A layer whose two sub-layers read the same rows leaves both outputs at once: ``pending`` and ``pending_second`` (of one
+    dtype) then join the residual together, and ``pending_scale`` multiplies what joins.  A norm that takes all three adds
+    them in its own pass (``take_deltas``); ``settle()`` does it alone.
     """
 
-    __slots__ = ("residual", "pending", "pending_norm", "extra", "_spare", "writer")
+    __slots__ = ("residual", "pending", "pending_norm", "extra", "_spare", "writer", "pending_second", "pending_scale")
 
     def __init__(self, residual: torch.Tensor, pending: Optional[torch.Tensor] = None) -> None:
         self.residual = residual
@@ -47,11 +51,26 @@ class ResidualStream:
         self.extra: Optional[torch.Tensor] = None
         self._spare: Optional[torch.Tensor] = None
         self.writer = None
+        self.pending_second: Optional[torch.Tensor] = None
+        self.pending_scale = 1.0
+
+    @property
+    def scaled(self) -> bool:
+        """True when the outstanding delta is more than one plain tensor: a second one or a factor goes with it."""
+        return self.pending is not None and (self.pending_second is not None or self.pending_scale != 1.0)
 
     @property
     def plain(self) -> bool:
         """True when what is outstanding is at most a plain delta (``pending``) to be added as it is."""
-        return self.pending_norm is None and self.extra is None and self.writer is None and self.residual.dim() == 2
+        return (self.pending_norm is None and self.extra is None and self.writer is None and self.residual.dim() == 2
+                and not self.scaled)
+
+    def take_deltas(self) -> tuple:
+        """``(pending, pending_second, pending_scale)``; the caller adds them and nothing is pending any more."""
+        out = (self.pending, self.pending_second, self.pending_scale)
+        self.pending = self.pending_second = None
+        self.pending_scale = 1.0
+        return out
 
     def wanted_rows(self, indices: torch.Tensor) -> torch.Tensor:
         """32-bit rows [len(indices), W] of the stream at the tokens ``indices`` with everything outstanding folded in
@@ -62,8 +81,9 @@ class ResidualStream:
             write = self.writer.coefficients() if self.writer is not None else None
             kernels.hyper_gather(self.residual, self.pending if write else None, write, indices, rows)
             return rows
-        self.settle()
-        kernels.gather_rows(self.residual, self.pending, indices, rows)
+        if self.pending_norm is not None or self.extra is not None:
+            self.settle()
+        kernels.gather_rows(self.residual, self.pending, indices, rows, delta2=self.pending_second, scale=self.pending_scale)
         return rows
 
     def collapsed(self) -> torch.Tensor:
@@ -79,8 +99,14 @@ class ResidualStream:
         return self.residual + self.pending.float() if self.pending is not None else self.residual
 
     def settle(self) -> None:
-        """Fold a normed delta and extra rows into the residual.  A plain pending delta stays pending: every norm and
-        the gather of the wanted rows add it themselves."""
+        """Fold a normed delta, a scaled one and extra rows into the residual.  A plain pending delta stays pending: every
+        norm and the gather of the wanted rows add it themselves."""
+        if self.scaled:
+            from .. import kernels
+            if self.pending_norm is not None:
+                raise RuntimeError("a delta that is normed before it is added has no second delta and no factor")
+            delta, second, scale = self.take_deltas()
+            kernels.group_rms(self.residual, delta, second, scale, None, 1, None)
         if self.writer is not None:
             self.writer.fold(self)
         if self.pending_norm is not None:

@@ -60,6 +60,32 @@ class PreNormBlock(Block):
         return norm.add_norm(stream)
 
 
+@BLOCKS.register("parallel")
+class ParallelBlock(Block):
+    """``h = norm(x); x += multiplier * (mixer(h) + feed_forward(h))``: one norm, whose rows both sub-layers read.  Spec:
+    ``PartSpec("parallel", norm_name=..., multiplier=1.0)``.  A layer whose feed-forward is of kind ``none`` has the mixer
+    only.
+
+    Both outputs stay pending with the factor; the next norm adds them, stores the residual and norms in one kernel."""
+
+    def __init__(self, spec: PartSpec, *, mixer: Mixer, feed_forward: FeedForward,
+                 make_norm: Callable[[str], Norm], prefix: str) -> None:
+        super().__init__(spec, mixer=mixer, feed_forward=feed_forward, make_norm=make_norm, prefix=prefix)
+        self.norm = make_norm(f"{prefix}.{spec.get('norm_name', 'norm1')}")
+        self.multiplier = float(spec.get("multiplier", 1.0))
+        self.has_feed_forward = not getattr(feed_forward, "absent", False)
+
+    def parts(self) -> List[Part]:
+        return [self.norm, self.mixer] + ([self.feed_forward] if self.has_feed_forward else [])
+
+    def forward(self, stream: ResidualStream, ctx: StepContext, run: int) -> None:
+        h = self.norm.add_norm(stream)
+        stream.pending = self.mixer.forward(h, ctx, run)
+        if self.has_feed_forward:
+            stream.pending_second = self.feed_forward.forward(h, ctx)
+        stream.pending_scale = self.multiplier
+
+
 @BLOCKS.register("sandwich")
 class SandwichBlock(Block):
     """``x += post1(mixer(pre1(x))); x += post2(feed_forward(pre2(x)))``: every sub-layer has a norm on its input and

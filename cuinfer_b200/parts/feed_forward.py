@@ -205,7 +205,12 @@ class RoutedExperts(FeedForward):
       tensor ``correction_name``; None: no correction) among the ``groups = (count, keep)`` best groups — the experts form
       ``count`` equal groups of neighbours, a group's mark is the sum of its two largest choice scores, and only experts
       of the ``keep`` best groups can be chosen; the weights are the chosen experts' ``s`` times ``route_scale``, not
-      renormalised.
+      renormalised;
+    * ``"softmax"``: the same with ``s`` the softmax over all logits.
+
+    ``identity`` n > 0 (with a scored choice): the router has n more rows, whose experts have no matrices and give back
+    their input; they are chosen and weighted like the others (their part of the output is ``h`` times the sum of their
+    weights, added where the experts' outputs are combined).
 
     An expert (``activation``), no biases: ``"silu"``: ``down(silu(gate h) * up h)``; ``"clamped"`` with ``limit`` L:
     ``g = min(gate h, L), u = clamp(up h, -L, L)``, ``down(g * sigmoid(1.702 g) * (u + 1))``; ``"relu2"``: no gate,
@@ -215,33 +220,39 @@ class RoutedExperts(FeedForward):
     token and is added, multiplied by ``sigmoid(g . h)`` when ``shared_gate_name`` names a row ``[1, W]``.
 
     Spec: ``PartSpec("moe_routed", experts=E, top=k, intermediate_size=I, activation, limit, score, correction_name, groups,
-    route_scale, router_name="router", expert_names=("e{}.gate", "e{}.up", "e{}.down"), shared_size, shared_names,
+    route_scale, identity=0, router_name="router", expert_names=("e{}.gate", "e{}.up", "e{}.down"), shared_size, shared_names,
     shared_gate_name)``.  The experts' matrices are stacked at load as for the table-routed mixture, whose kernels run
     the experts here too (rows by token and choice for few rows, grouped by expert on the tensor cores for many)."""
 
     def __init__(self, spec: PartSpec, *, hidden_size: int, prefix: str, dtype: torch.dtype) -> None:
         super().__init__(spec, hidden_size=hidden_size, prefix=prefix, dtype=dtype)
         self.experts, self.top, self.intermediate_size = int(spec.experts), int(spec.top), int(spec.intermediate_size)
-        if not 0 < self.top <= self.experts:
-            raise ValueError(f"moe_routed: top={self.top} of {self.experts} experts")
+        if self.experts <= 0:
+            raise ValueError(f"moe_routed: {self.experts} experts")
         self.activation = spec.get("activation", "silu")
         if self.activation not in ("silu", "clamped", "relu2"):
             raise ValueError(f"moe_routed: activation {self.activation!r} is not silu, clamped or relu2")
         self.gated = self.activation != "relu2"
         self.limit = float(spec.limit) if self.activation == "clamped" else None
         self.score = spec.get("score", "softmax_chosen")
-        if self.score not in ("softmax_chosen", "sigmoid"):
-            raise ValueError(f"moe_routed: score {self.score!r} is not softmax_chosen or sigmoid")
+        if self.score not in ("softmax_chosen", "sigmoid", "softmax"):
+            raise ValueError(f"moe_routed: score {self.score!r} is not softmax_chosen, sigmoid or softmax")
+        self.identity = int(spec.get("identity", 0) or 0)
+        if self.identity < 0 or (self.identity and self.score == "softmax_chosen"):
+            raise ValueError("moe_routed: identity experts belong to a scored choice")
+        routes = self.experts + self.identity
+        if not 0 < self.top <= routes:
+            raise ValueError(f"moe_routed: top={self.top} of {routes} experts")
         groups = spec.get("groups") or (1, 1)
         self.groups, self.keep = int(groups[0]), int(groups[1])
         self.route_scale = float(spec.get("route_scale", 1.0))
-        if self.score == "sigmoid":
-            if self.groups <= 0 or self.experts % self.groups or not 0 < self.keep <= self.groups:
-                raise ValueError(f"moe_routed: {self.groups} groups ({self.keep} kept) of {self.experts} experts")
-            if self.keep * (self.experts // self.groups) < self.top:
-                raise ValueError(f"moe_routed: {self.keep} groups of {self.experts // self.groups} experts cannot give {self.top}")
+        if self.score != "softmax_chosen":
+            if self.groups <= 0 or routes % self.groups or not 0 < self.keep <= self.groups:
+                raise ValueError(f"moe_routed: {self.groups} groups ({self.keep} kept) of {routes} experts")
+            if self.keep * (routes // self.groups) < self.top:
+                raise ValueError(f"moe_routed: {self.keep} groups of {routes // self.groups} experts cannot give {self.top}")
         elif (self.groups, self.keep) != (1, 1) or spec.get("correction_name") or self.route_scale != 1.0:
-            raise ValueError("moe_routed: groups, a correction and a scale belong to score='sigmoid'")
+            raise ValueError("moe_routed: groups, a correction and a scale belong to a scored choice")
         p = prefix
         names = spec.get("expert_names", ("e{}.gate", "e{}.up", "e{}.down") if self.gated else ("e{}.up", "e{}.down"))
         if len(names) != (3 if self.gated else 2):
@@ -251,13 +262,13 @@ class RoutedExperts(FeedForward):
                                for e in range(self.experts) for n in first]
         self._down_specs = [TensorSpec(f"{p}.{down.format(e)}", (hidden_size, self.intermediate_size)) for e in range(self.experts)]
         correction = spec.get("correction_name")
-        self._correction_spec = TensorSpec(f"{p}.{correction}", (self.experts,), keep_stored_precision=True, init="zeros") if correction else None
+        self._correction_spec = TensorSpec(f"{p}.{correction}", (routes,), keep_stored_precision=True, init="zeros") if correction else None
         # the router's rows and the shared expert's gate row are one stacked projection with 32-bit output
         self.shared_size = int(spec.get("shared_size", 0) or 0)
         gate_name = spec.get("shared_gate_name") if self.shared_size else None
         self.has_shared_gate = bool(gate_name)
         router_names = [f"{p}.{spec.get('router_name', 'router')}"] + ([f"{p}.{gate_name}"] if gate_name else [])
-        self.router = Linear(router_names, [self.experts] + ([1] if gate_name else []), hidden_size, dtype)
+        self.router = Linear(router_names, [routes] + ([1] if gate_name else []), hidden_size, dtype, pad=True)
         self.shared_first: Optional[Linear] = None
         self.shared_down: Optional[Linear] = None
         if self.shared_size:
@@ -268,6 +279,8 @@ class RoutedExperts(FeedForward):
             self.shared_down = Linear([f"{p}.{shared[-1]}"], [hidden_size], self.shared_size, dtype)
             if self.activation == "clamped":
                 raise ValueError("moe_routed: a shared expert with the clamped gate is not built")
+            if self.identity:
+                raise ValueError("moe_routed: identity experts beside a shared expert are not built")
         self.gate_up: Optional[torch.Tensor] = None
         self.down: Optional[torch.Tensor] = None
         self.correction: Optional[torch.Tensor] = None
@@ -285,12 +298,6 @@ class RoutedExperts(FeedForward):
         self.gate_up = store.get_stacked(self._gate_up_specs).to(self.dtype).view(E, (2 if self.gated else 1) * I, H)
         self.down = store.get_stacked(self._down_specs).to(self.dtype).view(E, H, I)
         self.router.load(store)
-        rows = self.router.weight.shape[0]
-        if rows % 8:
-            # rows of zeros up to a multiple of eight: the product then takes the tensor-core and library paths that the
-            # other projections take (nothing reads the columns they produce)
-            pad = torch.zeros((8 - rows % 8, self.hidden_size), dtype=self.router.weight.dtype, device=self.router.weight.device)
-            self.router.weight = torch.cat([self.router.weight, pad]).contiguous()
         if self._correction_spec is not None:
             self.correction = store.get(self._correction_spec).float().contiguous()
         if self.shared_size:
@@ -319,19 +326,21 @@ class RoutedExperts(FeedForward):
 
     def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
         T = x.shape[0]
-        routed = self.router.forward(x, out_dtype=torch.float32)              # [T, E (+ 1: the shared expert's gate)]
-        logits = routed[:, :self.experts]
+        routed = self.router.forward(x, out_dtype=torch.float32)              # [T, E + identity (+ 1: the shared expert's gate)]
+        logits = routed[:, :self.experts + self.identity]
         choice = torch.empty((T, self.top), dtype=torch.int32, device=x.device)
         weight = torch.empty((T, self.top), dtype=torch.float32, device=x.device)
-        if self.score == "sigmoid":
+        kept = torch.empty(T, dtype=torch.float32, device=x.device) if self.identity else None
+        if self.score != "softmax_chosen":
             kernels.router_scored_topk(logits, self.top, choice, weight, correction=self.correction, groups=self.groups,
-                                       keep=self.keep, scale=self.route_scale)
+                                       keep=self.keep, scale=self.route_scale, softmax=self.score == "softmax",
+                                       identity_from=self.experts if self.identity else None, identity_weight=kept)
         else:
             kernels.router_topk(logits, self.top, choice, weight)
-        base = self._shared(x) if self.shared_size else None
-        base_gate = routed[:, self.experts] if self.has_shared_gate else None
+        base = self._shared(x) if self.shared_size else x if self.identity else None
+        base_gate = routed[:, self.experts] if self.has_shared_gate else kept
         out = torch.empty((T, self.hidden_size), dtype=x.dtype, device=x.device)
         kernels.moe_table_feed_forward(x, None, choice, self.gate_up, self.down, base, out, weights=weight,
                                        clamp_limit=self.limit, activation="relu2" if self.activation == "relu2" else None,
-                                       base_gate=base_gate)
+                                       base_gate=base_gate, base_gate_plain=bool(self.identity))
         return out

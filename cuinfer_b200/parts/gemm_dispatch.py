@@ -91,7 +91,9 @@ def bf16_matmul_nt(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> 
         if choice == "skinny" and weight.is_contiguous() and kernels.gemm_skinny_supports(M, N, K):
             kernels.gemm_skinny(weight, out, act=x)
             return
-    library_ok = K % 8 == 0 and N % 8 == 0 and x.is_contiguous() and weight.is_contiguous()
+    # (rows that lie inside wider rows are fine for the library as long as each starts on a 16-byte boundary)
+    library_ok = (K % 8 == 0 and N % 8 == 0 and x.stride(1) == 1 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0
+                  and weight.is_contiguous())
     if takes_tcgen05(x, weight, fused=not library_ok):       # a product the library call cannot take stays on the kernel
         kernels.gemm_tcgen05(x, weight, out)
         return

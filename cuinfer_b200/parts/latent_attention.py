@@ -42,26 +42,12 @@ from . import attention_dispatch
 from . import gemm_dispatch  # noqa: F401  (sets the library products to 32-bit accumulation before the first one runs)
 from .base import Mixer
 from .context import StepContext
-from .linear import Linear
+from .linear import Linear, per_head_products
 from .registry import MIXERS, POSITION_ENCODINGS
 from .spec import PagedCacheNeed, PartSpec, TensorSpec
 
 _DEFAULT_NAMES = {"dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "q": "q", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk",
                   "uv": "uv", "sink": "sink", "g": "g", "o": "o"}
-
-
-def per_head_products(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
-    """``out[h] = a[h] @ w[h]^T`` for every head h; ``a [H, T, K]`` and ``out [H, T, N]`` are views of rows in which
-    the heads lie side by side, ``w [H, N, K]`` is dense.  bfloat16 with sizes in multiples of 8: the library's
-    strided batched product (as for the plain projections); else the FMA kernel, which is also the 32-bit path."""
-    H, T, K = a.shape
-    N = w.shape[1]
-    if (a.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and K % 8 == 0 and N % 8 == 0
-            and a.stride(1) % 8 == 0 and a.stride(0) % 8 == 0 and out.stride(1) % 8 == 0 and out.stride(0) % 8 == 0 and T > 0):
-        torch.bmm(a, w.transpose(1, 2), out=out)
-        kernels.launch_count += 1
-        return
-    kernels.gemm_generic_batched(a, w, out)
 
 
 @MIXERS.register("latent_attention")

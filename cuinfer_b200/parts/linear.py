@@ -36,25 +36,76 @@ def matmul_nt(x: torch.Tensor, weight: torch.Tensor, out_dtype: Optional[torch.d
     return out
 
 
+def per_head_products(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+    """``out[h] = a[h] @ w[h]^T`` for every head h, or for every one of several products of one size; ``a [H, T, K]`` and
+    ``out [H, T, N]`` may be views of rows in which the heads lie side by side, ``w [H, N, K]`` is dense.  bfloat16 with
+    sizes in multiples of 8: the library's strided batched product (as for the plain projections); else the FMA kernel,
+    which is also the 32-bit path."""
+    from . import gemm_dispatch  # noqa: F401  (sets the library products to 32-bit accumulation before the first one runs)
+    H, T, K = a.shape
+    N = w.shape[1]
+    if (a.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and K % 8 == 0 and N % 8 == 0
+            and a.stride(1) % 8 == 0 and a.stride(0) % 8 == 0 and out.stride(1) % 8 == 0 and out.stride(0) % 8 == 0 and T > 0):
+        torch.bmm(a, w.transpose(1, 2), out=out)
+        kernels.launch_count += 1
+        return
+    kernels.gemm_generic_batched(a, w, out)
+
+
+def padded_rows(weight: torch.Tensor, multiple: int = 8) -> torch.Tensor:
+    """``weight`` with rows of zeros up to a multiple of ``multiple``: the product then takes the tensor-core and library
+    paths that other projections take (nothing reads the columns that the extra rows produce)."""
+    rows = weight.shape[0]
+    if rows % multiple == 0:
+        return weight
+    pad = torch.zeros((multiple - rows % multiple, weight.shape[1]), dtype=weight.dtype, device=weight.device)
+    return torch.cat([weight, pad]).contiguous()
+
+
+def dense_operand(x: torch.Tensor) -> torch.Tensor:
+    """``x`` (a column range of wider rows) as a product's kernels take it: as it is when its rows start on 16-byte
+    boundaries (or in 32 bits), else a copy."""
+    if x.dtype == torch.bfloat16 and (x.stride(0) % 8 or x.data_ptr() % 16):
+        return x.contiguous()
+    return x
+
+
 class Linear:
-    def __init__(self, names: Sequence[str], out_features: Sequence[int], in_features: int, dtype: torch.dtype) -> None:
+    """``pad``: the loaded weight gets rows of zeros up to a multiple of eight (see ``padded_rows``; the output then has as
+    many more columns).  ``free_out``: places in ``names`` whose number of rows the checkpoint decides, ``free_in``: the
+    width is (see ``TensorSpec.free_axes``); ``out_features`` and ``in_features`` hold the real sizes once loaded."""
+
+    def __init__(self, names: Sequence[str], out_features: Sequence[int], in_features: int, dtype: torch.dtype, *,
+                 pad: bool = False, free_out: Sequence[int] = (), free_in: bool = False) -> None:
         if len(names) != len(out_features):
             raise ValueError("one out_features per name")
         self.names = list(names)
         self.out_features = list(out_features)
         self.in_features = in_features
         self.dtype = dtype
+        self.pad = pad
+        self.free_out = tuple(free_out)
+        self.free_in = free_in
         self.weight: Optional[torch.Tensor] = None
         self.warm_next: Optional[torch.Tensor] = None     # what the step reads right after this projection (a hint for the L2)
 
     def tensors(self) -> List[TensorSpec]:
-        return [TensorSpec(n, (o, self.in_features)) for n, o in zip(self.names, self.out_features)]
+        return [TensorSpec(n, (o, self.in_features), free_axes=((0,) if i in self.free_out else ()) + ((1,) if self.free_in else ()))
+                for i, (n, o) in enumerate(zip(self.names, self.out_features))]
 
     def load(self, store) -> None:
         specs = self.tensors()
-        self.weight = store.get(specs[0]) if len(specs) == 1 else store.get_stacked(specs)
+        if self.free_out:
+            parts = [store.get(s) for s in specs]
+            self.out_features = [p.shape[0] for p in parts]
+            self.weight = torch.cat(parts).contiguous()
+        else:
+            self.weight = store.get(specs[0]) if len(specs) == 1 else store.get_stacked(specs)
+        self.in_features = self.weight.shape[1]
         if self.weight.dtype != self.dtype:
             self.weight = self.weight.to(self.dtype)
+        if self.pad:
+            self.weight = padded_rows(self.weight)
 
     def workspace_bytes(self, tokens: int, silu_pair: bool = False) -> int:
         """Bytes of the projection's output for ``tokens`` rows (with ``silu_pair`` the stacked product may exist

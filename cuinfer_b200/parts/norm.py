@@ -2,7 +2,9 @@
 in 32 bits and one rounding at the end (csrc/ops/rms_norm.cu:43-71; eps inside the square root, the
 weight multiplies directly).  Spec: ``PartSpec("rmsnorm", eps=..., weight_suffix=".weight", one_plus=False)``: the gain is
 the tensor ``prefix + weight_suffix``, or, with ``one_plus``, one plus that tensor (a weight stored around zero; the sum
-is taken once at load, in 32 bits, and the gain stays 32-bit).
+is taken once at load, in 32 bits, and the gain stays 32-bit).  ``groups`` n > 1: the row is n equal consecutive parts,
+each divided by the root of its own mean square.  ``gain_scale``: a factor on the gain, taken once at load in 32 bits (a
+constant on the logits, on the final norm, costs nothing that way).
 
 The RMS norm also serves on a sub-layer's OUTPUT (a delta that is normed before it joins the residual): as
 ``stream.pending_norm`` it is folded by the next RMS norm of the stream in the same kernel, or alone by ``fold``.
@@ -25,6 +27,10 @@ class RMSNorm(Norm):
         super().__init__(spec, hidden_size=hidden_size, prefix=prefix, dtype=dtype)
         self.eps = float(spec.eps)
         self.one_plus = bool(spec.get("one_plus", False))
+        self.groups = int(spec.get("groups", 1))
+        self.gain_scale = float(spec.get("gain_scale", 1.0))
+        if self.groups <= 0 or hidden_size % self.groups:
+            raise ValueError(f"rmsnorm: a row of {hidden_size} values does not split into {self.groups} groups")
         self.weight: torch.Tensor | None = None
 
     def tensors(self) -> List[TensorSpec]:
@@ -35,14 +41,21 @@ class RMSNorm(Norm):
         self.weight = store.get(self.tensors()[0])
         if self.one_plus:
             self.weight = (1.0 + self.weight.float()).contiguous()
+        if self.gain_scale != 1.0:
+            self.weight = (self.weight.float() * self.gain_scale).contiguous()
 
     def fusable_rms(self):
-        return (self.weight, self.eps) if self.weight is not None else None
+        return (self.weight, self.eps) if self.weight is not None and self.groups == 1 else None
 
     def add_norm(self, stream: ResidualStream) -> torch.Tensor:
         out = torch.empty(stream.residual.shape, dtype=self.dtype, device=stream.residual.device)
         post = stream.pending_norm
-        if isinstance(post, RMSNorm) and stream.extra is None and stream.pending is not None:
+        if self.groups > 1 or stream.scaled:
+            if post is not None or stream.extra is not None or stream.writer is not None:
+                stream.settle()
+            kernels.group_rms(stream.residual, *stream.take_deltas(), (self.weight, self.eps), self.groups, out)
+            return out
+        if isinstance(post, RMSNorm) and post.groups == 1 and stream.extra is None and stream.pending is not None:
             # the delta goes through its own RMS norm, joins the residual and the sum is normed: one kernel
             kernels.rms_stream(stream.residual, stream.pending, (post.weight, post.eps), (self.weight, self.eps), out)
             stream.pending = stream.pending_norm = None
@@ -53,12 +66,17 @@ class RMSNorm(Norm):
         return out
 
     def fold(self, stream: ResidualStream) -> None:
+        if self.groups > 1:
+            raise NotImplementedError("rmsnorm: a norm in groups on a sub-layer's output is not built")
         kernels.rms_stream(stream.residual, stream.pending, (self.weight, self.eps), None, None)
         stream.pending = stream.pending_norm = None
 
     def norm_rows(self, rows: torch.Tensor) -> torch.Tensor:
         out = torch.empty(rows.shape, dtype=self.dtype, device=rows.device)
-        kernels.add_rmsnorm(rows, None, self.weight, self.eps, out)
+        if self.groups > 1:
+            kernels.group_rms(rows, None, None, 1.0, (self.weight, self.eps), self.groups, out)
+        else:
+            kernels.add_rmsnorm(rows, None, self.weight, self.eps, out)
         return out
 
 

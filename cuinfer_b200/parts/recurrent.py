@@ -1,6 +1,6 @@
-"""Mixers that carry a matrix per head from token to token instead of a cache of keys.
+"""Mixers that carry a matrix per head from token to token instead of a cache of keys, and a pair of mixers side by side.
 
-Both keep their state in 32 bits in the request's state slot (zero when the request is admitted), read it at the start
+The recurrent ones keep their state in 32 bits in the request's state slot (zero when the request is admitted), read it at the start
 of a step and write it back at the end, so a prompt may be cut anywhere.  What enters the recurrence besides the
 projections — gates, decays, their logarithms and exponentials, unit norms, the read-out, the norm after it — is 32-bit.
 
@@ -23,9 +23,30 @@ q also times ``1 / sqrt(d)``; ``beta = sigmoid(Wb h)`` and ``g = exp(-exp(A_log)
 
 then each head's o divided by its root mean square over dv, times a gain of dv values shared by the heads, times
 ``silu(Wg h)``, then ``Wo``.  Spec: ``PartSpec("gated_delta", num_heads, num_kv_heads, dim, vdim, taps, eps, names={...})``.
+
+``channel_delta`` — the gated delta rule with a decay per head and key channel and low-rank gates.  As above, except that the
+decay is a vector over the key channels, ``g = exp(-exp(A_log_h) * softplus(A2 (A1 h) + dt_bias))`` laid out [H, d], which
+multiplies the rows of S, and the output gate is ``sigmoid(G2 (G1 h))``.  The inner sizes of the two low-rank products are
+the checkpoint's.  Spec: ``PartSpec("channel_delta", num_heads, num_kv_heads, dim, vdim, taps, eps, rank, names={...})``
+(``rank``: what the random-weights mode draws).
+
+``wkv`` — RWKV-style time mixing.  With h' the previous token's h (zeros for a sequence's first), each of r, k, v, g, w reads
+a mix ``h + (h' - h) * mu_s`` of its own; ``r = Wr mix_r``, ``k = Wk mix_k``, ``v = Wv mix_v`` (H heads of d),
+``gate = silu(Wg mix_g)``, decay ``w = exp(-exp(W2 tanh(W1 mix_w) + w0))`` per head and channel::
+
+    o = (S + diag(u) k v^T)^T r;  S <- diag(w) S + k v^T
+
+then each head's o divided by its root mean square, times a gain over all heads, times the gate, then ``Wo``.  The previous
+h is state too.  Spec: ``PartSpec("wkv", num_heads, dim, eps, rank, names={...})``.
+
+``side_by_side`` — two mixers that read the same h: half the sum of their outputs, each RMS-normed over the model width.
+Spec: ``PartSpec("side_by_side", left=PartSpec(...), right=PartSpec(...), eps, names={"left": "left", "right": "right",
+"out": "out"})``: the mixers' tensors lie under ``left`` and ``right``, the norms' gains are ``left.out`` and ``right.out``.  One of
+the two may keep a paged cache; both may keep state.
 """
 from __future__ import annotations
 
+from dataclasses import replace
 from typing import Dict, List, Optional
 
 import torch
@@ -33,7 +54,7 @@ import torch
 from .. import kernels
 from .base import Mixer
 from .context import StepContext
-from .linear import Linear
+from .linear import Linear, dense_operand, per_head_products
 from .registry import MIXERS
 from .spec import PartSpec, StateNeed, TensorSpec
 
@@ -166,9 +187,233 @@ class GatedDelta(Mixer):
         gates = self.gates.forward(x, out_dtype=torch.float32)
         qkv = torch.empty((rows.shape[0], self.channels), dtype=torch.float32, device=rows.device)
         kernels.delta_prep(rows, self.conv_taps, state["conv"], ctx.query_start_loc, ctx.token_request, ctx.state_slots, G, H, d, dv,
-                           DELTA_UNIT_EPS, d ** -0.5, qkv)
+                           DELTA_UNIT_EPS, d ** -0.5, qkv, one_token_each=ctx.decode_only)
         o = torch.empty((rows.shape[0], H * dv), dtype=torch.float32, device=rows.device)
         kernels.delta_scan(qkv, gates, self.a_log, self.dt_bias, state["memory"], ctx.query_start_loc, ctx.state_slots, o, G, H, d, dv)
         out = torch.empty((rows.shape[0], H * dv), dtype=rows.dtype, device=rows.device)
         kernels.head_rms_gate(o, rows[:, self.channels:], self.gain, self.eps, True, out, H, dv)
         return self.o.forward(out)
+
+
+@MIXERS.register("channel_delta")
+class ChannelDelta(Mixer):
+    def __init__(self, spec: PartSpec, *, hidden_size: int, prefix: str, dtype: torch.dtype) -> None:
+        super().__init__(spec, hidden_size=hidden_size, prefix=prefix, dtype=dtype)
+        self.num_heads, self.num_kv_heads = int(spec.num_heads), int(spec.num_kv_heads)
+        self.dim, self.vdim, self.taps = int(spec.dim), int(spec.vdim), int(spec.taps)
+        self.eps = float(spec.get("eps", 1e-6))
+        if min(self.num_heads, self.num_kv_heads, self.dim, self.vdim, self.taps) <= 0 or self.num_heads % self.num_kv_heads:
+            raise ValueError("channel_delta: sizes must be positive and num_heads a multiple of num_kv_heads")
+        if self.dim > 256:
+            raise ValueError(f"channel_delta: key size {self.dim} is beyond what the scan kernel keeps in registers (256)")
+        n = _names(spec, {"q": "q", "k": "k", "v": "v", "o": "o", "norm": "norm", "b": "b", "a1": "a1", "a2": "a2", "g1": "g1", "g2": "g2",
+                          "A_log": "A_log", "dt_bias": "dt_bias", "conv": "{}.conv"})
+        p, H, G, d, dv = prefix, self.num_heads, self.num_kv_heads, self.dim, self.vdim
+        rank = int(spec.get("rank", 64))
+        self.channels = 2 * G * d + H * dv
+        # one projection of h: queries, keys, values and the inner values of the two low-rank products
+        self.main = Linear([f"{p}.{n[r]}" for r in ("q", "k", "v", "a1", "g1")], [G * d, G * d, H * dv, rank, rank], hidden_size, dtype,
+                           pad=True, free_out=(3, 4))
+        self.beta = Linear([f"{p}.{n['b']}"], [H], hidden_size, dtype, pad=True)
+        self.decay = Linear([f"{p}.{n['a2']}"], [H * d], rank, dtype, pad=True, free_in=True)
+        self.gate = Linear([f"{p}.{n['g2']}"], [H * dv], rank, dtype, pad=True, free_in=True)
+        self.o = Linear([f"{p}.{n['o']}"], [hidden_size], H * dv, dtype)
+        self._tap_specs = [TensorSpec(f"{p}.{n['conv'].format(n[role])}", (size, self.taps))
+                           for role, size in (("q", G * d), ("k", G * d), ("v", H * dv))]
+        self._vec_specs = [TensorSpec(f"{p}.{n['norm']}", (dv,), keep_stored_precision=True, init="ones"),
+                           TensorSpec(f"{p}.{n['A_log']}", (H,), keep_stored_precision=True, init="zeros"),
+                           TensorSpec(f"{p}.{n['dt_bias']}", (H * d,), keep_stored_precision=True, init="zeros")]
+        self.conv_taps = self.gain = self.a_log = self.dt_bias = None
+
+    def _linears(self) -> List[Linear]:
+        return [self.main, self.beta, self.decay, self.gate, self.o]
+
+    def tensors(self) -> List[TensorSpec]:
+        return [t for lin in self._linears() for t in lin.tensors()] + self._tap_specs + self._vec_specs
+
+    def load(self, store) -> None:
+        for lin in self._linears():
+            lin.load(store)
+        if (self.decay.in_features, self.gate.in_features) != tuple(self.main.out_features[3:]):
+            raise ValueError(f"{self.prefix}: the two halves of a low-rank product have different inner sizes")
+        self.conv_taps = store.get_stacked(self._tap_specs).to(self.dtype).contiguous()
+        self.gain, self.a_log, self.dt_bias = (store.get(s) for s in self._vec_specs)
+        if self.a_log.dtype != self.dt_bias.dtype:
+            self.a_log, self.dt_bias = self.a_log.float(), self.dt_bias.float()
+
+    def first_weight(self) -> Optional[torch.Tensor]:
+        return self.main.weight
+
+    def warm_after(self, weight: Optional[torch.Tensor]) -> None:
+        self.o.warm_next = weight
+
+    def state_need(self):
+        return (StateNeed((self.num_heads, self.dim * self.vdim), "float32", name="memory"),
+                StateNeed((max(self.taps - 1, 1), self.channels), "float32", name="conv"))
+
+    def workspace_bytes(self, tokens: int) -> int:
+        width = 2 if self.dtype == torch.bfloat16 else 4
+        return (sum(lin.workspace_bytes(tokens) for lin in (self.main, self.gate, self.o))
+                + tokens * (self.num_heads * (1 + 2 * self.dim) + self.channels) * 4 + tokens * self.num_heads * self.vdim * (4 + width))
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, run: int) -> torch.Tensor:
+        H, G, d, dv = self.num_heads, self.num_kv_heads, self.dim, self.vdim
+        state = ctx.run_state(run)
+        rows = self.main.forward(x)
+        beta = self.beta.forward(x, out_dtype=torch.float32)
+        at, ra, rg = self.channels, self.main.out_features[3], self.main.out_features[4]
+        decay = self.decay.forward(dense_operand(rows[:, at:at + ra]), out_dtype=torch.float32)
+        gate = self.gate.forward(dense_operand(rows[:, at + ra:at + ra + rg]))
+        qkv = torch.empty((rows.shape[0], self.channels), dtype=torch.float32, device=rows.device)
+        kernels.delta_prep(rows, self.conv_taps, state["conv"], ctx.query_start_loc, ctx.token_request, ctx.state_slots, G, H, d, dv,
+                           DELTA_UNIT_EPS, d ** -0.5, qkv, one_token_each=ctx.decode_only)
+        o = torch.empty((rows.shape[0], H * dv), dtype=torch.float32, device=rows.device)
+        kernels.channel_delta_scan(qkv, beta, decay, self.a_log, self.dt_bias, state["memory"], ctx.query_start_loc, ctx.state_slots,
+                                   o, G, H, d, dv)
+        out = torch.empty((rows.shape[0], H * dv), dtype=rows.dtype, device=rows.device)
+        kernels.head_rms_gate(o, gate[:, :H * dv], self.gain, self.eps, False, out, H, dv)
+        return self.o.forward(out)
+
+
+WKV_STREAMS = ("r", "k", "v", "g", "w")       # what reads a mix of the token and the one before it, the decay last
+
+
+@MIXERS.register("wkv")
+class TimeMixing(Mixer):
+    def __init__(self, spec: PartSpec, *, hidden_size: int, prefix: str, dtype: torch.dtype) -> None:
+        super().__init__(spec, hidden_size=hidden_size, prefix=prefix, dtype=dtype)
+        self.num_heads, self.dim = int(spec.num_heads), int(spec.dim)
+        self.eps = float(spec.get("eps", 1e-6))
+        if min(self.num_heads, self.dim) <= 0:
+            raise ValueError("wkv: sizes must be positive")
+        if self.dim > 256:
+            raise ValueError(f"wkv: head size {self.dim} is beyond what the scan kernel keeps in registers (256)")
+        n = _names(spec, {"r": "r", "k": "k", "v": "v", "g": "g", "w1": "w1", "w2": "w2", "w0": "w0", "u": "u", "mu": "mu.{}", "norm": "norm",
+                          "o": "o"})
+        p, H, d = prefix, self.num_heads, self.dim
+        rank = int(spec.get("rank", 64))
+        self._product_specs = [TensorSpec(f"{p}.{n[s]}", (H * d, hidden_size)) for s in WKV_STREAMS[:4]]
+        self.w1 = Linear([f"{p}.{n['w1']}"], [rank], hidden_size, dtype, pad=True, free_out=(0,))
+        self.w2 = Linear([f"{p}.{n['w2']}"], [H * d], rank, dtype, pad=True, free_in=True)
+        self.o = Linear([f"{p}.{n['o']}"], [hidden_size], H * d, dtype)
+        self._mu_specs = [TensorSpec(f"{p}.{n['mu'].format(s)}", (hidden_size,), keep_stored_precision=True, init="zeros") for s in WKV_STREAMS]
+        self._vec_specs = [TensorSpec(f"{p}.{n['norm']}", (H * d,), keep_stored_precision=True, init="ones"),
+                           TensorSpec(f"{p}.{n['w0']}", (H * d,), keep_stored_precision=True, init="zeros"),
+                           TensorSpec(f"{p}.{n['u']}", (H, d), keep_stored_precision=True, init="zeros")]
+        self.products: Optional[torch.Tensor] = None          # [4, H d, W]
+        self.mu: Optional[torch.Tensor] = None                # 32-bit [5, W]
+        self.gain = self.w0 = self.bonus = None
+
+    def tensors(self) -> List[TensorSpec]:
+        return self._product_specs + self.w1.tensors() + self.w2.tensors() + self.o.tensors() + self._mu_specs + self._vec_specs
+
+    def load(self, store) -> None:
+        self.products = store.get_stacked(self._product_specs).to(self.dtype).view(4, self.num_heads * self.dim, self.hidden_size)
+        for lin in (self.w1, self.w2, self.o):
+            lin.load(store)
+        if self.w2.in_features != self.w1.out_features[0]:
+            raise ValueError(f"{self.prefix}: the two halves of a low-rank product have different inner sizes")
+        self.mu = torch.stack([store.get(s).float() for s in self._mu_specs]).contiguous()
+        self.gain, self.w0, self.bonus = (store.get(s) for s in self._vec_specs)
+        if self.w0.dtype != self.bonus.dtype:
+            self.w0, self.bonus = self.w0.float(), self.bonus.float()
+
+    def first_weight(self) -> Optional[torch.Tensor]:
+        return self.products
+
+    def warm_after(self, weight: Optional[torch.Tensor]) -> None:
+        self.o.warm_next = weight
+
+    def state_need(self):
+        return (StateNeed((self.num_heads, self.dim * self.dim), "float32", name="memory"),
+                StateNeed((self.hidden_size,), "float32", name="shift"))
+
+    def workspace_bytes(self, tokens: int) -> int:
+        width = 2 if self.dtype == torch.bfloat16 else 4
+        hd = self.num_heads * self.dim
+        return tokens * (5 * self.hidden_size * width + 4 * hd * width + hd * (8 + width)) + 3 * self.w1.workspace_bytes(tokens) + self.o.workspace_bytes(tokens)
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, run: int) -> torch.Tensor:
+        H, d, T = self.num_heads, self.dim, x.shape[0]
+        state = ctx.run_state(run)
+        mixes = torch.empty((5, T, self.hidden_size), dtype=x.dtype, device=x.device)
+        kernels.token_shift(x, self.mu, state["shift"], ctx.query_start_loc, ctx.token_request, ctx.state_slots, mixes)
+        rkvg = torch.empty((4, T, H * d), dtype=x.dtype, device=x.device)
+        per_head_products(mixes[:4], self.products, rkvg)
+        low = self.w1.forward(mixes[4], out_dtype=torch.float32)
+        inner = torch.empty((T, self.w1.out_features[0]), dtype=x.dtype, device=x.device)
+        kernels.tanh_rows(low, inner)
+        decay = self.w2.forward(dense_operand(inner), out_dtype=torch.float32)
+        o = torch.empty((T, H * d), dtype=torch.float32, device=x.device)
+        kernels.wkv_scan(rkvg[0], rkvg[1], rkvg[2], decay, self.w0, self.bonus, state["memory"], ctx.query_start_loc, ctx.state_slots,
+                         o, H, d, d)
+        out = torch.empty((T, H * d), dtype=x.dtype, device=x.device)
+        kernels.head_rms_gate(o, rkvg[3], self.gain, self.eps, True, out, H, d)
+        return self.o.forward(out)
+
+
+@MIXERS.register("side_by_side")
+class SideBySide(Mixer):
+    def __init__(self, spec: PartSpec, *, hidden_size: int, prefix: str, dtype: torch.dtype) -> None:
+        super().__init__(spec, hidden_size=hidden_size, prefix=prefix, dtype=dtype)
+        self.eps = float(spec.get("eps", 1e-6))
+        n = _names(spec, {"left": "left", "right": "right", "out": "out"})
+        self.sides: Dict[str, Mixer] = {}
+        for side in ("left", "right"):
+            sub: PartSpec = spec.get(side)
+            self.sides[side] = MIXERS.get(sub.kind)(sub, hidden_size=hidden_size, prefix=f"{prefix}.{n[side]}", dtype=dtype)
+        if all(m.cache_need() is not None for m in self.sides.values()):
+            raise ValueError("side_by_side: one of the two mixers may keep a paged cache")
+        self.capturable = all(m.capturable for m in self.sides.values())
+        self._gain_specs = [TensorSpec(f"{prefix}.{n[side]}.{n['out']}", (hidden_size,), keep_stored_precision=True, init="ones")
+                            for side in ("left", "right")]
+        self.gains: Optional[List[torch.Tensor]] = None
+
+    def tensors(self) -> List[TensorSpec]:
+        return [t for m in self.sides.values() for t in m.tensors()] + self._gain_specs
+
+    def load(self, store) -> None:
+        for m in self.sides.values():
+            m.load(store)
+        self.gains = [store.get(s) for s in self._gain_specs]
+        if self.gains[0].dtype != self.gains[1].dtype:
+            self.gains = [g.float() for g in self.gains]
+
+    def first_weight(self) -> Optional[torch.Tensor]:
+        return self.sides["left"].first_weight()
+
+    def warm_after(self, weight: Optional[torch.Tensor]) -> None:
+        self.sides["left"].warm_after(self.sides["right"].first_weight())
+        self.sides["right"].warm_after(weight)
+
+    def cache_need(self):
+        needs = [m.cache_need() for m in self.sides.values()]
+        return needs[0] if needs[0] is not None else needs[1]
+
+    def _state_needs(self, side: str) -> tuple:
+        need = self.sides[side].state_need()
+        return () if need is None else tuple(need) if isinstance(need, (tuple, list)) else (need,)
+
+    def state_need(self):
+        """Both mixers' tensors under names of their own."""
+        out = tuple(replace(need, name=f"{side}.{need.name}") for side in self.sides for need in self._state_needs(side))
+        return out or None
+
+    def _context(self, side: str, ctx: StepContext, run: int) -> StepContext:
+        """The step as one of the mixers sees it: its own state tensors under the names it gave them."""
+        needs = self._state_needs(side)
+        if not needs:
+            return ctx
+        have = ctx.run_state(run)
+        own = {need.name: have[f"{side}.{need.name}"] for need in needs}
+        return replace(ctx, state={run: own if needs[0].name else own[""]})
+
+    def workspace_bytes(self, tokens: int) -> int:
+        width = 2 if self.dtype == torch.bfloat16 else 4
+        return max(m.workspace_bytes(tokens) for m in self.sides.values()) + 2 * tokens * self.hidden_size * width
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, run: int) -> torch.Tensor:
+        left, right = (self.sides[side].forward(x, self._context(side, ctx, run), run) for side in ("left", "right"))
+        out = torch.empty_like(left)
+        kernels.pair_rms_mean(left, right, self.gains[0], self.gains[1], self.eps, out)
+        return out

@@ -136,6 +136,15 @@ class TensorSpec:
     integer: bool = False    # an integer table (kept as int32); a floating tensor in its place is refused, and vice versa
     init: str = "normal"     # how the random-weights mode fills it: "normal", "ones" (a gain), "zeros" (a bias), "identity" (a square matrix around one on its diagonal)
     modulus: int = 0         # for an integer table: entries are drawn from 0..modulus-1, different within a row
+    # axes whose size the checkpoint decides (the inner size of a low-rank product, which no configuration names): the
+    # number in ``shape`` is then only what the random-weights mode draws
+    free_axes: tuple[int, ...] = ()
+
+    def accepts(self, shape) -> bool:
+        """Whether a stored tensor of this shape is the one expected."""
+        shape = tuple(shape)
+        return len(shape) == len(self.shape) and all(
+            have == want or (axis in self.free_axes and have > 0) for axis, (have, want) in enumerate(zip(shape, self.shape)))
 
 
 @dataclass(frozen=True)

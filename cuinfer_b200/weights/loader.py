@@ -42,7 +42,7 @@ class WeightStore:
         for name, spec in expected.items():
             if name in self.checkpoint:
                 got = self.checkpoint.entry(name).shape
-                if tuple(got) != tuple(spec.shape):
+                if not spec.accepts(got):
                     wrong.append(f"{name}: expected {list(spec.shape)}, got {list(got)}")
                 elif self.checkpoint.entry(name).dtype.is_floating_point == spec.integer:
                     wrong.append(f"{name}: expected {'an integer' if spec.integer else 'a floating'} dtype, "
@@ -73,7 +73,7 @@ class WeightStore:
         if spec.name not in self.checkpoint:
             raise WeightError(f"missing checkpoint tensor '{spec.name}' in {self.model_dir}")
         entry = self.checkpoint.entry(spec.name)
-        if tuple(entry.shape) != tuple(spec.shape):
+        if not spec.accepts(entry.shape):
             raise WeightError(
                 f"mismatched shape for '{spec.name}': expected {list(spec.shape)}, got {list(entry.shape)}"
             )
