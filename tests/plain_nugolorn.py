@@ -250,3 +250,128 @@ def greedy(config: dict, weights: Dict[str, torch.Tensor], prompt, steps: int) -
         out.append(nxt)
         toks.append(nxt)
     return out
+
+
+# ---- how safe the routers' choices are ------------------------------------------------------------------------------------
+def choice_margins(scores, top: int):
+    """For rows of choice scores [N, E]: how far the last chosen lies above the first rejected, per row."""
+    if top >= scores.shape[1]:
+        return torch.full((scores.shape[0],), math.inf, dtype=scores.dtype)
+    ranked = scores.sort(-1, descending=True).values
+    return ranked[:, top - 1] - ranked[:, top]
+
+
+def router_margin(config: dict, weights: Dict[str, torch.Tensor], tokens) -> float:
+    """The smallest margin over the sequence's tokens and layers; the tests assert that their weights leave a safe one, so
+    that an engine that rounds differently still chooses the same experts."""
+    seen: list = []
+    forward(config, weights, tokens, routers=seen)
+    return min([float(choice_margins(scores, top).min()) for top, scores in seen] + [math.inf])
+
+
+# ---- random weights for the tests -------------------------------------------------------------------------------------------
+def random_model(config: dict, seed: int, dtype=torch.float32, rank: Optional[int] = None) -> Dict[str, torch.Tensor]:
+    """Weights whose values are bfloat16 numbers.  The routers are made robust against rounding, so that a bfloat16
+    engine and this implementation choose the same experts: the first columns of the embedding carry, per token id, the
+    router's logits (a router's row e reads column e, plus a little of everything else), drawn again until every layer's
+    choice has a safe margin at every size the stream's norm may have; every tensor that writes into the stream is small
+    in those columns.  ``rank``: the inner size of the low-rank products (else one per product, all different)."""
+    g = torch.Generator().manual_seed(seed)
+    W, V = config["width"], config["vocab"]
+    groups = int(config["norm"].get("groups", 1))
+    mixtures = [(i, L["mlp"]) for i, L in enumerate(config["layers"]) if L.get("mlp") and L["mlp"]["kind"] == "moe"]
+    routes = {i: f["router"]["experts"] + int(f["router"].get("identity") or 0) for i, f in mixtures}
+    E_max = max(list(routes.values()) + [0])
+    assert E_max <= W // groups, "the router's columns lie in the first group of the norm"
+    ranks = iter(range(3, 1000, 2))
+
+    def low_rank():
+        return rank or next(ranks)
+
+    def mat(o, i, gain=1.0):
+        return (torch.randn(o, i, generator=g) * gain / math.sqrt(i)).bfloat16().to(dtype)
+
+    def vec(n, around=0.0, spread=0.1):
+        return (around + spread * torch.randn(n, generator=g)).bfloat16().to(dtype)
+
+    def taps(n, K):
+        return (torch.randn(n, K, generator=g) * 0.6).bfloat16().to(dtype)
+
+    def writer(i, gain=0.4):                         # [W, i]: output rows of the router's columns are small
+        m = torch.randn(W, i, generator=g) * gain / math.sqrt(i)
+        m[:E_max] *= 0.001
+        return m.bfloat16().to(dtype)
+
+    t: Dict[str, torch.Tensor] = {"head": mat(V, W, 2.0), "final.norm": vec(W, 1.0)}
+    corrections = {}
+    for i, f in mixtures:
+        corrections[i] = (0.1 * torch.randn(routes[i], generator=g)).bfloat16().double()
+        t[f"l{i}.mlp.correction"] = corrections[i].to(dtype)
+    embed = torch.randn(V, W, generator=g)
+    if E_max:
+        accepted = torch.zeros(0, E_max, dtype=torch.float64)
+        for _ in range(400):
+            if len(accepted) >= V:
+                break
+            cand = ((torch.rand(8192, E_max, generator=g) * 2 - 1) * 1.5).bfloat16().double()
+            for stride in (12, 1):                                # a coarse look first, then the whole range
+                for i, f in mixtures:
+                    for step in range(0, 72, stride):             # logits = 2 * column / rms(stream): 0.15 to 3.2
+                        z = cand[:, :routes[i]] * 0.15 * 2.0 ** (step / 16)
+                        cand = cand[choice_margins(torch.softmax(z, -1) + corrections[i], f["router"]["top"]) > 0.011]
+            accepted = torch.cat([accepted, cand])
+        assert len(accepted) >= V, "no safe logits found for some token ids"
+        embed[:, :E_max] = accepted[:V].float()
+    t["embed"] = embed.bfloat16().to(dtype)
+    for i, L in enumerate(config["layers"]):
+        p = f"l{i}."
+        m = L["mixer"]
+        t[p + "norm1"] = vec(W, 1.0)
+        t[p + "norm1"][:E_max] = 1.0
+        if L["type"] == "attention":
+            H, G, d, dv, K = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
+            rows = [("q", H * d, 2.0)] + ([("k", G * d, 2.0), ("v", G * dv, 1.0)] if m.get("kv_from") is None else [])
+            for n, size, gain in rows:
+                t[p + f"mix.{n}"], t[p + f"mix.{n}.b"], t[p + f"mix.{n}.conv"] = mat(size, W, gain), vec(size, 0.0, 0.5), taps(size, K)
+            t[p + "mix.pb"], t[p + "mix.g"], t[p + "mix.o"] = vec(H, -4.0, 0.7), mat(H, W, 2.0), writer(H * dv)
+        elif L["type"] == "parallel":
+            a, b = m["left"], m["right"]
+            H, G, d, dv = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            q = p + "mix.left."
+            t[q + "q"], t[q + "k"], t[q + "v"], t[q + "g"] = mat(H * d, W, 2.0), mat(G * d, W, 2.0), mat(G * dv, W), mat(H * dv, W, 2.0)
+            t[q + "r1"], t[q + "r2"], t[q + "o"] = vec(H, 0.6, 0.3), vec(H, 0.5, 0.1).abs(), writer(H * dv)
+            H, G, d, dv, K = b["heads"], b["kv_heads"], b["dim"], b["vdim"], b["conv"]
+            q = p + "mix.right."
+            for n, size in (("q", G * d), ("k", G * d), ("v", H * dv)):
+                t[q + n], t[q + n + ".conv"] = mat(size, W, 2.0), taps(size, K)
+            ra, rg = low_rank(), low_rank()
+            t[q + "b"], t[q + "A_log"], t[q + "dt_bias"] = mat(H, W, 2.0), vec(H, -1.0, 0.7), vec(H * d, 0.0, 1.0)
+            t[q + "a1"], t[q + "a2"], t[q + "g1"], t[q + "g2"] = mat(ra, W, 2.0), mat(H * d, ra), mat(rg, W, 2.0), mat(H * dv, rg)
+            t[q + "norm"], t[q + "o"] = vec(dv, 1.0), writer(H * dv)
+            for side in ("left", "right"):
+                out = vec(W, 0.6)
+                out[:E_max] = 0.001
+                t[p + f"mix.{side}.out"] = out
+        else:
+            H, d = m["heads"], m["dim"]
+            q = p + "mix."
+            for s in "rkvgw":
+                t[q + f"mu.{s}"] = torch.rand(W, generator=g).bfloat16().to(dtype)
+            for s in "rkvg":
+                t[q + s] = mat(H * d, W, 1.0)
+            r = low_rank()
+            t[q + "w1"], t[q + "w2"], t[q + "w0"] = mat(r, W, 2.0), mat(H * d, r), vec(H * d, -1.5, 1.0)
+            t[q + "u"], t[q + "norm"], t[q + "o"] = vec(H * d, 0.0, 0.7).view(H, d), vec(H * d, 1.0), writer(H * d)
+        f = L.get("mlp")
+        if f and f["kind"] == "dense":
+            t[p + "mlp.gate"], t[p + "mlp.up"], t[p + "mlp.down"] = mat(f["ff"], W, 1.5), mat(f["ff"], W, 1.5), writer(f["ff"])
+        elif f:
+            ff = f["expert"]["ff"]
+            for e in range(f["router"]["experts"]):
+                t[f"{p}mlp.e{e}.gate"], t[f"{p}mlp.e{e}.up"], t[f"{p}mlp.e{e}.down"] = mat(ff, W, 1.5), mat(ff, W, 1.5), writer(ff)
+            router = torch.randn(routes[i], W, generator=g) * 0.008 / math.sqrt(W)
+            router[:, :E_max] = 0.0
+            for e in range(routes[i]):
+                router[e, e] = 2.0
+            t[p + "mlp.router"] = router.bfloat16().to(dtype)
+    return t

@@ -1,0 +1,821 @@
+"""Nugolorn through the engine against the plain implementation (``plain_nugolorn``), mechanism by mechanism and as a
+whole: every way of cutting the work, pages and slots that are used again, keys far away and at page borders, the first
+tokens of a sequence, keys and values that a later layer reads from an earlier one's cache, convolution, shift and matrix
+states carried over portions of every size, identity experts, sizes that are odd, equal to one or absent, and greedy
+generation through the entry point and the scheduler.
+"""
+from __future__ import annotations
+
+import json
+import math
+import os
+
+import numpy as np
+import pytest
+import torch
+
+import plain_nugolorn as plain
+import traces
+from conftest import note_error, random_tokens
+
+pytestmark = pytest.mark.gpu
+
+
+def _attention(heads, kv_heads, dim, vdim, scale, conv, rot=None, kv_from=None, mlp=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "conv": conv}
+    if rot:
+        m["rot"] = {"base": rot[0], "dims": rot[1]}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "attention", "mixer": m, "mlp": mlp}
+
+
+def _pair(left, right, temp=None, mlp=None):
+    """``left = (heads, kv_heads, dim, vdim, scale)``, ``right = (heads, kv_heads, dim, vdim, conv)``."""
+    a = dict(zip(("heads", "kv_heads", "dim", "vdim", "scale"), left))
+    if temp:
+        a["q_temp"] = {"coef": temp[0], "every": temp[1]}
+    return {"type": "parallel", "mixer": {"left": a, "right": dict(zip(("heads", "kv_heads", "dim", "vdim", "conv"), right))}, "mlp": mlp}
+
+
+def _wkv(heads, dim, mlp=None):
+    return {"type": "wkv", "mixer": {"heads": heads, "dim": dim}, "mlp": mlp}
+
+
+def _dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def _moe(experts, top, ff, identity=0):
+    return {"kind": "moe", "router": {"experts": experts, "top": top, "identity": identity}, "expert": {"ff": ff}}
+
+
+def _config(vocab, width, layers, groups=1, eps=1e-6, mult=1.0, logits=1.0):
+    return {"architecture": "Nugolorn", "vocab": vocab, "width": width, "norm": {"eps": eps, "groups": groups},
+            "residual_mult": mult, "logit_scale": logits, "layers": layers}
+
+
+# odd sizes everywhere, three groups; the reader has another convolution than its source; as many experts chosen as there are
+ODD = _config(97, 72, [
+    _attention(4, 2, 12, 10, 0.3, 3, (100.0, 8), mlp=_moe(6, 3, 20, 2)),
+    _wkv(3, 20, mlp=None),
+    _pair((3, 3, 10, 14, 0.25), (4, 2, 12, 6, 2), (0.25, 7), mlp=_dense(36)),
+    _attention(4, 2, 12, 10, 0.35, 5, (100.0, 8), kv_from=0, mlp=_moe(4, 4, 28)),
+    _wkv(1, 40, mlp=_dense(28)),
+], groups=3, eps=1e-5, mult=0.7, logits=1.3)
+# the pair first; one group, no factors, no rotation, convolutions of one tap, no temperature; more identity experts than
+# others and one chosen; a layer read by two; one key head; pages of 32
+LATE = _config(300, 128, [
+    _pair((2, 1, 32, 16, 0.2), (2, 2, 16, 32, 1), mlp=_moe(3, 1, 32, 5)),
+    _attention(4, 4, 16, 24, 0.3, 1, mlp=_dense(64)),
+    _attention(4, 4, 16, 24, 0.25, 2, kv_from=1, mlp=None),
+    _wkv(2, 48, mlp=_moe(5, 2, 24, 1)),
+    _attention(4, 4, 16, 24, 0.2, 4, kv_from=1, mlp=_dense(40)),
+])
+# sizes in multiples of 64, for the tensor-core paths in bfloat16 (both forms of the attention, grouped experts, tcgen05
+# projections, the library's batched product); keys of 256 in a scan
+WIDE = _config(768, 384, [
+    _attention(8, 2, 64, 32, 0.12, 4, (1e4, 32), mlp=_moe(6, 2, 128, 2)),
+    _pair((4, 2, 128, 64, 0.09), (4, 2, 64, 64, 4), (0.2, 32), mlp=_dense(512)),
+    _wkv(3, 128, mlp=_moe(8, 3, 64, 1)),
+    _attention(8, 2, 64, 32, 0.15, 4, (1e4, 32), kv_from=0, mlp=_dense(320)),
+    _pair((6, 6, 64, 128, 0.12), (2, 1, 256, 32, 3), mlp=None),
+], groups=4, mult=0.4, logits=0.5)
+MODELS = {"odd": (ODD, 16, 41), "late": (LATE, 32, 42), "wide": (WIDE, 16, 43)}
+
+# Largest error of a row of logits (see _row_error).  float32: only the order of sums differs, and the angle, which the
+# engine takes in 32 bits as the design says and the plain model in 64.  bfloat16: the engine rounds where it stores
+# (normed rows, projections, cached rows, mixer outputs, activations).
+TOLERANCE = {"float32": 1.5e-5, "bfloat16": 6e-2}
+# Between two ways of cutting the same request the engine may differ only by which kernel a step's size selects.
+CUT_TOLERANCE = {"float32": 1e-5, "bfloat16": 6e-2}
+MARGIN = 0.0025        # what the routers of the test models must leave (see plain.choice_margins)
+
+
+def _write(folder, cfg, tensors, dtype):
+    from cuinfer_b200.weights.safetensors_io import write_safetensors
+
+    os.makedirs(folder, exist_ok=True)
+    store = {k: v.to(torch.bfloat16 if dtype == "bfloat16" else torch.float32) for k, v in tensors.items()}
+    write_safetensors(os.path.join(folder, "model.safetensors"), store)
+    with open(os.path.join(folder, "config.json"), "w") as fh:
+        json.dump(cfg, fh)
+    return folder
+
+
+@pytest.fixture(scope="module")
+def folders(tmp_path_factory):
+    """{name: (config, {dtype: folder}, tensors in float64, page size)}; the values are bfloat16 numbers, so that both
+    engines and the plain implementation read the same weights."""
+    out = {}
+    for name, (cfg, block, seed) in MODELS.items():
+        tensors = plain.random_model(cfg, seed, rank=16 if name == "wide" else None)
+        dirs = {d: _write(str(tmp_path_factory.mktemp(f"nugolorn_{name}_{d}")), cfg, tensors, d) for d in TOLERANCE}
+        out[name] = (cfg, dirs, {k: v.double() for k, v in tensors.items()}, block)
+    return out
+
+
+def _row_error(row, ref):
+    """Root mean square of the difference over the vocabulary, the common offset taken off (it changes no probability),
+    as a fraction of the root mean square of the plain logits about their mean."""
+    d = row.astype(np.float64) - ref
+    return float(np.sqrt(((d - d.mean()) ** 2).mean()) / np.sqrt(((ref - ref.mean()) ** 2).mean()))
+
+
+def _requests(cfg, lengths, seed):
+    return {f"r{i}": random_tokens(cfg["vocab"], n, seed * 100 + i) for i, n in enumerate(lengths)}
+
+
+_PLAIN, _WHOLE = {}, {}
+
+
+def _plain_rows(cfg, tensors, toks):
+    """Plain logits of a request; the routers along it must not rest on a close call."""
+    key = (id(tensors), tuple(toks))
+    if key not in _PLAIN:
+        routers = []
+        rows = plain.forward(cfg, tensors, list(toks), routers=routers).numpy()
+        _PLAIN[key] = (rows, min([float(plain.choice_margins(s, top).min()) for top, s in routers] + [math.inf]))
+    return _PLAIN[key]
+
+
+def _whole_rows(folders, name, dtype, rid, toks, tmp_path):
+    """The engine's own logits of a request fed whole and alone."""
+    key = (name, dtype, tuple(toks))
+    if key not in _WHOLE:
+        cfg, dirs, _tensors, block = folders[name]
+        steps = traces.whole({rid: toks})
+        out = str(tmp_path / f"whole_{name}_{dtype}_{rid}")
+        traces.replay_in_process(dirs[dtype], dtype, steps, out, traces.live_token_peak(steps), block)
+        _WHOLE[key] = traces.collect(steps, out, cfg["vocab"])[rid]
+    return _WHOLE[key]
+
+
+def _check(folders, name, dtype, steps, requests, tmp_path, max_tokens=None, **kw):
+    """Every row against the plain implementation, and against the engine's own logits of the request fed whole."""
+    cfg, dirs, tensors, block = folders[name]
+    out = str(tmp_path / f"out_{name}_{dtype}")
+    runner = traces.replay_in_process(dirs[dtype], dtype, steps, out, max_tokens or traces.live_token_peak(steps), block, **kw)
+    got = traces.collect(steps, out, cfg["vocab"])
+    worst = 0.0
+    for rid, toks in requests.items():
+        ref, margin = _plain_rows(cfg, tensors, toks)
+        assert margin > MARGIN, f"the test's routers must not rest on a close call ({margin:.2e})"
+        assert sorted(got.get(rid, {})) == list(range(len(toks)))
+        whole = _whole_rows(folders, name, dtype, rid, list(toks), tmp_path)
+        for pos, row in sorted(got[rid].items()):
+            assert np.isfinite(row).all(), f"request {rid} position {pos}: logits are not finite"
+            cut = _row_error(row, whole[pos].astype(np.float64))
+            assert cut <= CUT_TOLERANCE[dtype], f"{name}/{dtype}: request {rid}: position {pos} of {len(toks)} depends on how the work was cut ({cut:.3e})"
+            err = _row_error(row, ref[pos])
+            assert err <= TOLERANCE[dtype], f"{name}/{dtype}: request {rid}: first wrong position {pos} of {len(toks)} (error {err:.3e})"
+            worst = max(worst, err)
+    note_error(dtype, f"model {name}", worst, family="Nugolorn")
+    return runner
+
+
+NAMES, DTYPES = list(MODELS), list(TOLERANCE)
+
+
+# ---- the whole model under every way of cutting the work ------------------------------------------------------------
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_whole_prompts(folders, name, dtype, tmp_path):
+    requests = _requests(folders[name][0], [1, 2, 17, 33, 150], seed=1)
+    _check(folders, name, dtype, traces.whole(requests), requests, tmp_path)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_prefill_then_token_by_token(folders, name, dtype, tmp_path):
+    requests = _requests(folders[name][0], [40, 131], seed=2)
+    _check(folders, name, dtype, traces.tail_decode(requests, 60), requests, tmp_path)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_portions_down_to_two_tokens(folders, name, dtype, tmp_path):
+    """Portions shorter than the convolutions and longer, with single tokens between them."""
+    requests = _requests(folders[name][0], [64, 131, 90], seed=3)
+    _check(folders, name, dtype, traces.portions(requests), requests, tmp_path)
+    _check(folders, name, dtype, traces.portions(requests, sizes=(2, 3, 1, 2, 16, 1, 1, 40)), requests, tmp_path)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", NAMES)
+def test_mixed_batches_reuse_pages_and_slots(folders, name, dtype, tmp_path):
+    requests = _requests(folders[name][0], [70, 33, 120, 58, 90, 45, 101], seed=4)
+    steps = traces.mixed(requests, max_live=4)
+    peak = traces.live_token_peak(steps)
+    assert peak < sum((len(t) + 63) // 64 * 64 for t in requests.values()), "pages must be used again"
+    runner = _check(folders, name, dtype, steps, requests, tmp_path, max_tokens=peak, max_live=4)
+    assert runner.num_pages * runner.page_size == peak and runner.manager.slots.num_slots == 4
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_long_decoding_from_the_first_token(folders, dtype, tmp_path):
+    requests = _requests(folders["odd"][0], [200], seed=5)
+    _check(folders, "odd", dtype, traces.tail_decode(requests, 199), requests, tmp_path)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["odd", "wide"])
+def test_a_long_prompt_then_decoding(folders, name, dtype, tmp_path):
+    """Seven hundred tokens: many key tiles a query and many chunks of the scans; most of it in one step, then token by
+    token; and cut into portions throughout."""
+    requests = _requests(folders[name][0], [700], seed=10)
+    _check(folders, name, dtype, traces.tail_decode(requests, 30), requests, tmp_path)
+    _check(folders, name, dtype, traces.portions(requests, sizes=(130, 2, 64, 3, 257, 16)), requests, tmp_path)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["wide", "odd"])
+def test_steps_through_cuda_graphs(folders, name, dtype, tmp_path):
+    """The same logits when decode steps and repeated step shapes are replayed from graphs, as generation runs them:
+    padding rows and the padding request own no slot and no page."""
+    requests = _requests(folders[name][0], [70, 40, 90, 33], seed=6)
+    steps = traces.mixed(requests, max_live=3, sizes=(32, 40, 35))
+    runner = _check(folders, name, dtype, steps, requests, tmp_path, cuda_graph=True, passes=2, max_live=4)
+    assert runner.model.capturable and runner.graph_steps + runner.step_graph_replays > 0
+
+
+@pytest.mark.parametrize("graphs", [False, True])
+def test_many_requests_decoding_together(folders, graphs, tmp_path):
+    """Nineteen requests decode side by side (more rows than the few-rows product takes), eagerly and from a graph whose
+    bucket has padding rows."""
+    requests = _requests(folders["wide"][0], [20 + 3 * i for i in range(19)], seed=8)
+    heads = {rid: len(t) - 5 for rid, t in requests.items()}
+    steps = [{"step": 0, "entries": [{"id": rid, "tokens": t[:heads[rid]], "want": list(range(heads[rid]))} for rid, t in requests.items()], "end": []}]
+    for k in range(5):
+        steps.append({"step": k + 1, "entries": [{"id": rid, "tokens": [t[heads[rid] + k]], "want": [0]} for rid, t in requests.items()],
+                      "end": list(requests) if k == 4 else []})
+    runner = _check(folders, "wide", "bfloat16", steps, requests, tmp_path, cuda_graph=graphs, passes=2 if graphs else 1, max_live=20)
+    assert not graphs or runner.graph_steps > 0
+
+
+def test_the_stream_after_every_layer(folders):
+    """The residual stream after each layer of a short prompt, in 32 bits, against the plain model's."""
+    from cuinfer_b200.engine import replay
+    from cuinfer_b200.engine.runner import StepEntry
+
+    for name in NAMES:
+        cfg, dirs, tensors, block = folders[name]
+        toks = random_tokens(cfg["vocab"], 29, 77)
+        want = []
+        plain.forward(cfg, tensors, toks, tap=lambda i, x: want.append(x.clone()))
+        runner = replay.make_runner(dirs["float32"], "float32", 64, block)
+        entries = [StepEntry("a", toks, [0])]
+        assert runner.reserve("a", len(toks))
+        runner.storage.zero_slots(runner.manager.take_newly_admitted())
+        ctx, _ = runner.build_context(entries)
+        got = []
+        runner.model.forward(ctx, tap=lambda run, stream: got.append(stream.collapsed().double().cpu()))
+        assert len(got) == len(want) == len(cfg["layers"])
+        for i, (g, w) in enumerate(zip(got, want)):
+            err = float((g - w).abs().max() / w.abs().max())
+            assert err < 1e-5, f"{name}: the stream after layer {i} is off by {err:.3e}"
+
+
+def test_greedy_generation_through_the_entry_point(folders):
+    from cuinfer_b200 import LLM, SamplingParams
+
+    for name in ("odd", "late"):
+        cfg, dirs, tensors, block = folders[name]
+        prompts = [random_tokens(cfg["vocab"], n, 70 + n) for n in (3, 19, 8)]
+        llm = LLM(dirs["float32"], dtype="float32", block_size=block, num_blocks=24, max_num_seqs=3, max_num_scheduled_tokens=16)
+        outs = llm.generate(prompts, SamplingParams(max_tokens=12, temperature=0.0, ignore_eos=True))
+        for prompt, out in zip(prompts, outs):
+            assert out.token_ids == plain.greedy(cfg, tensors, prompt, 12), f"{name}: prompt of {len(prompt)} tokens"
+
+
+def test_command_line(folders):
+    import subprocess
+    import sys
+
+    from conftest import ROOT
+
+    cfg, dirs, tensors, block = folders["late"]
+    prompt = random_tokens(cfg["vocab"], 9, 95)
+    proc = subprocess.run([sys.executable, "-m", "cuinfer_b200", "generate", "--model", dirs["float32"], "--dtype", "float32",
+                           "--prompt-ids", ",".join(map(str, prompt)), "--max-tokens", "5", "--temperature", "0", "--ignore-eos",
+                           "--num-blocks", "16", "--max-num-seqs", "4", "--block-size", str(block)],
+                          capture_output=True, text=True, cwd=ROOT, timeout=900)
+    assert proc.returncode == 0, proc.stderr[-2000:]
+    line = [json.loads(l) for l in proc.stdout.splitlines() if l.startswith("{")][0]
+    assert line["token_ids"] == plain.greedy(cfg, tensors, prompt, 5)
+
+
+# ---- mechanisms alone -------------------------------------------------------------------------------------------------
+def _dev(t, dtype):
+    return t.to(device="cuda", dtype=dtype).contiguous()
+
+
+def _close(got, want, dtype, what, tol=None):
+    tol = tol or (2e-5 if dtype == torch.float32 else 2e-2)
+    assert torch.isfinite(got.float()).all(), f"{what}: not finite"
+    err = float((got.double().cpu() - want).abs().max() / want.abs().max().clamp_min(1e-9))
+    assert err <= tol, f"{what} in {dtype}: error {err:.3e} of the largest value"
+
+
+def _ints(values):
+    return torch.tensor(values, dtype=torch.int32, device="cuda")
+
+
+BOTH = [torch.float32, torch.bfloat16]
+
+
+@pytest.mark.parametrize("dtype", BOTH)
+@pytest.mark.parametrize("rows,W,groups", [(3, 72, 3), (3, 70, 2), (300, 64, 4), (97, 4096, 2), (5, 5000, 1), (260, 33, 3), (1, 8, 8), (40, 1536, 12)])
+def test_scaled_sum_of_two_deltas_and_norm_in_groups(dtype, rows, W, groups):
+    from cuinfer_b200 import kernels
+
+    g = torch.Generator().manual_seed(rows + W)
+    x = torch.randn(rows, W, generator=g).float()
+    x[:, :W // groups] *= 30.0                                      # parts of very different size: each has its own mean square
+    a, b = torch.randn(rows, W, generator=g).to(dtype), torch.randn(rows, W, generator=g).to(dtype)
+    gain = (1 + 0.3 * torch.randn(W, generator=g)).bfloat16()
+    for deltas, scale in (((None, None), 1.0), ((a, None), 0.3), ((a, b), -0.7)):
+        res = x.clone().cuda()
+        dev = [None if d is None else d.cuda() for d in deltas]
+        out = torch.empty(rows, W, dtype=dtype, device="cuda")
+        kernels.group_rms(res, *dev, scale, (gain.cuda(), 1e-3), groups, out)
+        want = x.double() + scale * sum([d.double() for d in deltas if d is not None], torch.zeros(rows, W, dtype=torch.float64))
+        _close(res, want, torch.float32, "the sum", tol=1e-6)
+        _close(out, plain.group_rms_norm(want, gain.double(), 1e-3, groups), dtype, f"norm in {groups} groups", tol=1e-5 if dtype == torch.float32 else 8e-3)
+        idx = _ints([rows - 1, 0, rows // 2])
+        picked = torch.empty(3, W, dtype=torch.float32, device="cuda")
+        kernels.gather_rows(x.cuda(), dev[0], idx, picked, delta2=dev[1], scale=scale)
+        _close(picked, want[idx.cpu().long()], torch.float32, "gathered rows", tol=1e-6)
+        alone = x.clone().cuda()
+        kernels.group_rms(alone, *dev, scale, None, 1, None)
+        assert torch.equal(alone, res) if deltas[0] is not None else torch.equal(alone.cpu(), x)
+
+
+@pytest.mark.parametrize("dtype", BOTH)
+@pytest.mark.parametrize("rows,W", [(3, 72), (1, 35), (200, 384), (2, 5000)])
+def test_half_the_sum_of_two_normed_rows_and_tanh(dtype, rows, W):
+    from cuinfer_b200 import kernels
+
+    g = torch.Generator().manual_seed(W)
+    a, b = (torch.randn(rows, W, generator=g) * 5).to(dtype), (torch.randn(rows, W, generator=g) * 0.01).to(dtype)
+    ga, gb = torch.randn(W, generator=g), torch.randn(W, generator=g)
+    out = torch.empty(rows, W, dtype=dtype, device="cuda")
+    kernels.pair_rms_mean(a.cuda(), b.cuda(), ga.cuda(), gb.cuda(), 1e-5, out)
+    _close(out, 0.5 * (plain.rms(a.double(), 1e-5) * ga.double() + plain.rms(b.double(), 1e-5) * gb.double()), dtype, "half the sum",
+           tol=1e-5 if dtype == torch.float32 else 8e-3)
+    z = torch.randn(rows, W + 3, generator=g) * 3
+    kernels.tanh_rows(z.cuda(), out)
+    _close(out, torch.tanh(z[:, :W].double()), dtype, "tanh", tol=1e-6 if dtype == torch.float32 else 8e-3)
+
+
+@pytest.mark.parametrize("E,identity,top", [(6, 2, 3), (3, 5, 1), (4, 0, 4), (130, 7, 9), (1, 1, 2), (1000, 24, 8)])
+def test_softmax_scores_with_correction_and_identity_experts(E, identity, top):
+    """Choice by softmax score over all plus correction, weights by the score alone; the weights of the chosen identity
+    experts are summed."""
+    from cuinfer_b200 import kernels
+
+    g = torch.Generator().manual_seed(E)
+    T, N = 67, E + identity
+    z = (torch.randn(T, N + 3, generator=g) * 2).float()
+    z[5] += 200.0                                                   # a large common offset changes nothing
+    corr = (torch.randn(N, generator=g) * (0.5 if N < 100 else 0.02)).float()
+    choice = torch.empty(T, top, dtype=torch.int32, device="cuda")
+    weight = torch.empty(T, top, dtype=torch.float32, device="cuda")
+    kept = torch.full((T,), -1.0, dtype=torch.float32, device="cuda")
+    kernels.router_scored_topk(z.cuda()[:, :N], top, choice, weight, correction=corr.cuda(), softmax=True, identity_from=E, identity_weight=kept)
+    margins = plain.choice_margins(torch.softmax(z[:, :N].double(), -1) + corr.double(), top)
+    checked = 0
+    for t in range(T):
+        if margins[t] < 1e-5:
+            continue                                    # a close call in float32 may fall either way
+        want, scores = plain.choose_experts(z[t, :N].double(), corr.double(), top)
+        assert choice[t].tolist() == want, f"token {t}: chose {choice[t].tolist()}, plain {want}"
+        assert np.allclose(weight[t].cpu().numpy(), scores.numpy(), rtol=2e-5, atol=1e-7)
+        assert abs(float(kept[t]) - float(sum([s for e, s in zip(want, scores) if e >= E], torch.tensor(0.0)))) < 1e-5
+        checked += 1
+    assert checked > T // 2
+
+
+@pytest.mark.parametrize("dtype", BOTH)
+@pytest.mark.parametrize("W,ff,E,identity,top,T", [(72, 36, 5, 2, 3, 9), (64, 32, 3, 3, 2, 300), (128, 96, 9, 1, 1, 700), (40, 24, 1, 2, 2, 5)])
+def test_experts_that_give_back_their_input(dtype, W, ff, E, identity, top, T):
+    """``sum_k w_k expert_k(h) + (sum of identity weights) h`` on both expert paths, with tokens whose choices are all
+    identity experts."""
+    from cuinfer_b200 import kernels
+
+    g = torch.Generator().manual_seed(W + T)
+    h = torch.randn(T, W, generator=g).to(dtype).double()
+    gate, up = ((torch.randn(E, ff, W, generator=g) / math.sqrt(W)).to(dtype).double() for _ in range(2))
+    down = (torch.randn(E, W, ff, generator=g) / math.sqrt(ff)).to(dtype).double()
+    choice = torch.stack([torch.randperm(E + identity, generator=g)[:top] for _ in range(T)]).to(torch.int32)
+    if identity >= top:
+        choice[1] = torch.arange(E, E + top)
+    weights = torch.rand(T, top, generator=g).float()
+    kept = (weights * (choice >= E)).sum(-1)
+    want = torch.zeros(T, W, dtype=torch.float64)
+    for t in range(T):
+        for k in range(top):
+            e = int(choice[t, k])
+            want[t] += float(weights[t, k]) * (plain.gated_ff(h[t:t + 1], gate[e], up[e], down[e])[0] if e < E else h[t])
+    out = torch.empty(T, W, dtype=dtype, device="cuda")
+    kernels.moe_table_feed_forward(_dev(h, dtype), None, choice.cuda(), _dev(torch.cat([gate, up], 1), dtype), _dev(down, dtype),
+                                   _dev(h, dtype), out, weights=weights.cuda(), base_gate=kept.cuda(), base_gate_plain=True)
+    _close(out, want, dtype, "experts beside identity experts", tol=3e-5 if dtype == torch.float32 else 3e-2)
+
+
+# ---- the step before the attention: bias, convolution, rotation, cache --------------------------------------------------
+def _angles32(position, freqs):
+    """The design takes the angle in 32 bits: position times frequency, both float32.  The plain rotation gets those
+    angles as "frequencies" at "position" one."""
+    return (torch.tensor(float(position), dtype=torch.float32) * torch.tensor(freqs, dtype=torch.float32)).double().tolist()
+
+
+def _rotated(x, positions, freqs):
+    out = torch.empty_like(x)
+    for t in range(x.shape[0]):
+        out[t] = plain.rotate_halves(x[t:t + 1], torch.ones(1), _angles32(positions[t], freqs))[0]
+    return out
+
+
+@pytest.mark.parametrize("dtype", BOTH)
+@pytest.mark.parametrize("q_only", [False, True])
+@pytest.mark.parametrize("K,H,G,d,dv,dims", [(4, 4, 2, 10, 7, 6), (1, 3, 3, 8, 12, 0), (2, 2, 1, 64, 64, 64), (6, 4, 2, 20, 33, 20), (3, 2, 2, 130, 6, 64)])
+def test_convolution_before_the_rotation(dtype, q_only, K, H, G, d, dv, dims):
+    """Two requests fed in portions of one, two and more tokens (and a padding request that owns no slot): bias, then the
+    convolution over what came before, in this step or in the state, then the rotation; keys and values land in the
+    cache, queries in rows of their own, the projected rows stay.  A slot that nobody owns keeps its state."""
+    from cuinfer_b200 import kernels
+
+    g = torch.Generator().manual_seed(K * 10 + d)
+    page, lengths = 4, [23, 14]
+    columns = H * d + (0 if q_only else G * (d + dv))
+    full = [torch.randn(n, columns + 5, generator=g).to(dtype) for n in lengths]
+    bias = torch.randn(columns, generator=g).float()
+    taps = (torch.randn(columns, K, generator=g) * 0.7).bfloat16().float()
+    freqs = plain.rotary_frequencies(50.0, dims)
+    want = []
+    for rows in full:
+        y = plain.causal_conv(rows[:, :columns].double() + bias.double(), taps.double())
+        n = len(rows)
+        parts = [_rotated(y[:, :H * d].view(n, H, d), range(n), freqs)]
+        if not q_only:
+            parts += [_rotated(y[:, H * d:(H + G) * d].view(n, G, d), range(n), freqs), y[:, (H + G) * d:].view(n, G, dv)]
+        want.append(parts)
+    state = torch.full((5, max(K - 1, 1), columns), 9.0, dtype=torch.float32, device="cuda")
+    slots = [3, 1]
+    state[slots] = 0.0
+    cache = torch.zeros(2, 8, 1, G, page, d + dv, dtype=dtype, device="cuda")[0]
+    freq = torch.tensor(freqs, dtype=torch.float32).cuda() if dims else None
+    done = [0, 0]
+    for new in ([2, 1], [1, 1], [1, 2], [7, 3], [1, 1], [5, 0], [6, 6]):
+        rows = torch.cat([full[r][done[r]:done[r] + n] for r, n in enumerate(new)] + [torch.ones(2, columns + 5).to(dtype)]).cuda()
+        pos = [p for r, n in enumerate(new) for p in range(done[r], done[r] + n)] + [0, 1]
+        treq = [r for r, n in enumerate(new) for _ in range(n)] + [2, 2]
+        qsl = [0, new[0], sum(new), sum(new) + 2]
+        place = [(r * 16 + p) % 32 for r, p in zip(treq[:-2], pos[:-2])] + [-1, -1]
+        one = all(n == 1 for n in new)
+        if one:                                                       # the padding request brings one token as well
+            rows, pos, treq, qsl, place = rows[:-1], pos[:-1], treq[:-1], qsl[:-1] + [qsl[-1] - 1], place[:-1]
+        before = rows.clone()
+        q_out = torch.empty(rows.shape[0], H * d, dtype=dtype, device="cuda")
+        conv = kernels.ShortConv(taps.t().contiguous().cuda(), state, _ints(qsl), _ints(treq), _ints(slots + [-1]), one_token_each=one)
+        kernels.window_attention_prep(rows, _ints(pos), None if q_only else _ints(place), freq, dims, 1e-6, H, G, d, dv, None, None,
+                                      None if q_only else cache, bias=bias.cuda(), norm=False, rot_half=True, q_only=q_only, q_out=q_out, conv=conv)
+        assert torch.equal(rows, before)
+        for i, (r, p) in enumerate(zip(treq, pos)):
+            if r == 2:
+                continue
+            _close(q_out[i].view(H, d), want[r][0][p], dtype, f"queries of token {p} of request {r}")
+            if not q_only:
+                got = cache[place[i] // page, 0, :, place[i] % page]
+                _close(got[:, :d], want[r][1][p], dtype, f"keys of token {p} of request {r}")
+                _close(got[:, d:], want[r][2][p], dtype, f"values of token {p} of request {r}")
+        done = [a + b for a, b in zip(done, new)]
+        if K > 1:
+            for r in range(2):
+                past = torch.zeros(K - 1, columns, dtype=torch.float64)
+                have = min(K - 1, done[r])
+                if have:
+                    past[K - 1 - have:] = full[r][done[r] - have:done[r], :columns].double() + bias.double()
+                _close(state[slots[r]], past, torch.float32, f"state of request {r} after {done[r]} tokens", tol=1e-6)
+    assert float((state[[0, 2, 4]] - 9.0).abs().max()) == 0.0, "a slot nobody owns changed"
+
+
+@pytest.mark.parametrize("dtype", BOTH)
+def test_rotation_at_far_positions_and_the_query_temperature(dtype):
+    from cuinfer_b200 import kernels
+
+    g = torch.Generator().manual_seed(2)
+    H, G, d, dv, dims = 2, 1, 12, 5, 8
+    positions = [0, 1, 5, 6, 7, 13, 1000, 70000]
+    rows = torch.randn(len(positions), H * d + G * (d + dv), generator=g).to(dtype)
+    freqs = plain.rotary_frequencies(300.0, dims)
+    cache = torch.zeros(2, 1, G, 8, d + dv, dtype=dtype, device="cuda")
+    dev = rows.cuda()
+    kernels.window_attention_prep(dev, _ints(positions), _ints(list(range(8))), torch.tensor(freqs, dtype=torch.float32).cuda(), dims, 1e-6,
+                                  H, G, d, dv, None, None, cache, norm=False, rot_half=True, q_temp=(0.4, 7))
+    temp = plain.query_temperature(positions, 0.4, 7, torch.float64)
+    assert len(set(temp.tolist())) == 5
+    q = _rotated(rows[:, :H * d].double().view(-1, H, d), positions, freqs) * temp[:, None, None]
+    for t in range(len(positions)):
+        _close(dev[t, :H * d].view(H, d), q[t], dtype, f"query at {positions[t]}", tol=1e-5 if dtype == torch.float32 else 8e-3)
+    k = _rotated(rows[:, H * d:(H + G) * d].double().view(-1, G, d), positions, freqs)
+    _close(cache[0, 0, 0, :, :d], k[:, 0], dtype, "keys", tol=1e-5 if dtype == torch.float32 else 8e-3)
+
+
+# ---- the two forms of attention over a paged cache -------------------------------------------------------------------------
+def _paged(g, lengths, page, heads, width, dtype, spare=3):
+    """A cache ``[pages, 1, heads, page, width]`` of random rows behind block tables in a shuffled order."""
+    pages_per = [-(-n // page) for n in lengths]
+    num_pages = sum(pages_per) + spare
+    perm = torch.randperm(num_pages, generator=g).tolist()
+    table = torch.full((len(lengths), max(pages_per)), -1, dtype=torch.int32)
+    cache = (torch.randn(num_pages, 1, heads, page, width, generator=g) * 0.5).to(dtype)
+    rows, at = {}, 0
+    for r, n in enumerate(lengths):
+        table[r, :pages_per[r]] = torch.tensor(perm[at:at + pages_per[r]], dtype=torch.int32)
+        at += pages_per[r]
+        rows[r] = torch.stack([cache[int(table[r, j // page]), 0, :, j % page] for j in range(n)]).double()     # [n, heads, width]
+    return cache, table, rows
+
+
+def _attention_case(form, dtype, H, G, d, dv, lengths, new, page, seed, sharpen=None, tensor_cores=False, splits=1, gate=None):
+    """``form``: "sigmoid" or "log"; ``sharpen = {token: key}``: the token's score with that key stands out for every head;
+    ``gate``: None, "head" or "value".  Returns the kernel's output and the plain result [T, H, dv]."""
+    from cuinfer_b200 import kernels
+
+    g = torch.Generator().manual_seed(seed)
+    cache, table, rows = _paged(g, lengths, page, G, d + dv, dtype)
+    pos = [p for n, k in zip(lengths, new) for p in range(n - k, n)]
+    treq = [r for r, k in enumerate(new) for _ in range(k)]
+    qsl = np.cumsum([0] + list(new)).tolist()
+    T = len(pos)
+    q = (torch.randn(T, H, d, generator=g) * 0.4).to(dtype).double()
+    scale = 0.8
+    for t, j in (sharpen or {}).items():
+        for h in range(H):
+            key = rows[treq[t]][j, h // (H // G), :d]
+            q[t, h] = (14.0 * key / key.norm() ** 2 / scale).to(dtype).double()
+    bias = (torch.randn(H, generator=g) - (7.0 if sharpen else 3.0)).float()
+    r1, r2 = (0.8 * torch.rand(H, generator=g)).float(), (torch.rand(H, generator=g) * 2).float()
+    r1[0] = 0.0
+    want = torch.zeros(T, H, dv, dtype=torch.float64)
+    for r, k in enumerate(new):
+        kv = rows[r]
+        sel = slice(qsl[r], qsl[r + 1])
+        if k:
+            want[sel] = (plain.sigmoid_attention(q[sel], kv[..., :d], kv[..., d:], scale, bias.double()) if form == "sigmoid"
+                         else plain.log_bias_attention(q[sel], kv[..., :d], kv[..., d:], scale, r1.double(), r2.double()))
+    gates = None
+    if gate:
+        wide = (torch.randn(T, 3 + H * dv, generator=g) * 2).to(dtype)
+        logits = wide[:, 3:3 + (H if gate == "head" else H * dv)]
+        want = want * torch.sigmoid(logits.double()).view(T, H, 1 if gate == "head" else dv)
+        gates = wide.cuda()[:, 3:3 + logits.shape[1]]
+    kw = {"sigmoid_bias": bias.cuda()} if form == "sigmoid" else {"log_bias": (r1.cuda(), r2.cuda())}
+    out = torch.empty(T, H * dv, dtype=dtype, device="cuda")
+    if tensor_cores:
+        assert kernels.window_attention_mma_supports(d, dv, H, G)
+        kernels.window_attention_mma(_dev(q.reshape(T, H * d), dtype), out, cache.cuda(), table.cuda(), _ints(qsl), _ints(lengths),
+                                     list(new), H, G, d, dv, scale, 0.0, 0, 0, splits=splits, gate=gates, **kw)
+    else:
+        kernels.window_attention_generic(_dev(q.reshape(T, H * d), dtype), out, cache.cuda(), table.cuda(), _ints(pos), _ints(treq),
+                                         H, G, d, dv, scale, 0.0, 0, 0, gate=gates, **kw)
+    return out.view(T, H, dv), want
+
+
+KERNELS = [(False, torch.float32), (False, torch.bfloat16), (True, torch.bfloat16)]
+
+
+@pytest.mark.parametrize("tensor_cores,dtype", KERNELS)
+@pytest.mark.parametrize("form", ["sigmoid", "log"])
+def test_one_far_key_among_hundreds(form, tensor_cores, dtype):
+    """The last query of a long request looks at ONE key — the first of the sequence, the last of a page, the first of the
+    next, both sides of a key tile, itself — in a prompt's portion and decoded alone (with its keys split over CTAs)."""
+    n, page = 700, 16
+    d, dv = (64, 32) if tensor_cores else (20, 9)
+    for j in (0, 1, page - 1, page, 63, 64, 333, n - 2, n - 1):
+        for new, t, splits in (([1, 1], 0, 3 if tensor_cores else 1), ([40, 2], 39, 1)):
+            got, want = _attention_case(form, dtype, 4, 2, d, dv, [n, 40], new, page, 10 + j, sharpen={t: j}, tensor_cores=tensor_cores, splits=splits)
+            _close(got, want, dtype, f"{form}: query at {n - 1} looking at key {j}")
+            assert float(want[t].abs().max()) > 0.2, "the case does not single a key out"
+
+
+@pytest.mark.parametrize("gate", [None, "head", "value"])
+@pytest.mark.parametrize("form", ["sigmoid", "log"])
+@pytest.mark.parametrize("H, G, d, dv, lengths, new, page, splits", [
+    (4, 2, 64, 32, [37, 1, 64, 129], [37, 1, 1, 5], 8, 1),              # prompts beside single tokens
+    (6, 6, 64, 128, [50, 33, 200], [2, 33, 100], 16, 1),
+    (4, 1, 128, 64, [300, 90], [170, 1], 16, 1),
+    (16, 1, 128, 128, [130, 7], [130, 7], 32, 1),                        # more rows than a tile per token pair
+    (8, 2, 64, 64, [700, 90, 33], [1, 1, 1], 16, 5),                     # a decode step: keys split, more splits than some have tiles
+    (2, 2, 128, 32, [70, 1, 200], [1, 1, 1], 16, 1),
+])
+def test_both_forms_on_both_kernels(form, gate, H, G, d, dv, lengths, new, page, splits):
+    got, want = _attention_case(form, torch.bfloat16, H, G, d, dv, lengths, new, page, seed=H, tensor_cores=True, splits=splits, gate=gate)
+    _close(got, want, torch.bfloat16, f"tensor-core attention, {form}")
+    for dtype in BOTH:
+        got, want = _attention_case(form, dtype, H, G, d, dv, lengths, new, page, seed=H, gate=gate)
+        _close(got, want, dtype, f"all-sizes attention, {form}")
+
+
+def test_sigmoid_weights_are_not_normalised():
+    """A key that is there twice counts twice, a number per head far below zero gives nothing and far above gives the sum."""
+    from cuinfer_b200 import kernels
+
+    for tensor_cores, d, dv, dtype in ((False, 6, 5, torch.float32), (True, 64, 32, torch.bfloat16)):
+        cache = torch.ones(4, 1, 1, 16, d + dv, dtype=dtype, device="cuda")
+        q = torch.zeros(1, 3 * d, dtype=dtype, device="cuda")
+        bias = torch.tensor([0.0, -90.0, 90.0], device="cuda")
+        out = torch.empty(1, 3 * dv, dtype=dtype, device="cuda")
+        args = (_ints([[2, 0, 3, 1]]),)
+        for n in (1, 10, 50):
+            if tensor_cores:
+                kernels.window_attention_mma(q, out, cache, *args, _ints([0, 1]), _ints([n]), [1], 3, 1, d, dv, 1.0, 0.0, 0, 0, sigmoid_bias=bias)
+            else:
+                kernels.window_attention_generic(q, out, cache, *args, _ints([n - 1]), _ints([0]), 3, 1, d, dv, 1.0, 0.0, 0, 0, sigmoid_bias=bias)
+            heads = out.view(3, dv).float().cpu()
+            assert torch.allclose(heads[0], torch.full((dv,), n / 2.0), rtol=1e-2)
+            assert float(heads[1].abs().max()) < 1e-6 and torch.allclose(heads[2], torch.full((dv,), float(n)), rtol=1e-2)
+
+
+# ---- the recurrences --------------------------------------------------------------------------------------------------------
+PORTIONS = ([2, 1, 3], [1, 1, 1], [17, 0, 2], [1, 33, 16], [4, 2, 1])
+
+
+@pytest.mark.parametrize("H,G,d,dv", [(4, 2, 12, 6), (2, 1, 32, 40), (3, 3, 50, 130), (2, 2, 128, 64), (2, 1, 200, 33), (1, 1, 1, 1)])
+def test_delta_rule_with_a_decay_per_channel(H, G, d, dv):
+    """Three requests in portions of none, one, two and more tokens, slots out of order, a slot nobody owns and a padding
+    request without one; channels that forget everything, nothing, and in between."""
+    from cuinfer_b200 import kernels
+
+    g = torch.Generator().manual_seed(H * d + dv)
+    totals = [sum(p[r] for p in PORTIONS) for r in range(3)]
+    C = 2 * G * d + H * dv
+    a_log, dt_bias = (torch.randn(H, generator=g) - 0.5).float(), torch.randn(H * d, generator=g).float()
+    data, want = [], []
+    for n in totals:
+        q, k = plain.unit(torch.randn(n, G, d, generator=g).double()) * d ** -0.5, plain.unit(torch.randn(n, G, d, generator=g).double())
+        v, zb, za = torch.randn(n, H, dv, generator=g).double(), torch.randn(n, H, generator=g).double(), torch.randn(n, H * d, generator=g).double() * 2
+        za[:, ::5] = 60.0                                             # decay 0: the channel forgets at once
+        za[:, 1::5] = -60.0                                           # decay 1
+        decay = torch.exp(-torch.exp(a_log.double())[None, :, None] * torch.nn.functional.softplus(za + dt_bias.double()).view(n, H, d))
+        want.append(plain.channel_delta_rule(q, k, v, torch.sigmoid(zb), decay))
+        data.append((torch.cat([q.reshape(n, -1), k.reshape(n, -1), v.reshape(n, -1)], 1).float(), zb.float(), za.float()))
+    state = torch.full((6, H, d * dv), 7.0, dtype=torch.float32, device="cuda")
+    slots = [4, 0, 2]
+    state[slots] = 0.0
+    done = [0, 0, 0]
+    for new in PORTIONS:
+        parts = [tuple(x[done[r]:done[r] + n] for x in data[r]) for r, n in enumerate(new)]
+        pad = (torch.ones(2, C), torch.zeros(2, H), torch.zeros(2, H * d))
+        qkv, zb, za = (torch.cat([p[i] for p in parts] + [pad[i]]) for i in range(3))
+        zb, za = torch.nn.functional.pad(zb, (0, 3)), torch.nn.functional.pad(za, (0, 2))         # rows wider than what is read
+        qsl = np.cumsum([0] + list(new) + [2]).tolist()
+        out = torch.empty(qkv.shape[0], H * dv, dtype=torch.float32, device="cuda")
+        kernels.channel_delta_scan(qkv.cuda(), zb.cuda(), za.cuda(), a_log.cuda(), dt_bias.cuda(), state, _ints(qsl), _ints(slots + [-1]), out, G, H, d, dv)
+        for r, n in enumerate(new):
+            if n:
+                _close(out[qsl[r]:qsl[r + 1]].view(n, H, dv), want[r][0][done[r]:done[r] + n], torch.float32, f"request {r} tokens {done[r]}..")
+            done[r] += n
+    for r in range(3):
+        _close(state[slots[r]].view(H, d, dv), want[r][1], torch.float32, f"state of request {r}")
+    assert float((state[[1, 3, 5]] - 7.0).abs().max()) == 0.0, "a slot nobody owns changed"
+
+
+@pytest.mark.parametrize("dtype", BOTH)
+@pytest.mark.parametrize("H,d", [(3, 20), (1, 40), (2, 64), (2, 128), (1, 200), (2, 1)])
+def test_time_mixing_scan(dtype, H, d):
+    from cuinfer_b200 import kernels
+
+    g = torch.Generator().manual_seed(H * d)
+    totals = [sum(p[r] for p in PORTIONS) for r in range(3)]
+    w0, u = (torch.randn(H * d, generator=g) - 1).float(), torch.randn(H, d, generator=g).float()
+    data, want = [], []
+    for n in totals:
+        r, k, v = (torch.randn(n, H * d, generator=g).to(dtype) for _ in range(3))
+        zw = torch.randn(n, H * d, generator=g).float()
+        zw[:, ::4] = -40.0                                            # decay 1: the channel keeps everything
+        zw[:, 1::4] = 5.0                                             # decay 0
+        decay = torch.exp(-torch.exp(zw.double() + w0.double())).view(n, H, d)
+        want.append(plain.wkv_rule(*(x.double().view(n, H, d) for x in (r, k, v)), decay, u.double()))
+        data.append((r, k, v, zw))
+    state = torch.full((6, H, d * d), 7.0, dtype=torch.float32, device="cuda")
+    slots = [4, 0, 2]
+    state[slots] = 0.0
+    done = [0, 0, 0]
+    for new in PORTIONS:
+        rkv = torch.stack([torch.cat([data[r][i][done[r]:done[r] + n] for r, n in enumerate(new)] + [torch.ones(2, H * d).to(dtype)]) for i in range(3)]).cuda()
+        zw = torch.cat([data[r][3][done[r]:done[r] + n] for r, n in enumerate(new)] + [torch.zeros(2, H * d)]).cuda()
+        qsl = np.cumsum([0] + list(new) + [2]).tolist()
+        out = torch.empty(zw.shape[0], H * d, dtype=torch.float32, device="cuda")
+        kernels.wkv_scan(rkv[0], rkv[1], rkv[2], zw, w0.cuda(), u.cuda(), state, _ints(qsl), _ints(slots + [-1]), out, H, d, d)
+        for r, n in enumerate(new):
+            if n:
+                _close(out[qsl[r]:qsl[r + 1]].view(n, H, d), want[r][0][done[r]:done[r] + n], torch.float32, f"request {r} tokens {done[r]}..")
+            done[r] += n
+    for r in range(3):
+        _close(state[slots[r]].view(H, d, d), want[r][1], torch.float32, f"state of request {r}")
+    assert float((state[[1, 3, 5]] - 7.0).abs().max()) == 0.0, "a slot nobody owns changed"
+
+
+@pytest.mark.parametrize("dtype", BOTH)
+@pytest.mark.parametrize("W,S", [(72, 5), (35, 1), (4096, 5)])
+def test_token_shift(dtype, W, S):
+    from cuinfer_b200 import kernels
+
+    g = torch.Generator().manual_seed(W)
+    totals = [sum(p[r] for p in PORTIONS) for r in range(3)]
+    mu = torch.rand(S, W, generator=g).float()
+    full = [torch.randn(n, W, generator=g).to(dtype) for n in totals]
+    state = torch.full((6, W), 7.0, dtype=torch.float32, device="cuda")
+    slots = [4, 0, 2]
+    state[slots] = 0.0
+    done = [0, 0, 0]
+    for new in PORTIONS:
+        x = torch.cat([full[r][done[r]:done[r] + n] for r, n in enumerate(new)] + [torch.ones(2, W).to(dtype)]).cuda()
+        treq = [r for r, n in enumerate(list(new) + [2]) for _ in range(n)]
+        qsl = np.cumsum([0] + list(new) + [2]).tolist()
+        out = torch.empty(S, x.shape[0], W, dtype=dtype, device="cuda")
+        kernels.token_shift(x, mu.cuda(), state, _ints(qsl), _ints(treq), _ints(slots + [-1]), out)
+        for r, n in enumerate(new):
+            for i in range(n):
+                h = full[r][done[r] + i].double()
+                before = full[r][done[r] + i - 1].double() if done[r] + i else torch.zeros(W, dtype=torch.float64)
+                _close(out[:, qsl[r] + i], h + (before - h) * mu.double(), dtype, f"token {done[r] + i} of request {r}", tol=1e-6 if dtype == torch.float32 else 8e-3)
+            done[r] += n
+    for r in range(3):
+        assert torch.equal(state[slots[r]].cpu(), full[r][-1].float())
+    assert float((state[[1, 3, 5]] - 7.0).abs().max()) == 0.0, "a slot nobody owns changed"
+
+
+# ---- other sizes, drawn at random ------------------------------------------------------------------------------------------
+def _random_config(seed):
+    """A small configuration whose every size, count, constant and order of layers is drawn: odd and even, ones, absent
+    parts; from the sixth on every size is odd or no multiple of eight."""
+    import random
+
+    rnd = random.Random(seed)
+    odd = seed >= 5
+    width, groups = rnd.choice([(45, 3), (57, 1), (99, 3), (66, 2)] if odd else [(40, 1), (64, 2), (104, 4), (96, 3)])
+    layers, sources = [], []
+    for i in range(rnd.randint(3, 6)):
+        mlp = rnd.choice([None, _dense(rnd.choice([9, 21] if odd else [16, 40]))] + 2 * [_moe(
+            *rnd.choice([(4, 2), (6, 3), (3, 1), (1, 1), (2, 3)]), rnd.choice([7, 15] if odd else [8, 16]), rnd.choice([1, 2]))])
+        kind = rnd.choice(["attention", "attention", "parallel", "wkv"])
+        if kind == "attention":
+            source = rnd.choice(sources) if sources and rnd.random() < 0.5 else None
+            if source is not None:
+                m = dict(layers[source]["mixer"], kv_from=source, scale=rnd.choice([0.1, 0.3]), conv=rnd.choice([1, 2, 4]))
+                layers.append({"type": "attention", "mixer": m, "mlp": mlp})
+                continue
+            kv, d = rnd.randint(1, 3), rnd.choice([6, 10, 22] if odd else [8, 16, 32])
+            dims = rnd.choice([0, d, d // 4 * 2])
+            layers.append(_attention(kv * rnd.randint(1, 3), kv, d, rnd.choice([1, 5, 11] if odd else [8, 16]), rnd.choice([0.15, 0.3]), rnd.choice([1, 2, 3, 5]),
+                                     (rnd.choice([50.0, 1e5]), dims) if dims else None, mlp=mlp))
+            sources.append(i)
+        elif kind == "parallel":
+            a, b = rnd.randint(1, 2), rnd.randint(1, 2)
+            layers.append(_pair((a * rnd.randint(1, 3), a, rnd.choice([5, 9] if odd else [8, 16]), rnd.choice([3, 7] if odd else [8, 24]), rnd.choice([0.2, 0.4])),
+                                (b * rnd.randint(1, 3), b, rnd.choice([3, 13, 33] if odd else [8, 40]), rnd.choice([1, 5] if odd else [8, 16]), rnd.randint(1, 4)),
+                                rnd.choice([None, (0.3, 1), (0.1, 5), (-0.1, 16)]), mlp=mlp))
+        else:
+            layers.append(_wkv(rnd.randint(1, 4), rnd.choice([5, 11, 35] if odd else [8, 24, 40]), mlp=mlp))
+    return _config(rnd.choice([33, 64, 131]), width, layers, groups=groups, eps=rnd.choice([1e-6, 1e-5, 1e-3]), mult=rnd.choice([0.25, 0.6, 1.0]),
+                   logits=rnd.choice([0.125, 1.0, 3.0]))
+
+
+@pytest.mark.parametrize("seed", range(12))
+def test_configurations_drawn_at_random(seed, tmp_path):
+    cfg = _random_config(seed)
+    tensors = plain.random_model(cfg, 100 + seed)
+    t64 = {k: v.double() for k, v in tensors.items()}
+    requests = _requests(cfg, [1, 23, 61, 9], seed=30 + seed)
+    steps = traces.mixed(requests, max_live=3, sizes=(5, 2, 11, 3))
+    for dtype in ("float32", "bfloat16"):
+        folder = _write(str(tmp_path / dtype), cfg, tensors, dtype)
+        out = str(tmp_path / f"out_{dtype}")
+        traces.replay_in_process(folder, dtype, steps, out, traces.live_token_peak(steps), 16, max_live=4)
+        got = traces.collect(steps, out, cfg["vocab"])
+        whole_steps = traces.whole(requests)
+        whole_out = str(tmp_path / f"whole_{dtype}")
+        traces.replay_in_process(folder, dtype, whole_steps, whole_out, traces.live_token_peak(whole_steps), 16)
+        whole = traces.collect(whole_steps, whole_out, cfg["vocab"])
+        errors = []
+        for rid, toks in requests.items():
+            ref, margin = _plain_rows(cfg, t64, toks)
+            for pos, row in sorted(got[rid].items()):
+                assert np.isfinite(row).all()
+                if dtype == "float32":
+                    cut = _row_error(row, whole[rid][pos].astype(np.float64))
+                    assert cut <= CUT_TOLERANCE[dtype], f"configuration {seed}: request {rid} position {pos} depends on the cut ({cut:.3e}): {json.dumps(cfg)}"
+                if margin > MARGIN or dtype == "float32":
+                    errors.append((_row_error(row, ref[pos]), rid, pos))
+        worst = max(errors)
+        if dtype == "float32":
+            assert worst[0] <= TOLERANCE[dtype], f"configuration {seed}: request {worst[1]} position {worst[2]} (error {worst[0]:.3e}): {json.dumps(cfg)}"
+        else:
+            # very narrow layers now and then give a token a sub-layer output that nearly cancels, which magnifies the
+            # rounding of bfloat16; the bfloat16 run is held by its median row, which a wrong shape or kernel would move
+            median = sorted(e for e, _, _ in errors)[len(errors) // 2]
+            assert median <= 0.05, f"configuration {seed} in bfloat16: median row error {median:.3e}: {json.dumps(cfg)}"
