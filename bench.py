@@ -451,7 +451,7 @@ def main() -> int:
                              "design and size; see cuinfer_b200/bench_designs.py)")
     parser.add_argument("--design-sizes", default="small,large", help="with --designs: which of its sizes to run")
     parser.add_argument("--design-names", default="bilolorn,qwen3",
-                        help="with --designs: which designs to run (bilolorn, kusolorn, kusolorn_attention, desilorn, zinunex, qwen3)")
+                        help="with --designs: which designs to run (bilolorn, kusolorn, kusolorn_attention, desilorn, zinunex, nugolorn, qwen3)")
     args = parser.parse_args()
     if args.impl == "reference":
         return reference_arm(args)

@@ -1,4 +1,4 @@
-"""Bilolorn, Kusolorn, Desilorn and Zinunex beside the Qwen3 dense decoder at equal layer sizes: prefill and decode throughput
+"""Bilolorn, Kusolorn, Desilorn, Zinunex and Nugolorn beside the Qwen3 dense decoder at equal layer sizes: prefill and decode throughput
 through the model runner, and the time of every kernel of a step with the share of its roofline that it reaches.
 
 ``bench.py --designs`` runs this (``--design-names kusolorn,qwen3`` chooses the designs; ``kusolorn_attention`` is
@@ -118,6 +118,25 @@ def zinunex_config(s: dict) -> dict:
             "token_side": {"dim": s["side_dim"]}, "layers": layers}
 
 
+def nugolorn_config(s: dict) -> dict:
+    """Four layers: attention with sigmoid weights behind convolutions (the Qwen3 arm's head counts and head size) with a
+    dense feed-forward, time mixing (heads of Kusolorn's delta head size), the pair of log-biased attention and the delta
+    rule with a decay per channel (Kusolorn's delta head counts and sizes) and a second attention layer that reads the first
+    one's keys and values, these three with experts of Kusolorn's sizes of which an eighth more give back their input."""
+    heads = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["head_dim"], "vdim": s["head_dim"]}
+    attention = dict(heads, scale=s["head_dim"] ** -0.5, conv=4, rot={"base": 1000000.0, "dims": s["head_dim"]})
+    pair = {"left": dict(heads, scale=s["head_dim"] ** -0.5, q_temp={"coef": 0.1, "every": 256}),
+            "right": {"heads": s["delta_heads"], "kv_heads": s["delta_kv_heads"], "dim": s["delta_dim"], "vdim": s["delta_vdim"], "conv": 4}}
+    mixing = {"heads": s["delta_heads"], "dim": s["delta_dim"]}
+    dense = {"kind": "dense", "ff": s["ff"]}
+    moe = {"kind": "moe", "router": {"experts": s["experts"], "top": s["top"], "identity": s["experts"] // 8}, "expert": {"ff": s["expert_ff"]}}
+    kinds = [("attention", attention, dense), ("wkv", mixing, moe), ("parallel", pair, moe), ("attention", attention, moe)]
+    layers = [{"type": t, "mixer": dict(m, kv_from=i // 4 * 4) if i % 4 == 3 else m, "mlp": f}
+              for i, (t, m, f) in enumerate((kinds * ((s["layers"] + 3) // 4))[:s["layers"]])]
+    return {"architecture": "Nugolorn", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6, "groups": 2},
+            "residual_mult": 0.5, "logit_scale": 0.5, "layers": layers}
+
+
 def qwen3_config(s: dict) -> dict:
     return dict(architectures=["Qwen3ForCausalLM"], num_hidden_layers=s["layers"], hidden_size=s["width"],
                 num_attention_heads=s["heads"], num_key_value_heads=s["kv_heads"], head_dim=s["head_dim"],
@@ -172,7 +191,7 @@ class KernelTimes:
             fn(*args, **kw)
             a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
             rep_args = args
-            if name in ("sandwich_layernorm", "add_rmsnorm", "rms_stream"):           # they add into their first argument
+            if name in ("sandwich_layernorm", "add_rmsnorm", "rms_stream", "group_rms"):           # they add into their first argument
                 rep_args = (args[0].clone(),) + tuple(args[1:])
             # the repeats are recorded into a CUDA graph and the graph is timed: the device's time, not Python's
             torch.cuda.synchronize()
@@ -236,10 +255,15 @@ class KernelTimes:
                 windowed(q, H, d, dv, window, keep, kw.get("chunked", False)),
             "mlstm_scan": lambda q, k, v, gates, ib, fb, cap, qs, state, qsl, slots, out, H, d, dv, **kw: scan(out.shape[0], H, d, dv, 4, state),
             "delta_scan": lambda qkv, gates, al, db, state, qsl, slots, out, G, H, d, dv: scan(out.shape[0], H, d, dv, 6, state),
-            "delta_prep": lambda x, taps, cs, qsl, tr, slots, G, H, d, dv, ue, qs, out: (0.0, _nbytes(out) + out.numel() * x.element_size()),
+            "delta_prep": lambda x, taps, cs, qsl, tr, slots, G, H, d, dv, ue, qs, out, **k: (0.0, _nbytes(out) + out.numel() * x.element_size()),
             "sandwich_layernorm": rowwise, "add_rmsnorm": rowwise, "relu_squared": rowwise, "sigmoid_gate": rowwise,
             "silu_mul": rowwise, "embedding_gather": lambda ids, table, out, *a, **k: (0.0, 2 * _nbytes(out)),
-            "gather_rows": lambda res, delta, idx, out: (0.0, 2 * _nbytes(out)),
+            "gather_rows": lambda res, delta, idx, out, **k: (0.0, 2 * _nbytes(out)),
+            "group_rms": lambda res, d1, d2, scale, norm, groups, out: (0.0, _nbytes(res) * (2 if d1 is not None else 1) + _nbytes(d1, d2, out)),
+            "pair_rms_mean": rowwise, "tanh_rows": rowwise,
+            "token_shift": lambda x, mu, state, qsl, tr, slots, out: (0.0, _nbytes(x, out, mu)),
+            "channel_delta_scan": lambda qkv, beta, decay, al, db, state, qsl, slots, out, G, H, d, dv, **k: scan(out.shape[0], H, d, dv, 7, state),
+            "wkv_scan": lambda r, k, v, decay, w0, u, state, qsl, slots, out, H, d, dv, **kw: scan(out.shape[0], H, d, dv, 5, state),
             "latent_prep": lambda proj, q_off, rq, kv_off, rk, dr, *a, **k: (0.0, proj.shape[0] * (2 * rq + 2 * (rk + dr)) * 2),
             "qk_norm_rope_kv_write": lambda qkv, *a, **k: (0.0, 2 * _nbytes(qkv)),
             "latent_attention_mma": lambda q_abs, q, out, cache, bt, qsl, sl, ql, freq, rd, sinks, H, dn, rk, dr, *a, **k:
@@ -292,7 +316,7 @@ def measure(design: str, size: str, prefill_tokens: int, batch: int, context: in
 
     s = SIZES[size]
     config = {"bilolorn": bilolorn_config, "kusolorn": kusolorn_config, "kusolorn_attention": kusolorn_attention_config,
-              "desilorn": desilorn_config, "zinunex": zinunex_config, "qwen3": qwen3_config}[design](s)
+              "desilorn": desilorn_config, "zinunex": zinunex_config, "nugolorn": nugolorn_config, "qwen3": qwen3_config}[design](s)
     pages = (batch * (context + steps + 64) + prefill_tokens) // 16 + 64
     runner = make_runner(config, pages, max_seqs=max(batch, 8), graphs=True)
     gen = torch.Generator().manual_seed(5)

@@ -85,8 +85,8 @@ def _declare(lib: ctypes.CDLL) -> None:
         "cib_window_attention_prep": [_P, _I, _I, _P, _I, _P, _P, _P, _I, _F, _I, _I, _I, _I, _P, _I, _P, _I, _P, ctypes.c_longlong, _I, _I,
                                       _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _F, _I, _P, _I, _P, _P, _P, _P, _I, _I, _P],
         "cib_conv_state_update": [_P, _I, _I, _I, _P, _P, _P, _I, _I, _I, _P, _P],
-        "cib_channel_delta_scan": [_P, _I, _I, _P, _I, _P, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _P, _I, _I, _I, _P],
-        "cib_wkv_scan": [_P, _P, _P, _I, _I, _P, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _P, _I, _I, _I, _P],
+        "cib_channel_delta_scan": [_P, _I, _I, _P, _I, _P, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _P, _P, _P, _I, _I, _I, _P],
+        "cib_wkv_scan": [_P, _P, _P, _I, _I, _P, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _P, _P, _P, _I, _I, _I, _P],
         "cib_token_shift": [_P, _I, _I, _P, _I, _P, _P, _P, _P, _I, _P, _I, _I, _P],
         "cib_group_rms": [_P, _P, _P, _I, _F, _P, _I, _F, _I, _P, _I, _I, _I, _P],
         "cib_pair_rms_mean": [_P, _P, _I, _P, _P, _I, _F, _P, _I, _I, _P],
@@ -1412,10 +1412,11 @@ def head_rms_gate(o: torch.Tensor, gate: torch.Tensor, gain: torch.Tensor, eps: 
 
 def channel_delta_scan(qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
                        state: torch.Tensor, query_start_loc: torch.Tensor, state_slots: torch.Tensor, out: torch.Tensor,
-                       num_kv_heads: int, num_heads: int, dim: int, vdim: int) -> None:
+                       num_kv_heads: int, num_heads: int, dim: int, vdim: int, one_token_each: bool = False) -> None:
     """The gated delta rule with a decay per head and key channel.  ``qkv`` float32 [T, C] from ``delta_prep``; ``beta``
     float32 [T, >= H] and ``decay`` float32 [T, >= H * dim] pre-activations (rows of any stride; the kernel takes
-    ``sigmoid(beta)`` and ``exp(-exp(a_log) * softplus(decay + dt_bias))``); ``state`` float32 [slots, H, dim * vdim]."""
+    ``sigmoid(beta)`` and ``exp(-exp(a_log) * softplus(decay + dt_bias))``); ``state`` float32 [slots, H, dim * vdim].  Two launches (the gates of all
+    tokens, then the walk), or one when every request brings one token (``one_token_each``)."""
     T = qkv.shape[0]
     if state.shape[1:] != (num_heads, dim * vdim) or out.shape != (T, num_heads * vdim) or qkv.shape[1] != 2 * num_kv_heads * dim + num_heads * vdim:
         raise KernelError("channel_delta_scan: state, rows or out do not fit")
@@ -1423,22 +1424,28 @@ def channel_delta_scan(qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tenso
         raise KernelError("channel_delta_scan: beta or decay do not fit")
     if a_log.dtype != dt_bias.dtype or a_log.numel() != num_heads or dt_bias.numel() != num_heads * dim:
         raise KernelError("channel_delta_scan: a_log has a number per head, dt_bias one per head and channel, in one dtype")
+    gates = None if one_token_each else torch.empty(T * num_heads * dim, dtype=torch.float32, device=qkv.device)
+    pairs = None if one_token_each else torch.empty(T * num_heads * 2, dtype=torch.float32, device=qkv.device)
     rc = library().cib_channel_delta_scan(
         _cuda(qkv, "qkv", torch.float32), qkv.stride(0), num_kv_heads, _cuda(beta, "beta", torch.float32, contiguous=False), beta.stride(0),
         _cuda(decay, "decay", torch.float32, contiguous=False), decay.stride(0), _cuda(a_log, "a_log"), _cuda(dt_bias, "dt_bias"),
         _code(a_log, "a_log"), _cuda(state, "state", torch.float32), _cuda(query_start_loc, "query_start_loc", torch.int32),
-        _cuda(state_slots, "state_slots", torch.int32), state.shape[0], state_slots.numel(), T, _cuda(out, "out", torch.float32),
+        _cuda(state_slots, "state_slots", torch.int32), state.shape[0], state_slots.numel(), T,
+        None if gates is None else gates.data_ptr(), None if pairs is None else pairs.data_ptr(), _cuda(out, "out", torch.float32),
         num_heads, dim, vdim, _stream())
     _check(rc, "channel_delta_scan")
     _count()
+    if not one_token_each:
+        _count()
 
 
 def wkv_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, w0: torch.Tensor, bonus: torch.Tensor,
              state: torch.Tensor, query_start_loc: torch.Tensor, state_slots: torch.Tensor, out: torch.Tensor, num_heads: int,
-             dim: int, vdim: int) -> None:
+             dim: int, vdim: int, one_token_each: bool = False) -> None:
     """RWKV-style time mixing over every request's rows.  ``r``, ``k`` [T, H * dim] and ``v`` [T, H * vdim] with one dtype and
     row stride; ``decay`` float32 [T, >= H * dim] (the kernel takes ``exp(-exp(decay + w0))``); ``bonus`` [H * dim], the
-    weight of the current token's own write in its read-out; ``state`` float32 [slots, H, dim * vdim]; ``out`` float32."""
+    weight of the current token's own write in its read-out; ``state`` float32 [slots, H, dim * vdim]; ``out`` float32.  Two launches (what does not depend on
+    the state, then the walk), or one when every request brings one token (``one_token_each``)."""
     T = out.shape[0]
     if not (r.stride(0) == k.stride(0) == v.stride(0)) or not (r.dtype == k.dtype == v.dtype) or r.stride(1) != 1:
         raise KernelError("wkv_scan: r, k and v must have one dtype and row stride")
@@ -1447,14 +1454,19 @@ def wkv_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Ten
         raise KernelError("wkv_scan: state, rows or out do not fit")
     if decay.shape[0] != T or decay.shape[1] < num_heads * dim or decay.stride(1) != 1 or w0.dtype != bonus.dtype or w0.numel() != num_heads * dim or bonus.numel() != w0.numel():
         raise KernelError("wkv_scan: decay, w0 or bonus do not fit")
+    rows = None if one_token_each else torch.empty(T * num_heads * (3 * dim + vdim), dtype=torch.float32, device=r.device)
+    pairs = None if one_token_each else torch.empty(T * num_heads * 2, dtype=torch.float32, device=r.device)
     rc = library().cib_wkv_scan(
         _cuda(r, "r", contiguous=False), _cuda(k, "k", contiguous=False), _cuda(v, "v", contiguous=False), _code(r, "r"), r.stride(0),
         _cuda(decay, "decay", torch.float32, contiguous=False), decay.stride(0), _cuda(w0, "w0"), _cuda(bonus, "bonus"), _code(w0, "w0"),
         _cuda(state, "state", torch.float32), _cuda(query_start_loc, "query_start_loc", torch.int32),
-        _cuda(state_slots, "state_slots", torch.int32), state.shape[0], state_slots.numel(), T, _cuda(out, "out", torch.float32),
+        _cuda(state_slots, "state_slots", torch.int32), state.shape[0], state_slots.numel(), T,
+        None if rows is None else rows.data_ptr(), None if pairs is None else pairs.data_ptr(), _cuda(out, "out", torch.float32),
         num_heads, dim, vdim, _stream())
     _check(rc, "wkv_scan")
     _count()
+    if not one_token_each:
+        _count()
 
 
 def token_shift(x: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, query_start_loc: torch.Tensor, token_request: torch.Tensor,

@@ -102,7 +102,6 @@ def bf16_matmul_nt(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> 
             torch.mm(x, weight.t(), out=out)
             return
         if out.dtype == torch.float32:
-            tmp = torch.mm(x, weight.t(), out_dtype=torch.float32)
-            out.copy_(tmp)
+            torch.mm(x, weight.t(), out_dtype=torch.float32, out=out)
             return
     kernels.gemm_generic(x, weight, out)

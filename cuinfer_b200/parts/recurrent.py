@@ -254,7 +254,7 @@ class ChannelDelta(Mixer):
     def workspace_bytes(self, tokens: int) -> int:
         width = 2 if self.dtype == torch.bfloat16 else 4
         return (sum(lin.workspace_bytes(tokens) for lin in (self.main, self.gate, self.o))
-                + tokens * (self.num_heads * (1 + 2 * self.dim) + self.channels) * 4 + tokens * self.num_heads * self.vdim * (4 + width))
+                + tokens * (self.num_heads * (3 + 3 * self.dim) + self.channels) * 4 + tokens * self.num_heads * self.vdim * (4 + width))
 
     def forward(self, x: torch.Tensor, ctx: StepContext, run: int) -> torch.Tensor:
         H, G, d, dv = self.num_heads, self.num_kv_heads, self.dim, self.vdim
@@ -269,7 +269,7 @@ class ChannelDelta(Mixer):
                            DELTA_UNIT_EPS, d ** -0.5, qkv, one_token_each=ctx.decode_only)
         o = torch.empty((rows.shape[0], H * dv), dtype=torch.float32, device=rows.device)
         kernels.channel_delta_scan(qkv, beta, decay, self.a_log, self.dt_bias, state["memory"], ctx.query_start_loc, ctx.state_slots,
-                                   o, G, H, d, dv)
+                                   o, G, H, d, dv, one_token_each=ctx.decode_only)
         out = torch.empty((rows.shape[0], H * dv), dtype=rows.dtype, device=rows.device)
         kernels.head_rms_gate(o, gate[:, :H * dv], self.gain, self.eps, False, out, H, dv)
         return self.o.forward(out)
@@ -331,7 +331,7 @@ class TimeMixing(Mixer):
     def workspace_bytes(self, tokens: int) -> int:
         width = 2 if self.dtype == torch.bfloat16 else 4
         hd = self.num_heads * self.dim
-        return tokens * (5 * self.hidden_size * width + 4 * hd * width + hd * (8 + width)) + 3 * self.w1.workspace_bytes(tokens) + self.o.workspace_bytes(tokens)
+        return tokens * (5 * self.hidden_size * width + 4 * hd * width + hd * (24 + width) + self.num_heads * 8) + 3 * self.w1.workspace_bytes(tokens) + self.o.workspace_bytes(tokens)
 
     def forward(self, x: torch.Tensor, ctx: StepContext, run: int) -> torch.Tensor:
         H, d, T = self.num_heads, self.dim, x.shape[0]
@@ -346,7 +346,7 @@ class TimeMixing(Mixer):
         decay = self.w2.forward(dense_operand(inner), out_dtype=torch.float32)
         o = torch.empty((T, H * d), dtype=torch.float32, device=x.device)
         kernels.wkv_scan(rkvg[0], rkvg[1], rkvg[2], decay, self.w0, self.bonus, state["memory"], ctx.query_start_loc, ctx.state_slots,
-                         o, H, d, d)
+                         o, H, d, d, one_token_each=ctx.decode_only)
         out = torch.empty((T, H * d), dtype=x.dtype, device=x.device)
         kernels.head_rms_gate(o, rkvg[3], self.gain, self.eps, True, out, H, d)
         return self.o.forward(out)

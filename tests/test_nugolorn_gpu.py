@@ -640,7 +640,7 @@ def test_sigmoid_weights_are_not_normalised():
 
 
 # ---- the recurrences --------------------------------------------------------------------------------------------------------
-PORTIONS = ([2, 1, 3], [1, 1, 1], [17, 0, 2], [1, 33, 16], [4, 2, 1])
+PORTIONS = ([2, 1, 3], [1, 1, 1], [17, 0, 2], [1, 33, 16], [1, 1, 1], [4, 2, 1])
 
 
 @pytest.mark.parametrize("H,G,d,dv", [(4, 2, 12, 6), (2, 1, 32, 40), (3, 3, 50, 130), (2, 2, 128, 64), (2, 1, 200, 33), (1, 1, 1, 1)])
@@ -668,12 +668,14 @@ def test_delta_rule_with_a_decay_per_channel(H, G, d, dv):
     done = [0, 0, 0]
     for new in PORTIONS:
         parts = [tuple(x[done[r]:done[r] + n] for x in data[r]) for r, n in enumerate(new)]
-        pad = (torch.ones(2, C), torch.zeros(2, H), torch.zeros(2, H * d))
+        one = all(n == 1 for n in new)                                # the one-launch form, whose padding request brings one token
+        extra = 1 if one else 2
+        pad = (torch.ones(extra, C), torch.zeros(extra, H), torch.zeros(extra, H * d))
         qkv, zb, za = (torch.cat([p[i] for p in parts] + [pad[i]]) for i in range(3))
         zb, za = torch.nn.functional.pad(zb, (0, 3)), torch.nn.functional.pad(za, (0, 2))         # rows wider than what is read
-        qsl = np.cumsum([0] + list(new) + [2]).tolist()
+        qsl = np.cumsum([0] + list(new) + [extra]).tolist()
         out = torch.empty(qkv.shape[0], H * dv, dtype=torch.float32, device="cuda")
-        kernels.channel_delta_scan(qkv.cuda(), zb.cuda(), za.cuda(), a_log.cuda(), dt_bias.cuda(), state, _ints(qsl), _ints(slots + [-1]), out, G, H, d, dv)
+        kernels.channel_delta_scan(qkv.cuda(), zb.cuda(), za.cuda(), a_log.cuda(), dt_bias.cuda(), state, _ints(qsl), _ints(slots + [-1]), out, G, H, d, dv, one_token_each=one)
         for r, n in enumerate(new):
             if n:
                 _close(out[qsl[r]:qsl[r + 1]].view(n, H, dv), want[r][0][done[r]:done[r] + n], torch.float32, f"request {r} tokens {done[r]}..")
@@ -705,11 +707,13 @@ def test_time_mixing_scan(dtype, H, d):
     state[slots] = 0.0
     done = [0, 0, 0]
     for new in PORTIONS:
-        rkv = torch.stack([torch.cat([data[r][i][done[r]:done[r] + n] for r, n in enumerate(new)] + [torch.ones(2, H * d).to(dtype)]) for i in range(3)]).cuda()
-        zw = torch.cat([data[r][3][done[r]:done[r] + n] for r, n in enumerate(new)] + [torch.zeros(2, H * d)]).cuda()
-        qsl = np.cumsum([0] + list(new) + [2]).tolist()
+        one = all(n == 1 for n in new)
+        extra = 1 if one else 2
+        rkv = torch.stack([torch.cat([data[r][i][done[r]:done[r] + n] for r, n in enumerate(new)] + [torch.ones(extra, H * d).to(dtype)]) for i in range(3)]).cuda()
+        zw = torch.cat([data[r][3][done[r]:done[r] + n] for r, n in enumerate(new)] + [torch.zeros(extra, H * d)]).cuda()
+        qsl = np.cumsum([0] + list(new) + [extra]).tolist()
         out = torch.empty(zw.shape[0], H * d, dtype=torch.float32, device="cuda")
-        kernels.wkv_scan(rkv[0], rkv[1], rkv[2], zw, w0.cuda(), u.cuda(), state, _ints(qsl), _ints(slots + [-1]), out, H, d, d)
+        kernels.wkv_scan(rkv[0], rkv[1], rkv[2], zw, w0.cuda(), u.cuda(), state, _ints(qsl), _ints(slots + [-1]), out, H, d, d, one_token_each=one)
         for r, n in enumerate(new):
             if n:
                 _close(out[qsl[r]:qsl[r + 1]].view(n, H, d), want[r][0][done[r]:done[r] + n], torch.float32, f"request {r} tokens {done[r]}..")
