@@ -21,8 +21,8 @@
 //   query at position i sees key j when j <= i and (window == 0 or i - j < window or j < keep_first); with `chunked`
 //   the window is a chunk instead: j >= floor(i / window) * window;
 //   softmax over the visible keys, whose denominator also holds exp(sink[head]) when sinks are given (a sink has no key
-//   and no value and is neither scaled nor biased); weighted sum of the values; with `sigmoid_bias` there is no softmax:
-//   the weight of a visible key is sigmoid(score + sigmoid_bias[head]), not normalised;
+//   and no value and is neither scaled nor biased); weighted sum of the values; with `sigmoid_bias` nothing is
+//   normalised: a key counts with sigmoid(score + sigmoid_bias[head]);
 //   with `gate` the result is multiplied by sigmoid of the token's gate logit, one per value or one per head.
 // Everything after the loads is 32-bit; exponentials, tangents, sines, logarithms are the exact ones.
 //

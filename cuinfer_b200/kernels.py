@@ -1250,8 +1250,8 @@ def window_attention_generic(q: torch.Tensor, out: torch.Tensor, cache: torch.Te
     """Attention of the query rows ``q[:, :H * dim]`` over the paged cache of [key | value] rows; ``out`` [T, H * vdim].
     ``softcap`` 0: no cap; ``window`` 0: every earlier key; ``chunked``: the window is a chunk, key j is seen when
     ``j // window == i // window``; ``slopes`` (float32 [H]): ``score -= slope * (i - j)``; ``sinks`` (float32 [H]): a
-    score per head that joins the softmax's denominator and nothing else.  ``sigmoid_bias`` (float32 [H]): no softmax, the
-    weight of a visible key is ``sigmoid(score + sigmoid_bias)``; ``log_bias = (r1, r2)`` (float32 [H] each):
+    score per head that joins the softmax's denominator and nothing else.  ``sigmoid_bias`` (float32 [H]): nothing is
+    normalised, a key counts with ``sigmoid(score + sigmoid_bias)``; ``log_bias = (r1, r2)`` (float32 [H] each):
     ``score -= r1 * ln(1 + r2 * (i - j))``; ``gate`` (rows' dtype, [T, H * vdim] or [T, H], any row stride): the result is
     multiplied by its sigmoid, per value or per head."""
     T = q.shape[0]

@@ -30,8 +30,8 @@ multiplies the rows of S, and the output gate is ``sigmoid(G2 (G1 h))``.  The in
 the checkpoint's.  Spec: ``PartSpec("channel_delta", num_heads, num_kv_heads, dim, vdim, taps, eps, rank, names={...})``
 (``rank``: what the random-weights mode draws).
 
-``wkv`` — RWKV-style time mixing.  With h' the previous token's h (zeros for a sequence's first), each of r, k, v, g, w reads
-a mix ``h + (h' - h) * mu_s`` of its own; ``r = Wr mix_r``, ``k = Wk mix_k``, ``v = Wv mix_v`` (H heads of d),
+``wkv`` — RWKV-style time mixing.  The five inputs of r, k, v, g and w are interpolations ``h + (h' - h) * mu_s`` between the
+row h and the row h' of the token before (zeros before a sequence's first), mix_s below; ``r = Wr mix_r``, ``k = Wk mix_k``, ``v = Wv mix_v`` (H heads of d),
 ``gate = silu(Wg mix_g)``, decay ``w = exp(-exp(W2 tanh(W1 mix_w) + w0))`` per head and channel::
 
     o = (S + diag(u) k v^T)^T r;  S <- diag(w) S + k v^T
@@ -39,7 +39,7 @@ a mix ``h + (h' - h) * mu_s`` of its own; ``r = Wr mix_r``, ``k = Wk mix_k``, ``
 then each head's o divided by its root mean square, times a gain over all heads, times the gate, then ``Wo``.  The previous
 h is state too.  Spec: ``PartSpec("wkv", num_heads, dim, eps, rank, names={...})``.
 
-``side_by_side`` — two mixers that read the same h: half the sum of their outputs, each RMS-normed over the model width.
+``side_by_side`` — two mixers on the same input: ``(rms(left) * left.out + rms(right) * right.out) / 2``, norms of whole rows.
 Spec: ``PartSpec("side_by_side", left=PartSpec(...), right=PartSpec(...), eps, names={"left": "left", "right": "right",
 "out": "out"})``: the mixers' tensors lie under ``left`` and ``right``, the norms' gains are ``left.out`` and ``right.out``.  One of
 the two may keep a paged cache; both may keep state.

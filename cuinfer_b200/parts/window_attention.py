@@ -9,7 +9,7 @@ and key size ``dim``, value size ``vdim``:
 * ``q = Wq h``, ``k = Wk h``, ``v = Wv h``; with ``bias`` each has a bias (the tensor's name plus ``bias_suffix``),
   added in 32 bits; with ``value_from_key`` there is no ``Wv``: a token's value is its key as projected, before norm and
   rotation (``vdim == dim``);
-* ``conv`` K > 0: a causal convolution of K taps over time on each channel of q, k and v (biases included in its input;
+* ``conv`` K > 0: every column of the projected rows is filtered along the sequence with K taps (biases included in its input;
   tensor names plus ``conv_suffix``, [channels, K], the last column the current token's; zeros before a sequence's start);
   the last K - 1 projected values of a request are its state;
 * ``own_kv`` False: the layer has no keys and values of its own (nor their biases and convolutions); it reads those that
@@ -28,8 +28,8 @@ and key size ``dim``, value size ``vdim``:
 * the query at position i sees key j when ``j <= i`` and (no window, or ``i - j < window``, or ``j < keep_first``);
   with ``chunked`` the window is a chunk counted from position 0: ``j // window == i // window``;
 * softmax; ``sink="learned"`` adds ``exp(sink_h)``, a learned number per head, to the denominator and ``sink="zero"``
-  adds one (a sink has no key and no value, is not scaled and gets no bias); with ``weights="sigmoid"`` there is no
-  softmax: a visible key has weight ``sigmoid(score + b_h)`` with a learned number per head, not normalised;
+  adds one (a sink has no key and no value, is not scaled and gets no bias); with ``weights="sigmoid"`` nothing
+  is normalised: a key counts with ``sigmoid(score + b_h)``, b a learned number per head;
 * ``gate``: the heads' outputs are multiplied by ``sigmoid(Wg h)``, one number per value (``"value"``) or per head
   (``"head"``), from the same input h; output projection ``Wo`` on the concatenated heads.
 
