@@ -13,7 +13,8 @@
 //   rotation of the first `rot_dims` values by the angle pos * freq[i] (32-bit angle, full-range sine and cosine, both
 //   multiplied by `rot_gain`), in neighbouring pairs (2i, 2i+1) or in halves (i, i + rot_dims / 2);
 //   q and k divided by their root mean square (eps inside the root) and multiplied by a gain of d values shared by all
-//   heads (null: no gain), after the rotation or, with `norm_first`, before it;
+//   heads (null: no gain), after the rotation or, with `norm_first`, before it; with `norm_rows` one root mean square over
+//   all of a token's query heads (and one over its key heads) with a gain per value of the row;
 //   q multiplied by the query temperature 1 + coef * ln(floor((pos + 1) / every) + 1);
 //   v = (1 - lambda) * v + lambda * v_first for a layer that mixes in an earlier layer's values of the same token;
 //   score = scale * q.k, then cap * tanh(score / cap) if cap > 0, then minus slope[head] * (i - j) (a distance bias) or
@@ -27,7 +28,7 @@
 // Everything after the loads is 32-bit; exponentials, tangents, sines, logarithms are the exact ones.
 //
 // Cache layout of one layer run: [page][kv head][slot in page][d + dv] — a token's key and value side by side.
-#include "common.cuh"
+#include "mma_utils.cuh"
 
 namespace cib {
 
@@ -57,6 +58,7 @@ struct PrepOptions {
     const int* state_slots;
     int num_state_slots;
     int conv_update;          // every request brings one token: the lane that reads a channel's state also moves it on
+    int norm_rows;            // the norm is over all query heads (all key heads) of a token; the gains have a value per column
 };
 
 // The conv of one column of one token's row (see PrepOptions): u_t = x_t + bias; y = sum_j taps[j] u_(t - taps_n + 1 + j).
@@ -84,18 +86,14 @@ __device__ __forceinline__ float conv_column(const T* __restrict__ rows, int str
 // One warp per (token, vector): H query heads, G key heads, G value heads of the packed rows [q | k | v] (with
 // `value_from_key` there are no value vectors: the key's warp stores the value too).  C: pairs of values a lane holds
 // (d <= 64 C).
+// row_factor: with `norm_rows`, one over the root mean square of the token's queries or keys.
 template <typename T, int C>
-__global__ void __launch_bounds__(kPrepWarps * 32)
-window_attention_prep_kernel(T* qkv, int stride, T* q_out, int q_out_stride, const int* __restrict__ positions,
-                             const int* __restrict__ slot_mapping, const float* __restrict__ freq, int rot_dims, float eps,
-                             int H, int G, int d, int dv, const T* __restrict__ v_first, int v_first_stride,
-                             AnyVec lambda, int has_lambda, T* __restrict__ cache, long long num_slots, int page_size,
-                             int num_tokens, PrepOptions opt) {
+__device__ __forceinline__ void
+prep_vector(int t, int vec, float row_factor, T* qkv, int stride, T* q_out, int q_out_stride, const int* __restrict__ positions,
+            const int* __restrict__ slot_mapping, const float* __restrict__ freq, int rot_dims, float eps,
+            int H, int G, int d, int dv, const T* __restrict__ v_first, int v_first_stride,
+            AnyVec lambda, int has_lambda, T* __restrict__ cache, long long num_slots, int page_size, const PrepOptions& opt) {
     const int lane = threadIdx.x & 31;
-    const int vectors = opt.q_only ? H : opt.value_from_key ? H + G : H + 2 * G;
-    const long long w = (long long)blockIdx.x * kPrepWarps + (threadIdx.x >> 5);
-    if (w >= (long long)num_tokens * vectors) return;
-    const int t = (int)(w / vectors), vec = (int)(w % vectors);
     T* row = qkv + (size_t)t * stride;
     const int slot = slot_mapping ? slot_mapping[t] : -1;
     const bool store = cache && slot >= 0 && slot < num_slots;
@@ -135,6 +133,7 @@ window_attention_prep_kernel(T* qkv, int stride, T* q_out, int q_out_stride, con
     T* x = row + off;
     const float* bias = opt.bias ? opt.bias + off : nullptr;
     const float* gain = is_key ? opt.k_gain : opt.q_gain;
+    if (gain && opt.norm_rows) gain += is_key ? (size_t)(vec - H) * d : off;
     const int ipos = positions[t];
     const float pos = (float)ipos;
     const int half = rot_dims / 2;
@@ -163,11 +162,14 @@ window_attention_prep_kernel(T* qkv, int stride, T* q_out, int q_out_stride, con
         }
     }
     auto normalise = [&]() {
-        float ss = 0.f;
+        float factor = row_factor;
+        if (!opt.norm_rows) {
+            float ss = 0.f;
 #pragma unroll
-        for (int c = 0; c < C; ++c) ss += a[c] * a[c] + b[c] * b[c];
-        ss = warp_sum(ss);
-        const float factor = 1.f / sqrtf(ss / (float)d + eps);
+            for (int c = 0; c < C; ++c) ss += a[c] * a[c] + b[c] * b[c];
+            ss = warp_sum(ss);
+            factor = 1.f / sqrtf(ss / (float)d + eps);
+        }
 #pragma unroll
         for (int c = 0; c < C; ++c) {
             const int p = c * 32 + lane, e0 = first_of(p), e1 = second_of(p);
@@ -205,6 +207,109 @@ window_attention_prep_kernel(T* qkv, int stride, T* q_out, int q_out_stride, con
         const int p = c * 32 + lane, e0 = first_of(p), e1 = second_of(p);
         if (e0 < d) dst[e0] = from_f32<T>(a[c]);
         if (e1 < d) dst[e1] = from_f32<T>(b[c]);
+    }
+}
+
+template <typename T, int C>
+__global__ void __launch_bounds__(kPrepWarps * 32)
+window_attention_prep_kernel(T* qkv, int stride, T* q_out, int q_out_stride, const int* __restrict__ positions,
+                             const int* __restrict__ slot_mapping, const float* __restrict__ freq, int rot_dims, float eps,
+                             int H, int G, int d, int dv, const T* __restrict__ v_first, int v_first_stride,
+                             AnyVec lambda, int has_lambda, T* __restrict__ cache, long long num_slots, int page_size,
+                             int num_tokens, PrepOptions opt) {
+    const int vectors = opt.q_only ? H : opt.value_from_key ? H + G : H + 2 * G;
+    const long long w = (long long)blockIdx.x * kPrepWarps + (threadIdx.x >> 5);
+    if (w >= (long long)num_tokens * vectors) return;
+    prep_vector<T, C>((int)(w / vectors), (int)(w % vectors), 1.f, qkv, stride, q_out, q_out_stride, positions, slot_mapping, freq, rot_dims,
+                      eps, H, G, d, dv, v_first, v_first_stride, lambda, has_lambda, cache, num_slots, page_size, opt);
+}
+
+// The norm over whole rows of queries and keys: a block per token sums both rows' squares (biases included), then its warps
+// take the vectors one by one.  PLAIN (bfloat16, sizes in multiples of 8, no bias, rotation or temperature): eight values a
+// lane, the rows staged in registers between the two passes where they fit.
+template <typename T, int C, bool PLAIN>
+__global__ void __launch_bounds__(kPrepWarps * 32)
+window_attention_prep_rows_kernel(T* qkv, int stride, const int* __restrict__ positions, const int* __restrict__ slot_mapping,
+                                  const float* __restrict__ freq, int rot_dims, float eps, int H, int G, int d, int dv,
+                                  T* __restrict__ cache, long long num_slots, int page_size, PrepOptions opt) {
+    __shared__ float scratch[33];
+    const int t = blockIdx.x;
+    T* row = qkv + (size_t)t * stride;
+    const int nq = H * d, nk = opt.q_only ? 0 : G * d;
+    griddep_launch();
+    griddep_wait();
+    if constexpr (PLAIN) {
+        constexpr int CH = 4;                             // rows of up to 8 192 values stay in registers
+        const int total = nq + nk;
+        uint4 held[CH];
+        float sq = 0.f, sk = 0.f;
+        auto add = [&](const uint4& v, int i) {
+            const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&v);
+            float s = 0.f;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const float2 f = __bfloat1622float2(h[e]);
+                s = fmaf(f.x, f.x, fmaf(f.y, f.y, s));
+            }
+            if (i < nq) sq += s; else sk += s;
+        };
+#pragma unroll
+        for (int c = 0; c < CH; ++c) {
+            const int i = (c * kPrepWarps * 32 + threadIdx.x) * 8;
+            if (i < total) held[c] = *reinterpret_cast<const uint4*>(row + i);
+        }
+#pragma unroll
+        for (int c = 0; c < CH; ++c) {
+            const int i = (c * kPrepWarps * 32 + threadIdx.x) * 8;
+            if (i < total) add(held[c], i);
+        }
+        for (int i = (CH * kPrepWarps * 32 + threadIdx.x) * 8; i < total; i += kPrepWarps * 32 * 8) add(*reinterpret_cast<const uint4*>(row + i), i);
+        sq = block_sum(sq, scratch);
+        sk = block_sum(sk, scratch);
+        const float fq = 1.f / sqrtf(sq / (float)nq + eps), fk = nk ? 1.f / sqrtf(sk / (float)nk + eps) : 0.f;
+        const int slot = slot_mapping ? slot_mapping[t] : -1;
+        const bool store = cache && slot >= 0 && slot < num_slots;
+        const int width = d + dv;
+        T* page = store ? cache + ((size_t)(slot / page_size) * G * page_size + slot % page_size) * width : nullptr;
+        auto place = [&](uint4 v, int i) {
+            const bool key = i >= nq;
+            if (key && !store) return;
+            const int at = key ? i - nq : i;
+            const float f = key ? fk : fq;
+            const float* gain = key ? opt.k_gain : opt.q_gain;
+            uint32_t* p = reinterpret_cast<uint32_t*>(&v);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const float2 x = __bfloat1622float2(reinterpret_cast<const __nv_bfloat162*>(&v)[e]);
+                const float2 g = gain ? *reinterpret_cast<const float2*>(gain + at + 2 * e) : make_float2(1.f, 1.f);
+                __nv_bfloat162 y = __floats2bfloat162_rn(x.x * f * g.x, x.y * f * g.y);
+                p[e] = *reinterpret_cast<uint32_t*>(&y);
+            }
+            T* dst = key ? page + (size_t)(at / d) * page_size * width + at % d : row + i;
+            *reinterpret_cast<uint4*>(dst) = v;
+        };
+#pragma unroll
+        for (int c = 0; c < CH; ++c) {
+            const int i = (c * kPrepWarps * 32 + threadIdx.x) * 8;
+            if (i < total) place(held[c], i);
+        }
+        for (int i = (CH * kPrepWarps * 32 + threadIdx.x) * 8; i < total; i += kPrepWarps * 32 * 8) place(*reinterpret_cast<const uint4*>(row + i), i);
+        if (!store || opt.q_only) return;
+        for (int i = threadIdx.x * 8; i < G * dv; i += kPrepWarps * 32 * 8)
+            *reinterpret_cast<uint4*>(page + (size_t)(i / dv) * page_size * width + d + i % dv) = *reinterpret_cast<const uint4*>(row + total + i);
+    } else {
+        float sq = 0.f, sk = 0.f;
+        for (int i = threadIdx.x; i < nq + nk; i += blockDim.x) {
+            const float x = to_f32(row[i]) + (opt.bias ? opt.bias[i] : 0.f);
+            if (i < nq) sq = fmaf(x, x, sq); else sk = fmaf(x, x, sk);
+        }
+        sq = block_sum(sq, scratch);
+        sk = block_sum(sk, scratch);                      // also: every square is in before a query is rewritten
+        const float fq = 1.f / sqrtf(sq / (float)nq + eps), fk = nk ? 1.f / sqrtf(sk / (float)nk + eps) : 0.f;
+        const int vectors = opt.q_only ? H : H + 2 * G;
+        for (int vec = threadIdx.x >> 5; vec < vectors; vec += kPrepWarps)
+            prep_vector<T, C>(t, vec, vec < H ? fq : fk, qkv, stride, nullptr, 0, positions, slot_mapping, freq, rot_dims, eps, H, G, d, dv,
+                              nullptr, 0, AnyVec{nullptr, 0}, 0, cache, num_slots, page_size, opt);
     }
 }
 
@@ -333,7 +438,9 @@ extern "C" int cib_window_attention_prep(void* qkv, int dtype, int stride, void*
                                          int rot_half, int has_temp, float temp_coef, int temp_every, int value_from_key,
                                          float rot_gain, int q_only, const float* taps, int taps_n, float* conv_state,
                                          const int* query_start_loc, const int* token_request, const int* state_slots,
-                                         int num_state_slots, int conv_update, cudaStream_t stream) {
+                                         int num_state_slots, int conv_update, int norm_rows, cudaStream_t stream) {
+    CIB_REQUIRE(!norm_rows || (norm && !taps && !value_from_key && !v_first && !q_out),
+                "window_attention_prep: a norm over whole rows beside a convolution, mixed values or values taken from keys is not built");
     CIB_REQUIRE(H > 0 && G > 0 && H % G == 0 && d > 0 && dv > 0, "window_attention_prep: bad head counts or sizes");
     CIB_REQUIRE(!taps || (taps_n >= 1 && q_out && (taps_n == 1 || conv_state) && query_start_loc && token_request && state_slots),
                 "window_attention_prep: a convolution needs its state, the requests' bounds and a place for the queries");
@@ -349,7 +456,23 @@ extern "C" int cib_window_attention_prep(void* qkv, int dtype, int stride, void*
     const int blocks = (int)((warps + kPrepWarps - 1) / kPrepWarps);
     AnyVec lam{lambda, lambda_dtype == kBF16};
     PrepOptions opt{bias, q_gain, k_gain, norm, norm_first, rot_half, has_temp, temp_coef, temp_every, value_from_key, rot_gain, q_only,
-                    taps, taps_n, conv_state, query_start_loc, token_request, state_slots, num_state_slots, conv_update};
+                    taps, taps_n, conv_state, query_start_loc, token_request, state_slots, num_state_slots, conv_update, norm_rows};
+    if (norm_rows) {
+        const bool pdl = prompt_pdl();
+        auto gain_ok = [](const float* g) { return (uintptr_t)g % 8 == 0; };
+        const bool plain = dtype == kBF16 && d % 8 == 0 && dv % 8 == 0 && stride % 8 == 0 && !bias && !rot_dims && !has_temp &&
+                           (uintptr_t)qkv % 16 == 0 && (uintptr_t)cache % 16 == 0 && gain_ok(q_gain) && gain_ok(k_gain);
+#define CIB_PREP_ROWS(T, C, PLAIN)                                                                                            \
+    launch_pdl(window_attention_prep_rows_kernel<T, C, PLAIN>, dim3(num_tokens), dim3(kPrepWarps * 32), 0, stream, pdl, (T*)qkv, stride,  \
+               positions, slot_mapping, freq, rot_dims, eps, H, G, d, dv, (T*)cache, num_slots, page_size, opt)
+        if (plain) CIB_PREP_ROWS(__nv_bfloat16, 1, true);
+        else if (dtype == kF32) { if (d <= 64) CIB_PREP_ROWS(float, 1, false); else if (d <= 128) CIB_PREP_ROWS(float, 2, false); else CIB_PREP_ROWS(float, 8, false); }
+        else if (dtype == kBF16) { if (d <= 64) CIB_PREP_ROWS(__nv_bfloat16, 1, false); else if (d <= 128) CIB_PREP_ROWS(__nv_bfloat16, 2, false); else CIB_PREP_ROWS(__nv_bfloat16, 8, false); }
+        else CIB_REQUIRE(false, "window_attention_prep: bad dtype %d", dtype);
+#undef CIB_PREP_ROWS
+        CIB_LAUNCH_CHECK("window_attention_prep");
+        return 0;
+    }
 #define CIB_PREP(T, C)                                                                                                        \
     window_attention_prep_kernel<T, C><<<blocks, kPrepWarps * 32, 0, stream>>>(                                               \
         (T*)qkv, stride, (T*)q_out, q_out_stride, positions, slot_mapping, freq, rot_dims, eps, H, G, d, dv, (const T*)v_first, v_first_stride, lam,    \

@@ -217,6 +217,42 @@ __global__ void relu_squared_kernel(const T* __restrict__ x, T* __restrict__ out
     }
 }
 
+// out = x + bias, or max(x + bias, 0)^2 (`squared_relu`), for rows of `cols` values; 32-bit with one rounding; out may be x.
+template <typename T, int V>
+__global__ void bias_rows_kernel(const T* x, const float* __restrict__ bias, T* out, int cols, size_t total, int squared_relu) {
+    griddep_launch();
+    griddep_wait();
+    for (size_t e = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * V; e < total; e += (size_t)gridDim.x * blockDim.x * V) {
+        const int j = (int)(e % cols);
+        float v[V];
+        Vec<T, V>::load(x + e, v);
+#pragma unroll
+        for (int k = 0; k < V; ++k) {
+            v[k] += bias[j + k];
+            if (squared_relu) {
+                v[k] = fmaxf(v[k], 0.f);
+                v[k] *= v[k];
+            }
+        }
+        Vec<T, V>::store(out + e, v);
+    }
+}
+
+// out = scale_a * a + scale_b * b, 32-bit with one rounding.
+template <typename T, int V>
+__global__ void pair_sum_kernel(const T* __restrict__ a, const T* __restrict__ b, float scale_a, float scale_b, T* __restrict__ out, size_t total) {
+    griddep_launch();
+    griddep_wait();
+    for (size_t e = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * V; e < total; e += (size_t)gridDim.x * blockDim.x * V) {
+        float x[V], y[V];
+        Vec<T, V>::load(a + e, x);
+        Vec<T, V>::load(b + e, y);
+#pragma unroll
+        for (int k = 0; k < V; ++k) x[k] = scale_a * x[k] + scale_b * y[k];
+        Vec<T, V>::store(out + e, x);
+    }
+}
+
 // ---- sigmoid gate -------------------------------------------------------------------------------------
 // out[t, j] = x[t, j] * sigmoid(gate[t, j]) with the exact exponential; the rows of x and of gate may lie inside wider
 // rows (their strides are given), out is dense.
@@ -248,6 +284,35 @@ extern "C" int cib_relu_squared(const void* x, void* out, int dtype, long long t
     else if (dtype == kBF16) relu_squared_kernel<__nv_bfloat16><<<flat_blocks(total), 256, 0, stream>>>((const __nv_bfloat16*)x, (__nv_bfloat16*)out, (size_t)total);
     else CIB_REQUIRE(false, "relu_squared: unsupported dtype %d", dtype);
     CIB_LAUNCH_CHECK("relu_squared");
+    return 0;
+}
+
+// x, out [rows][cols] (out may be x); bias float32 [cols].
+extern "C" int cib_bias_rows(const void* x, const float* bias, void* out, int dtype, int rows, int cols, int squared_relu, cudaStream_t stream) {
+    CIB_REQUIRE(rows >= 0 && cols > 0 && bias, "bias_rows: bad arguments");
+    if (rows == 0) return 0;
+    const size_t total = (size_t)rows * cols;
+    const bool v4 = cols % 4 == 0, pdl = prompt_pdl();
+#define CIB_BIAS(T, V) launch_pdl(bias_rows_kernel<T, V>, dim3(flat_blocks(total / V)), dim3(256), 0, stream, pdl, (const T*)x, bias, (T*)out, cols, total, squared_relu)
+    if (dtype == kF32) { if (v4) CIB_BIAS(float, 4); else CIB_BIAS(float, 1); }
+    else if (dtype == kBF16) { if (v4) CIB_BIAS(__nv_bfloat16, 4); else CIB_BIAS(__nv_bfloat16, 1); }
+    else CIB_REQUIRE(false, "bias_rows: bad dtype %d", dtype);
+#undef CIB_BIAS
+    CIB_LAUNCH_CHECK("bias_rows");
+    return 0;
+}
+
+extern "C" int cib_pair_sum(const void* a, const void* b, float scale_a, float scale_b, void* out, int dtype, long long total,
+                            cudaStream_t stream) {
+    CIB_REQUIRE(total >= 0, "pair_sum: bad size");
+    if (total == 0) return 0;
+    const bool v4 = total % 4 == 0, pdl = prompt_pdl();
+#define CIB_PAIR_SUM(T, V) launch_pdl(pair_sum_kernel<T, V>, dim3(flat_blocks((size_t)total / V)), dim3(256), 0, stream, pdl, (const T*)a, (const T*)b, scale_a, scale_b, (T*)out, (size_t)total)
+    if (dtype == kF32) { if (v4) CIB_PAIR_SUM(float, 4); else CIB_PAIR_SUM(float, 1); }
+    else if (dtype == kBF16) { if (v4) CIB_PAIR_SUM(__nv_bfloat16, 4); else CIB_PAIR_SUM(__nv_bfloat16, 1); }
+    else CIB_REQUIRE(false, "pair_sum: bad dtype %d", dtype);
+#undef CIB_PAIR_SUM
+    CIB_LAUNCH_CHECK("pair_sum");
     return 0;
 }
 
@@ -404,6 +469,69 @@ rms_stream_kernel(float* __restrict__ residual, const TD* __restrict__ delta, An
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) out[row + i] = from_f32<TO>(row_s[i] * f2 * gain[i]);
 }
 
+// Rows of a multiple of four values: four a lane and load, the row (CH * 4 values a thread) in registers, every load issued
+// before the first use; the gains come after the reductions.
+template <typename TD, typename TO, int CH>
+__global__ void __launch_bounds__(256)
+rms_stream_vec_kernel(float* __restrict__ residual, const TD* __restrict__ delta, AnyVec post_gain, int has_post, float post_eps,
+                      AnyVec gain, float eps, TO* __restrict__ out, TO* __restrict__ raw, int hidden) {
+    __shared__ float scratch[33];
+    griddep_launch();
+    griddep_wait();
+    const size_t row = (size_t)blockIdx.x * hidden;
+    float x[CH][4], y[CH][4];
+    auto at = [&](int c) { return (c * (int)blockDim.x + (int)threadIdx.x) * 4; };
+#pragma unroll
+    for (int c = 0; c < CH; ++c)
+        if (at(c) < hidden) Vec<float, 4>::load(residual + row + at(c), x[c]);
+    if (delta) {
+#pragma unroll
+        for (int c = 0; c < CH; ++c)
+            if (at(c) < hidden) Vec<TD, 4>::load(delta + row + at(c), y[c]);
+        float factor = 1.f;
+        if (has_post) {
+            float ss = 0.f;
+#pragma unroll
+            for (int c = 0; c < CH; ++c)
+                if (at(c) < hidden) {
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) ss = fmaf(y[c][k], y[c][k], ss);
+                }
+            ss = block_sum(ss, scratch);
+            factor = 1.f / sqrtf(ss / (float)hidden + post_eps);
+        }
+#pragma unroll
+        for (int c = 0; c < CH; ++c)
+            if (at(c) < hidden) {
+#pragma unroll
+                for (int k = 0; k < 4; ++k) x[c][k] += has_post ? y[c][k] * factor * post_gain[at(c) + k] : y[c][k];
+                Vec<float, 4>::store(residual + row + at(c), x[c]);
+            }
+    }
+    if (raw) {
+#pragma unroll
+        for (int c = 0; c < CH; ++c)
+            if (at(c) < hidden) Vec<TO, 4>::store(raw + row + at(c), x[c]);
+    }
+    if (!out) return;
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < CH; ++c)
+        if (at(c) < hidden) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k) ss = fmaf(x[c][k], x[c][k], ss);
+        }
+    ss = block_sum(ss, scratch);
+    const float f2 = 1.f / sqrtf(ss / (float)hidden + eps);
+#pragma unroll
+    for (int c = 0; c < CH; ++c)
+        if (at(c) < hidden) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k) y[c][k] = x[c][k] * f2 * gain[at(c) + k];
+            Vec<TO, 4>::store(out + row + at(c), y[c]);
+        }
+}
+
 // out[t, j] = gelu_tanh(x[t, j]) (* table[ids[t], j] when a table is given);
 // gelu_tanh(z) = 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))), 32-bit with the exact tangent.
 template <typename T>
@@ -434,14 +562,27 @@ extern "C" int cib_rms_stream(float* residual, const void* delta, int delta_dtyp
     AnyVec pg{post_gain, post_dtype == kBF16}, g{gain, gain_dtype == kBF16};
     const size_t smem = (size_t)hidden * sizeof(float);
     const int has_post = post_gain != nullptr;
-#define CIB_RMS_STREAM(TD, TO) \
-    rms_stream_kernel<TD, TO><<<rows, 256, smem, stream>>>(residual, (const TD*)delta, pg, has_post, post_eps, g, eps, (TO*)out, (TO*)raw, hidden)
+    // up to 1 024 values a row: as many threads as it has fours; beyond, 256 threads with up to eight fours each
+    const bool vec = hidden % 4 == 0 && hidden <= 8192, pdl = prompt_pdl();
+    const int threads = hidden >= 1024 ? 256 : std::max(32, (hidden / 4 + 31) / 32 * 32);
+#define CIB_RMS_VEC(TD, TO, CH)                                                                                                  \
+    launch_pdl(rms_stream_vec_kernel<TD, TO, CH>, dim3(rows), dim3(threads), 0, stream, pdl, residual, (const TD*)delta, pg, has_post,  \
+               post_eps, g, eps, (TO*)out, (TO*)raw, hidden)
+#define CIB_RMS_STREAM(TD, TO)                                                                                                   \
+    do {                                                                                                                         \
+        if (vec && hidden <= 1024) CIB_RMS_VEC(TD, TO, 1);                                                                       \
+        else if (vec && hidden <= 2048) CIB_RMS_VEC(TD, TO, 2);                                                                  \
+        else if (vec && hidden <= 4096) CIB_RMS_VEC(TD, TO, 4);                                                                  \
+        else if (vec) CIB_RMS_VEC(TD, TO, 8);                                                                                    \
+        else rms_stream_kernel<TD, TO><<<rows, 256, smem, stream>>>(residual, (const TD*)delta, pg, has_post, post_eps, g, eps, (TO*)out, (TO*)raw, hidden); \
+    } while (0)
     const bool d16 = delta && delta_dtype == kBF16, o16 = out_dtype == kBF16;
     if (d16 && o16) CIB_RMS_STREAM(__nv_bfloat16, __nv_bfloat16);
     else if (d16) CIB_RMS_STREAM(__nv_bfloat16, float);
     else if (o16) CIB_RMS_STREAM(float, __nv_bfloat16);
     else CIB_RMS_STREAM(float, float);
 #undef CIB_RMS_STREAM
+#undef CIB_RMS_VEC
     CIB_LAUNCH_CHECK("rms_stream");
     return 0;
 }

@@ -3,8 +3,9 @@
 // The reference sends every projection to cuBLAS with 32-bit accumulation
 // (csrc/ops/projection.cu:13-45).  This kernel is the true 32-bit path (no tensor cores, no reduced
 // precision mode) and the fallback for shapes the tensor-core kernels refuse.  Every output element
-// is one fused-multiply-add chain over k = 0..K-1 in that order, so a row's result does not depend on
-// how many other rows are in the batch.
+// is a sum of fused-multiply-add chains of kBK values each, in the order of k (a chain of its own per
+// tile keeps the rounding of a long K from growing with its running sum), so a row's result does not
+// depend on how many other rows are in the batch.
 #include "common.cuh"
 
 namespace cib {
@@ -43,6 +44,7 @@ gemm_generic_kernel(const TI* __restrict__ a, int lda, const TI* __restrict__ w,
             Ws[lk + e][lrow] = (wn < N && k < K) ? to_f32(w[(size_t)wn * ldw + k]) : 0.f;
         }
         __syncthreads();
+        float part[4][4] = {};
 #pragma unroll
         for (int kk = 0; kk < kBK; ++kk) {
             float av[4], wv[4];
@@ -53,8 +55,12 @@ gemm_generic_kernel(const TI* __restrict__ a, int lda, const TI* __restrict__ w,
 #pragma unroll
             for (int i = 0; i < 4; ++i)
 #pragma unroll
-                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], wv[j], acc[i][j]);
+                for (int j = 0; j < 4; ++j) part[i][j] = fmaf(av[i], wv[j], part[i][j]);
         }
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) acc[i][j] += part[i][j];
         __syncthreads();
     }
 #pragma unroll

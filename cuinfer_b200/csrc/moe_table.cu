@@ -14,9 +14,9 @@
 // and `act_kind` 1 selects the clamped gate  g = min(gate, limit), u = clamp(up, -limit, limit),
 // act = g * sigmoid(1.702 g) * (u + 1)  instead of silu(gate) * up.  `act_kind` 2 is an expert WITHOUT a gate,
 // down_e( relu(up_e h)^2 ): its first matrix is [E][ff][W] (up rows only).  `base_gate` (32-bit, one number per row, `base_gate_stride` apart; may
-// be null): base is multiplied by sigmoid(base_gate[t]) as it is added (a shared expert with a gate of its own), or,
-// with `base_gate_plain`, by base_gate[t] itself (experts whose output is their input: base is h and the factor the sum of
-// their weights).
+// be null): base is multiplied by sigmoid(base_gate[t]) as it is added (a shared expert with a gate of its own).
+// `self_weight` (32-bit, one number per row; may be null): self_weight[t] * h_t is added too (experts whose output is their
+// input: the sum of their weights).
 #include "common.cuh"
 
 namespace cib {
@@ -48,7 +48,7 @@ struct ExpertAct {
     }
 };
 
-__device__ __forceinline__ float base_factor(float g, int plain) { return plain ? g : 1.f / (1.f + expf(-g)); }
+__device__ __forceinline__ float base_factor(float g) { return 1.f / (1.f + expf(-g)); }
 
 template <typename T>
 __device__ __forceinline__ float dot_row(const T* __restrict__ w, const float* __restrict__ x, int n, int lane) {
@@ -195,7 +195,8 @@ __global__ void __launch_bounds__(kMoeWarps * 32)
 moe_table_down_kernel(const T* __restrict__ act, const int* __restrict__ ids, const int* __restrict__ table, int vocab,
                       int top, int experts, const T* __restrict__ down, const T* __restrict__ base, int base_stride,
                       float weight, const float* __restrict__ weights, const float* __restrict__ base_gate, int base_gate_stride,
-                      int base_gate_plain, T* __restrict__ out, int width, int ff, int outs) {
+                      const T* __restrict__ h, int h_stride, const float* __restrict__ self_weight, T* __restrict__ out, int width,
+                      int ff, int outs) {
     extern __shared__ float as[];                       // [top][ff]
     const int t = blockIdx.x;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -204,7 +205,7 @@ moe_table_down_kernel(const T* __restrict__ act, const int* __restrict__ ids, co
     const int id = ids ? ids[t] : t;
     const bool id_ok = id >= 0 && id < vocab;
     const int i0 = blockIdx.y * outs, i_end = min(width, i0 + outs);
-    const float bg = base && base_gate ? base_factor(base_gate[(size_t)t * base_gate_stride], base_gate_plain) : 1.f;
+    const float bg = base && base_gate ? base_factor(base_gate[(size_t)t * base_gate_stride]) : 1.f;
     for (int i = i0 + warp; i < i_end; i += 2 * kMoeWarps) {           // two outputs together
         const int i2 = i + kMoeWarps;
         float sum[2] = {0.f, 0.f};
@@ -225,6 +226,7 @@ moe_table_down_kernel(const T* __restrict__ act, const int* __restrict__ ids, co
                 if (o >= i_end) continue;
                 float v = weights ? sum[r] : sum[r] * weight;
                 if (base) v += to_f32(base[(size_t)t * base_stride + o]) * bg;
+                if (self_weight) v = fmaf(self_weight[t], to_f32(h[(size_t)t * h_stride + o]), v);
                 out[(size_t)t * width + o] = from_f32<T>(v);
             }
         }
@@ -256,8 +258,9 @@ extern "C" int cib_moe_table_gate_up(const void* h, int h_stride, int dtype, con
 
 extern "C" int cib_moe_table_down(const void* act, int dtype, const int* ids, const int* table, int vocab, int top,
                                   int experts, const void* down, const void* base, int base_stride, float weight,
-                                  const float* weights, const float* base_gate, int base_gate_stride, int base_gate_plain, void* out,
-                                  int num_tokens, int width, int ff, cudaStream_t stream) {
+                                  const float* weights, const float* base_gate, int base_gate_stride, const void* h, int h_stride,
+                                  const float* self_weight, void* out, int num_tokens, int width, int ff, cudaStream_t stream) {
+    CIB_REQUIRE(!self_weight || h, "moe_table: experts that give back their input need it");
     CIB_REQUIRE(num_tokens >= 0 && top > 0 && experts > 0 && width > 0 && ff > 0 && vocab > 0, "moe_table: bad sizes");
     CIB_REQUIRE((size_t)top * ff <= 50 * 1024, "moe_table: %d x %d activations too large for this kernel", top, ff);
     if (num_tokens == 0) return 0;
@@ -271,9 +274,9 @@ extern "C" int cib_moe_table_down(const void* act, int dtype, const int* ids, co
         if (rc != 0) return rc;
     }
     if (dtype == kF32)
-        moe_table_down_kernel<float><<<grid, kMoeWarps * 32, smem, stream>>>((const float*)act, ids, table, vocab, top, experts, (const float*)down, (const float*)base, base_stride, weight, weights, base_gate, base_gate_stride, base_gate_plain, (float*)out, width, ff, outs);
+        moe_table_down_kernel<float><<<grid, kMoeWarps * 32, smem, stream>>>((const float*)act, ids, table, vocab, top, experts, (const float*)down, (const float*)base, base_stride, weight, weights, base_gate, base_gate_stride, (const float*)h, h_stride, self_weight, (float*)out, width, ff, outs);
     else if (dtype == kBF16)
-        moe_table_down_kernel<__nv_bfloat16><<<grid, kMoeWarps * 32, smem, stream>>>((const __nv_bfloat16*)act, ids, table, vocab, top, experts, (const __nv_bfloat16*)down, (const __nv_bfloat16*)base, base_stride, weight, weights, base_gate, base_gate_stride, base_gate_plain, (__nv_bfloat16*)out, width, ff, outs);
+        moe_table_down_kernel<__nv_bfloat16><<<grid, kMoeWarps * 32, smem, stream>>>((const __nv_bfloat16*)act, ids, table, vocab, top, experts, (const __nv_bfloat16*)down, (const __nv_bfloat16*)base, base_stride, weight, weights, base_gate, base_gate_stride, (const __nv_bfloat16*)h, h_stride, self_weight, (__nv_bfloat16*)out, width, ff, outs);
     else
         CIB_REQUIRE(false, "moe_table: unsupported dtype %d", dtype);
     CIB_LAUNCH_CHECK("moe_table_down");
@@ -288,7 +291,7 @@ extern "C" int cib_moe_table_down(const void* act, int dtype, const int* ids, co
 //             which changes no result: every row is computed on its own)
 //   grouped : out rows of a tile = A rows x W_e^T on mma.sync m16n8k16 — with A gathered through the slot list and
 //             silu(gate) * up as the epilogue for the first product, plain for the second
-//   combine : out[t] = base[t] + weight * sum over the token's slots of its down-projected rows
+//   combine : out[t] = base[t] + weight * sum over the token's slots of its down-projected rows (+ self_weight * h[t])
 #include "mma_utils.cuh"
 
 namespace cib {
@@ -465,9 +468,10 @@ moe_grouped_gemm_kernel(const __nv_bfloat16* __restrict__ a, int lda, const int*
 __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const int* __restrict__ slot_pos, int top,
                                    const __nv_bfloat16* __restrict__ base, int base_stride, float weight,
                                    const float* __restrict__ weights, const float* __restrict__ base_gate, int base_gate_stride,
-                                   int base_gate_plain, __nv_bfloat16* __restrict__ out, int width) {
+                                   const __nv_bfloat16* __restrict__ h, int h_stride, const float* __restrict__ self_weight,
+                                   __nv_bfloat16* __restrict__ out, int width) {
     const int t = blockIdx.x;
-    const float bg = base && base_gate ? base_factor(base_gate[(size_t)t * base_gate_stride], base_gate_plain) : 1.f;
+    const float bg = base && base_gate ? base_factor(base_gate[(size_t)t * base_gate_stride]) : 1.f;
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
         float sum = 0.f;
         for (int k = 0; k < top; ++k) {
@@ -476,6 +480,7 @@ __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const in
         }
         float v = weights ? sum : sum * weight;
         if (base) v += __bfloat162float(base[(size_t)t * base_stride + i]) * bg;
+        if (self_weight) v = fmaf(self_weight[t], __bfloat162float(h[(size_t)t * h_stride + i]), v);
         out[(size_t)t * width + i] = __float2bfloat16_rn(v);
     }
 }
@@ -496,8 +501,8 @@ extern "C" long long cib_moe_table_grouped_workspace_ints(int num_tokens, int to
 // bfloat16 only.  act: [T * top, ff] and y: [T * top, width] scratch rows; ints: see above.
 extern "C" int cib_moe_table_grouped(const void* h, int h_stride, const int* ids, const int* table, int vocab, int top,
                                      int experts, const void* gate_up, const void* down, const void* base, int base_stride,
-                                     float weight, const float* weights, const float* base_gate, int base_gate_stride, int base_gate_plain,
-                                     void* out, void* act, void* y, int* ints, int num_tokens, int width, int ff, int act_kind, float limit,
+                                     float weight, const float* weights, const float* base_gate, int base_gate_stride,
+                                     const float* self_weight, void* out, void* act, void* y, int* ints, int num_tokens, int width, int ff, int act_kind, float limit,
                                      cudaStream_t stream) {
     using namespace cib;
     CIB_REQUIRE(num_tokens >= 0 && top > 0 && vocab > 0, "moe_table_grouped: bad sizes");
@@ -537,7 +542,8 @@ extern "C" int cib_moe_table_grouped(const void* h, int h_stride, const int* ids
                                                            tile_row0, num_tiles, width, ff, ExpertAct{-1, 0.f});
     CIB_LAUNCH_CHECK("moe_grouped_down");
     moe_combine_kernel<<<num_tokens, 256, 0, stream>>>((const __nv_bfloat16*)y, slot_pos, top, (const __nv_bfloat16*)base, base_stride,
-                                                       weight, weights, base_gate, base_gate_stride, base_gate_plain, (__nv_bfloat16*)out, width);
+                                                       weight, weights, base_gate, base_gate_stride, (const __nv_bfloat16*)h, h_stride, self_weight,
+                                                       (__nv_bfloat16*)out, width);
     CIB_LAUNCH_CHECK("moe_combine");
     return 0;
 }

@@ -2,7 +2,7 @@
 //  * router_topk: from logits z[t, 0..E-1] the `top` largest (the lower index wins a tie) and their weights, the softmax
 //    over the chosen logits only.
 //  * router_scored_topk: scores s = sigmoid(z); the choice goes by s + correction[e] (a learned number per expert, may be
-//    null), the weights by s alone, times `scale`, not renormalised.  The experts form `groups` equal groups of
+//    null), the weights by s alone, times `scale`, not renormalised or, with `renorm`, over their sum (+ 1e-20) first.  The experts form `groups` equal groups of
 //    neighbours (with `softmax` the scores are the softmax over ALL of the row's logits instead); a group's mark is the sum of its two largest choice scores (of its one, for groups of one), and only
 //    experts of the `keep` groups with the largest marks can be chosen (the lower group wins a tie).  `identity_weight`,
 //    if given, gets the sum of a token's weights of chosen experts from index `identity_from` on: experts without
@@ -64,7 +64,7 @@ constexpr int kScoredWarps = 4;
 // Shared memory per warp: E choice scores, then `groups` marks.
 __global__ void __launch_bounds__(kScoredWarps * 32)
 router_scored_topk_kernel(const float* __restrict__ logits, int stride, int experts, int top, const float* __restrict__ correction,
-                          int groups, int keep, float scale, int softmax, int identity_from, int* __restrict__ choice,
+                          int groups, int keep, float scale, int softmax, int renorm, int identity_from, int* __restrict__ choice,
                           float* __restrict__ weight, float* __restrict__ identity_weight, int num_tokens) {
     extern __shared__ float scored_s[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -147,13 +147,20 @@ router_scored_topk_kernel(const float* __restrict__ logits, int stride, int expe
         }
         __syncwarp();
     }
+    if (renorm && lane == 0) {                                    // the lane that has written the weights
+        float sum = 0.f;
+        for (int k = 0; k < top; ++k) sum += weight[(size_t)t * top + k];
+        const float inv = scale / (sum + scale * 1e-20f);
+        for (int k = 0; k < top; ++k) weight[(size_t)t * top + k] *= inv;
+        identity *= inv;
+    }
     if (identity_weight && lane == 0) identity_weight[t] = identity;
 }
 
 }  // namespace cib
 
 extern "C" int cib_router_scored_topk(const float* logits, int stride, int experts, int top, const float* correction,
-                                      int groups, int keep, float scale, int softmax, int identity_from, int* choice,
+                                      int groups, int keep, float scale, int softmax, int renorm, int identity_from, int* choice,
                                       float* weight, float* identity_weight, int num_tokens, cudaStream_t stream) {
     using namespace cib;
     CIB_REQUIRE(experts > 0 && top > 0 && top <= experts, "router_scored_topk: top %d of %d experts", top, experts);
@@ -165,7 +172,7 @@ extern "C" int cib_router_scored_topk(const float* logits, int stride, int exper
     static SmemLimit limit;
     if (smem > 48 * 1024 && raise_smem_limit(limit, router_scored_topk_kernel, 200 * 1024, "router_scored_topk") != 0) return -2;
     router_scored_topk_kernel<<<(num_tokens + kScoredWarps - 1) / kScoredWarps, kScoredWarps * 32, smem, stream>>>(
-        logits, stride, experts, top, correction, groups, keep, scale, softmax, identity_from, choice, weight, identity_weight,
+        logits, stride, experts, top, correction, groups, keep, scale, softmax, renorm, identity_from, choice, weight, identity_weight,
         num_tokens);
     CIB_LAUNCH_CHECK("router_scored_topk");
     return 0;

@@ -1,0 +1,498 @@
+// The state-space recurrence with a scalar decay per head (the Mamba-2 form), and the gated norm that follows it.
+//
+// Rows [x (H P) | B (G N) | C (G N)] of every token, a step size per head dt = softplus(z + dt_bias), head h with the B and C of
+// group h / (H / G); S is [P][N] (a head's state; N values of one output side by side):
+//
+//   S <- exp(-exp(A_log) dt) S + dt x B^T;     y = S C + D x
+//
+// Requests, slots and the order of tokens as in recurrent.cu.  Step sizes, decays, state and read-out are 32-bit.
+//
+// Two kernels.
+//  * ssm_walk: token after token in 32-bit FMA, any sizes; a warp holds four rows of S over its lanes.  Steps of single tokens,
+//    the 32-bit engine, sizes the other does not take.
+//  * ssm_chunk (bfloat16 rows): 64 tokens at a time on the tensor cores.  With L_t the sum of the log decays of a chunk's tokens
+//    up to t, and S0 the state before the chunk,
+//        y_t = exp(L_t) S0 C_t + sum_(s <= t) [exp(L_t - L_s) dt_s (C_t . B_s)] x_s + D x_t
+//        S   = exp(L_end) S0 + sum_s [exp(L_end - L_s) dt_s x_s] B_s^T
+//    x, B and C enter as they are stored; the 32-bit factors — S0 and the bracketed values — enter as two bfloat16 numbers
+//    each (value and remainder), so that a product keeps 16 bits of them.  S0 stays in registers as the accumulators of the
+//    update, whose layout is that of a product's first operand.
+#include "mma_utils.cuh"
+#include "scan_utils.cuh"
+
+namespace cib {
+
+constexpr int kSsmWarps = 4, kSsmRows = 4;       // a block walks kSsmWarps * kSsmRows rows of a head's state
+
+template <typename T, int C>
+__global__ void __launch_bounds__(kSsmWarps * 32)
+ssm_walk_kernel(const T* __restrict__ rows, int stride, const float* __restrict__ z, int z_stride, AnyVec dt_bias, AnyVec a_log, AnyVec skip,
+                float* __restrict__ state, const int* __restrict__ query_start_loc, const int* __restrict__ state_slots, int num_slots,
+                float* __restrict__ out, int H, int G, int P, int N) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int r = blockIdx.x, h = blockIdx.y, p0 = (blockIdx.z * kSsmWarps + warp) * kSsmRows;
+    griddep_launch();
+    const float a = -expf(a_log[h]), bias = dt_bias[h], dskip = skip[h];          // weights
+    griddep_wait();
+    const int t0 = query_start_loc[r], t1 = query_start_loc[r + 1];
+    if (t1 <= t0 || p0 >= P) return;
+    const int slot = state_slots[r];
+    const bool has = slot >= 0 && slot < num_slots;
+    float* st = has ? state + (((size_t)slot * H + h) * P + p0) * N : nullptr;
+    float S[kSsmRows][C];
+#pragma unroll
+    for (int q = 0; q < kSsmRows; ++q)
+#pragma unroll
+        for (int c = 0; c < C; ++c) S[q][c] = (has && p0 + q < P && c * 32 + lane < N) ? st[(size_t)q * N + c * 32 + lane] : 0.f;
+    const T* x_ = rows + (size_t)h * P + p0;
+    const T* b_ = rows + (size_t)H * P + (size_t)(h / (H / G)) * N;
+    const T* c_ = b_ + (size_t)G * N;
+    float nb[C], nc[C], nx[kSsmRows], nz;
+    auto fetch = [&](int t) {
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+            const bool ok = c * 32 + lane < N;
+            nb[c] = ok ? to_f32(b_[(size_t)t * stride + c * 32 + lane]) : 0.f;
+            nc[c] = ok ? to_f32(c_[(size_t)t * stride + c * 32 + lane]) : 0.f;
+        }
+#pragma unroll
+        for (int q = 0; q < kSsmRows; ++q) nx[q] = p0 + q < P ? to_f32(x_[(size_t)t * stride + q]) : 0.f;
+        nz = z[(size_t)t * z_stride + h];
+    };
+    fetch(t0);
+    for (int t = t0; t < t1; ++t) {
+        float b[C], cc[C], x[kSsmRows];
+#pragma unroll
+        for (int c = 0; c < C; ++c) { b[c] = nb[c]; cc[c] = nc[c]; }
+#pragma unroll
+        for (int q = 0; q < kSsmRows; ++q) x[q] = nx[q];
+        const float dt = softplusf_(nz + bias);
+        if (t + 1 < t1) fetch(t + 1);                       // the next token's values are on their way meanwhile
+        // g S as keep S + (g - keep) S, keep = 1 for a slow decay: what a decay close to one takes off is then rounded by
+        // itself, not with the one (over a thousand tokens the difference is a digit)
+        const float ld = a * dt, keep = ld > -0.5f ? 1.f : 0.f, rest = keep != 0.f ? expm1f(ld) : expf(ld);
+        float y[kSsmRows];
+#pragma unroll
+        for (int q = 0; q < kSsmRows; ++q) {
+            const float xd = dt * x[q];
+            float acc = 0.f;
+#pragma unroll
+            for (int c = 0; c < C; ++c) {
+                S[q][c] = fmaf(keep, S[q][c], fmaf(rest, S[q][c], xd * b[c]));
+                acc = fmaf(S[q][c], cc[c], acc);
+            }
+            y[q] = acc;
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+            for (int q = 0; q < kSsmRows; ++q) y[q] += __shfl_xor_sync(0xffffffffu, y[q], o);
+#pragma unroll
+        for (int q = 0; q < kSsmRows; ++q)
+            if (lane == q && p0 + q < P) out[(size_t)t * H * P + (size_t)h * P + p0 + q] = fmaf(dskip, x[q], y[q]);
+    }
+    if (!has) return;
+#pragma unroll
+    for (int q = 0; q < kSsmRows; ++q)
+#pragma unroll
+        for (int c = 0; c < C; ++c)
+            if (p0 + q < P && c * 32 + lane < N) st[(size_t)q * N + c * 32 + lane] = S[q][c];
+}
+
+// ---- chunks of 64 tokens on the tensor cores -----------------------------------------------------------------------------
+constexpr int kChunk = 64;
+constexpr int kChunkLd = kChunk + 8;
+
+__device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint32_t& lo) {
+    hi = pack_bf16(a, b);
+    const __nv_bfloat162 h = *reinterpret_cast<const __nv_bfloat162*>(&hi);
+    lo = pack_bf16(a - __low2float(h), b - __high2float(h));
+}
+
+template <int NP, int NW> constexpr size_t ssm_chunk_smem() {
+    constexpr int PT = NW * 16;
+    return (size_t)2 * (2 * kChunk * (NP + 8) + kChunk * (PT + 8)) * 2      // two stages of C, B, x
+           + (size_t)2 * kChunk * (PT + 8) * 2                              // weighted x, value and remainder
+           + (size_t)2 * kChunk * kChunkLd * 2                              // the weights of a chunk's pairs, likewise
+           + (size_t)4 * kChunk * 4;                                        // L, dt, exp(L), weights of the update
+}
+
+// A CTA of NW warps walks the chunks of one request for 16 NW rows of one head's S; each warp owns 16 rows, and
+// 64 / NW rows of the chunk's pairs.
+template <int NP, int NW>
+__global__ void __launch_bounds__(NW * 32)
+ssm_chunk_kernel(const __nv_bfloat16* __restrict__ rows, int stride, const float* __restrict__ z, int z_stride, AnyVec dt_bias, AnyVec a_log,
+                 AnyVec skip, float* __restrict__ state, const int* __restrict__ query_start_loc, const int* __restrict__ state_slots,
+                 int num_slots, float* __restrict__ out, int H, int G, int P, int N) {
+    constexpr int PT = NW * 16, LDN = NP + 8, LDP = PT + 8, MT = 4 / NW;
+    constexpr int kStage = 2 * kChunk * LDN + kChunk * LDP;
+    extern __shared__ __align__(16) unsigned char ssm_raw[];
+    __nv_bfloat16* stages = reinterpret_cast<__nv_bfloat16*>(ssm_raw);
+    __nv_bfloat16* xw_hi = stages + 2 * kStage;
+    __nv_bfloat16* xw_lo = xw_hi + kChunk * LDP;
+    __nv_bfloat16* w_hi = xw_lo + kChunk * LDP;
+    __nv_bfloat16* w_lo = w_hi + kChunk * kChunkLd;
+    float* Ls = reinterpret_cast<float*>(w_lo + kChunk * kChunkLd);
+    float* dts = Ls + kChunk;
+    float* eL = dts + kChunk;
+    float* wu = eL + kChunk;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int r = blockIdx.z, h = blockIdx.x, p_base = blockIdx.y * PT;
+    const int t0 = query_start_loc[r], t1 = query_start_loc[r + 1];
+    if (t1 <= t0) return;
+    const int slot = state_slots[r];
+    const bool has = slot >= 0 && slot < num_slots;
+    const int qrow = lane >> 2, quad = lane & 3, mat = lane >> 3, rr = lane & 7;
+    const int p_lo = p_base + warp * 16 + qrow, p_hi = p_lo + 8;
+    const float a = -expf(a_log[h]), bias = dt_bias[h], dskip = skip[h];
+    const __nv_bfloat16* x_ = rows + (size_t)h * P + p_base;
+    const __nv_bfloat16* b_ = rows + (size_t)H * P + (size_t)(h / (H / G)) * N;
+    const __nv_bfloat16* c_ = b_ + (size_t)G * N;
+
+    auto load = [&](int stage, int base) {
+        const int count = min(kChunk, t1 - base);
+        __nv_bfloat16* cs = stages + stage * kStage;
+        __nv_bfloat16 *bs = cs + kChunk * LDN, *xs = bs + kChunk * LDN;
+        for (int idx = tid; idx < kChunk * (NP / 8); idx += NW * 32) {
+            const int s = idx / (NP / 8), n = (idx % (NP / 8)) * 8;
+            const bool ok = s < count && n < N;
+            const size_t at = ok ? (size_t)(base + s) * stride + n : 0;
+            cp_async16(cs + s * LDN + n, c_ + at, ok);
+            cp_async16(bs + s * LDN + n, b_ + at, ok);
+        }
+        for (int idx = tid; idx < kChunk * (PT / 8); idx += NW * 32) {
+            const int s = idx / (PT / 8), p = (idx % (PT / 8)) * 8;
+            const bool ok = s < count && p_base + p < P;
+            cp_async16(xs + s * LDP + p, x_ + (ok ? (size_t)(base + s) * stride + p : 0), ok);
+        }
+    };
+    // the two step sizes of a chunk that this lane of the first warp takes care of: tokens 2 lane and 2 lane + 1
+    auto raw_step = [&](int base, int s) { return base + s < t1 ? z[(size_t)(base + s) * z_stride + h] : 0.f; };
+
+    load(0, t0);
+    cp_async_commit();
+    float z0 = 0.f, z1 = 0.f;
+    if (warp == 0) {
+        z0 = raw_step(t0, 2 * lane);
+        z1 = raw_step(t0, 2 * lane + 1);
+    }
+    float S[NP / 8][4];                                          // rows p_lo, p_hi; columns 8 j + 2 quad, + 1
+    {
+        const float* st = has ? state + ((size_t)slot * H + h) * P * N : nullptr;
+#pragma unroll
+        for (int j = 0; j < NP / 8; ++j) {
+            const int n = j * 8 + quad * 2;
+            const float2 lo = has && n < N && p_lo < P ? *reinterpret_cast<const float2*>(st + (size_t)p_lo * N + n) : make_float2(0.f, 0.f);
+            const float2 hi = has && n < N && p_hi < P ? *reinterpret_cast<const float2*>(st + (size_t)p_hi * N + n) : make_float2(0.f, 0.f);
+            S[j][0] = lo.x; S[j][1] = lo.y; S[j][2] = hi.x; S[j][3] = hi.y;
+        }
+    }
+    int stage = 0;
+    for (int base = t0; base < t1; base += kChunk, stage ^= 1) {
+        const int count = min(kChunk, t1 - base), next = base + kChunk;
+        if (next < t1) load(stage ^ 1, next);
+        cp_async_commit();
+        if (warp == 0) {
+            const bool ok0 = 2 * lane < count, ok1 = 2 * lane + 1 < count;
+            const float d0 = ok0 ? softplusf_(z0 + bias) : 0.f, d1 = ok1 ? softplusf_(z1 + bias) : 0.f;
+            if (next < t1) {
+                z0 = raw_step(next, 2 * lane);
+                z1 = raw_step(next, 2 * lane + 1);
+            }
+            const float l0 = a * d0, l1 = a * d1;
+            float sum = l0 + l1;                                 // inclusive over the lanes' pairs
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const float v = __shfl_up_sync(0xffffffffu, sum, o);
+                if (lane >= o) sum += v;
+            }
+            const float end = __shfl_sync(0xffffffffu, sum, 31);
+            const float first = sum - l1;
+            Ls[2 * lane] = first;
+            Ls[2 * lane + 1] = sum;
+            dts[2 * lane] = d0;
+            dts[2 * lane + 1] = d1;
+            eL[2 * lane] = expf(first);
+            eL[2 * lane + 1] = expf(sum);
+            wu[2 * lane] = expf(end - first) * d0;
+            wu[2 * lane + 1] = expf(end - sum) * d1;
+        }
+        cp_async_wait<1>();
+        __syncthreads();
+        const __nv_bfloat16* cs = stages + stage * kStage;
+        const __nv_bfloat16 *bs = cs + kChunk * LDN, *xs = bs + kChunk * LDN;
+
+        // x weighted for the update
+        for (int idx = tid; idx < kChunk * (PT / 2); idx += NW * 32) {
+            const int s = idx / (PT / 2), p = (idx % (PT / 2)) * 2;
+            const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(xs + s * LDP + p);
+            uint32_t hi, lo;
+            split_bf16(wu[s] * __low2float(v), wu[s] * __high2float(v), hi, lo);
+            *reinterpret_cast<uint32_t*>(xw_hi + s * LDP + p) = hi;
+            *reinterpret_cast<uint32_t*>(xw_lo + s * LDP + p) = lo;
+        }
+        // this warp's rows of C B^T, weighted; tiles above the diagonal are zero and never read
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+            const int tr = (warp * MT + m) * 16;
+            float g[kChunk / 8][4];
+#pragma unroll
+            for (int j = 0; j < kChunk / 8; ++j) g[j][0] = g[j][1] = g[j][2] = g[j][3] = 0.f;
+#pragma unroll 4
+            for (int kk = 0; kk < NP / 16; ++kk) {
+                uint32_t af[4];
+                ldmatrix_x4(af, smem_u32(cs + (tr + (mat & 1) * 8 + rr) * LDN + kk * 16 + (mat >> 1) * 8));
+#pragma unroll
+                for (int np = 0; np < kChunk / 16; ++np) {
+                    if (np * 16 > tr) continue;
+                    uint32_t bf[4];
+                    ldmatrix_x4(bf, smem_u32(bs + (np * 16 + (mat >> 1) * 8 + rr) * LDN + kk * 16 + (mat & 1) * 8));
+                    mma_bf16_16816(g[2 * np], af, bf[0], bf[1]);
+                    mma_bf16_16816(g[2 * np + 1], af, bf[2], bf[3]);
+                }
+            }
+            const int ta = tr + qrow, tb = ta + 8;
+            const float La = Ls[ta], Lb = Ls[tb];
+#pragma unroll
+            for (int j = 0; j < kChunk / 8; ++j) {
+                if (j * 8 >= tr + 16) continue;
+                const int s = j * 8 + quad * 2;
+                const float ls0 = Ls[s], ls1 = Ls[s + 1], d0 = dts[s], d1 = dts[s + 1];
+                uint32_t hi, lo;
+                split_bf16(s <= ta ? g[j][0] * expf(La - ls0) * d0 : 0.f, s + 1 <= ta ? g[j][1] * expf(La - ls1) * d1 : 0.f, hi, lo);
+                *reinterpret_cast<uint32_t*>(w_hi + ta * kChunkLd + s) = hi;
+                *reinterpret_cast<uint32_t*>(w_lo + ta * kChunkLd + s) = lo;
+                split_bf16(s <= tb ? g[j][2] * expf(Lb - ls0) * d0 : 0.f, s + 1 <= tb ? g[j][3] * expf(Lb - ls1) * d1 : 0.f, hi, lo);
+                *reinterpret_cast<uint32_t*>(w_hi + tb * kChunkLd + s) = hi;
+                *reinterpret_cast<uint32_t*>(w_lo + tb * kChunkLd + s) = lo;
+            }
+        }
+        // y = S0 C^T: rows of S from the registers
+        float y[kChunk / 8][4];
+#pragma unroll
+        for (int j = 0; j < kChunk / 8; ++j) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
+#pragma unroll
+        for (int kk = 0; kk < NP / 16; ++kk) {
+            uint32_t hi[4], lo[4];
+            split_bf16(S[2 * kk][0], S[2 * kk][1], hi[0], lo[0]);
+            split_bf16(S[2 * kk][2], S[2 * kk][3], hi[1], lo[1]);
+            split_bf16(S[2 * kk + 1][0], S[2 * kk + 1][1], hi[2], lo[2]);
+            split_bf16(S[2 * kk + 1][2], S[2 * kk + 1][3], hi[3], lo[3]);
+#pragma unroll
+            for (int np = 0; np < kChunk / 16; ++np) {
+                uint32_t bf[4];
+                ldmatrix_x4(bf, smem_u32(cs + (np * 16 + (mat >> 1) * 8 + rr) * LDN + kk * 16 + (mat & 1) * 8));
+                mma_bf16_16816(y[2 * np], hi, bf[0], bf[1]);
+                mma_bf16_16816(y[2 * np + 1], hi, bf[2], bf[3]);
+                mma_bf16_16816(y[2 * np], lo, bf[0], bf[1]);
+                mma_bf16_16816(y[2 * np + 1], lo, bf[2], bf[3]);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < kChunk / 8; ++j) {
+            const float e0 = eL[j * 8 + quad * 2], e1 = eL[j * 8 + quad * 2 + 1];
+            y[j][0] *= e0; y[j][1] *= e1; y[j][2] *= e0; y[j][3] *= e1;
+        }
+        const float e_end = eL[kChunk - 1];                      // a token beyond the chunk's count has a step of zero
+#pragma unroll
+        for (int j = 0; j < NP / 8; ++j) { S[j][0] *= e_end; S[j][1] *= e_end; S[j][2] *= e_end; S[j][3] *= e_end; }
+        __syncthreads();                                         // weighted x and pair weights are in place
+#pragma unroll
+        for (int kk = 0; kk < kChunk / 16; ++kk) {
+            const int s0 = kk * 16;
+            uint32_t xa[4], wa_hi[4], wa_lo[4];
+            const int at = (s0 + (mat >> 1) * 8 + rr) * LDP + warp * 16 + (mat & 1) * 8;
+            ldmatrix_x4_trans(xa, smem_u32(xs + at));
+            ldmatrix_x4_trans(wa_hi, smem_u32(xw_hi + at));
+            ldmatrix_x4_trans(wa_lo, smem_u32(xw_lo + at));
+#pragma unroll
+            for (int np = 0; np < kChunk / 16; ++np) {
+                if (np < kk) continue;                           // tokens before s0 do not see it
+                uint32_t bf[4];
+                ldmatrix_x4(bf, smem_u32(w_hi + (np * 16 + (mat >> 1) * 8 + rr) * kChunkLd + s0 + (mat & 1) * 8));
+                mma_bf16_16816(y[2 * np], xa, bf[0], bf[1]);
+                mma_bf16_16816(y[2 * np + 1], xa, bf[2], bf[3]);
+                ldmatrix_x4(bf, smem_u32(w_lo + (np * 16 + (mat >> 1) * 8 + rr) * kChunkLd + s0 + (mat & 1) * 8));
+                mma_bf16_16816(y[2 * np], xa, bf[0], bf[1]);
+                mma_bf16_16816(y[2 * np + 1], xa, bf[2], bf[3]);
+            }
+#pragma unroll
+            for (int nj = 0; nj < NP / 16; ++nj) {
+                uint32_t bf[4];
+                ldmatrix_x4_trans(bf, smem_u32(bs + (s0 + (mat & 1) * 8 + rr) * LDN + nj * 16 + (mat >> 1) * 8));
+                mma_bf16_16816(S[2 * nj], wa_hi, bf[0], bf[1]);
+                mma_bf16_16816(S[2 * nj + 1], wa_hi, bf[2], bf[3]);
+                mma_bf16_16816(S[2 * nj], wa_lo, bf[0], bf[1]);
+                mma_bf16_16816(S[2 * nj + 1], wa_lo, bf[2], bf[3]);
+            }
+        }
+        const int xl = warp * 16 + qrow;                         // this lane's rows within x's columns
+#pragma unroll
+        for (int j = 0; j < kChunk / 8; ++j) {
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int s = j * 8 + quad * 2 + e;
+                if (s >= count) continue;
+                float* dst = out + ((size_t)(base + s) * H + h) * P;
+                if (p_lo < P) dst[p_lo] = fmaf(dskip, __bfloat162float(xs[s * LDP + xl]), y[j][e]);
+                if (p_hi < P) dst[p_hi] = fmaf(dskip, __bfloat162float(xs[s * LDP + xl + 8]), y[j][2 + e]);
+            }
+        }
+        __syncthreads();                                         // the stage and the scratch are free
+    }
+    if (!has) return;
+    float* st = state + ((size_t)slot * H + h) * P * N;
+#pragma unroll
+    for (int j = 0; j < NP / 8; ++j) {
+        const int n = j * 8 + quad * 2;
+        if (n >= N) continue;
+        if (p_lo < P) *reinterpret_cast<float2*>(st + (size_t)p_lo * N + n) = make_float2(S[j][0], S[j][1]);
+        if (p_hi < P) *reinterpret_cast<float2*>(st + (size_t)p_hi * N + n) = make_float2(S[j][2], S[j][3]);
+    }
+}
+
+// ---- the gate, then an RMS norm in groups, then the gain --------------------------------------------------------------------
+// v = y * silu(z);  out = v / sqrt(mean over the group of v^2 + eps) * gain.  A block per (token, group), v in shared memory.
+template <typename TZ, typename TO, int V>
+__global__ void __launch_bounds__(256)
+gated_group_rms_kernel(const float* __restrict__ y, const TZ* __restrict__ z, int z_stride, AnyVec gain, float eps, TO* __restrict__ out,
+                       int groups, int width) {
+    extern __shared__ __align__(16) float gated_s[];
+    __shared__ float scratch[33];
+    griddep_launch();
+    griddep_wait();
+    const int t = blockIdx.x / groups, g = blockIdx.x % groups;
+    const size_t at = (size_t)blockIdx.x * width;
+    const TZ* zr = z + (size_t)t * z_stride + (size_t)g * width;
+    float ss = 0.f;
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+        float v[V], zz[V];
+        if constexpr (V == 4) {
+            const float4 f = *reinterpret_cast<const float4*>(y + at + i);
+            v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+            if constexpr (sizeof(TZ) == 2) {
+                const uint2 u = *reinterpret_cast<const uint2*>(zr + i);
+                const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&u.x), b = *reinterpret_cast<const __nv_bfloat162*>(&u.y);
+                zz[0] = __low2float(a); zz[1] = __high2float(a); zz[2] = __low2float(b); zz[3] = __high2float(b);
+            } else {
+                const float4 f2 = *reinterpret_cast<const float4*>(zr + i);
+                zz[0] = f2.x; zz[1] = f2.y; zz[2] = f2.z; zz[3] = f2.w;
+            }
+        } else {
+            v[0] = y[at + i];
+            zz[0] = to_f32(zr[i]);
+        }
+#pragma unroll
+        for (int k = 0; k < V; ++k) {
+            v[k] *= zz[k] / (1.f + expf(-zz[k]));
+            ss = fmaf(v[k], v[k], ss);
+            gated_s[i + k] = v[k];
+        }
+    }
+    ss = block_sum(ss, scratch);
+    const float factor = 1.f / sqrtf(ss / (float)width + eps);
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {           // the elements this thread has written itself
+        float v[V];
+#pragma unroll
+        for (int k = 0; k < V; ++k) v[k] = gated_s[i + k] * factor * gain[g * width + i + k];
+        if constexpr (V == 4 && sizeof(TO) == 2) *reinterpret_cast<uint2*>(out + at + i) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
+        else if constexpr (V == 4) *reinterpret_cast<float4*>(out + at + i) = make_float4(v[0], v[1], v[2], v[3]);
+        else out[at + i] = from_f32<TO>(v[0]);
+    }
+}
+
+}  // namespace cib
+
+using namespace cib;
+
+extern "C" int cib_ssm_chunk_supports(int H, int G, int P, int N) {
+    return H > 0 && G > 0 && P % 8 == 0 && N % 8 == 0 && N <= 256 && H % G == 0;
+}
+
+template <int NP, int NW>
+static int launch_ssm_chunk(const void* rows, int stride, const float* z, int z_stride, AnyVec db, AnyVec al, AnyVec sk, float* state,
+                            const int* query_start_loc, const int* state_slots, int num_slots, int num_requests, float* out, int H, int G, int P,
+                            int N, cudaStream_t stream) {
+    constexpr size_t smem = ssm_chunk_smem<NP, NW>();
+    static SmemLimit limit;
+    if (int rc = raise_smem_limit(limit, ssm_chunk_kernel<NP, NW>, smem, "ssm_chunk")) return rc;
+    const dim3 grid(H, (P + NW * 16 - 1) / (NW * 16), num_requests);
+    ssm_chunk_kernel<NP, NW><<<grid, NW * 32, smem, stream>>>((const __nv_bfloat16*)rows, stride, z, z_stride, db, al, sk, state, query_start_loc,
+                                                             state_slots, num_slots, out, H, G, P, N);
+    CIB_LAUNCH_CHECK("ssm_chunk");
+    return 0;
+}
+
+// rows [tokens][>= H P + 2 G N] `stride` apart; z float32 step-size logits [tokens][>= H] `z_stride` apart; dt_bias, a_log, skip [H];
+// state float32 [slots][H][P][N]; out float32 [tokens][H P].  chunks: take the tensor-core form (bfloat16 rows on 16-byte
+// boundaries, sizes in multiples of 8).
+extern "C" int cib_ssm_scan(const void* rows, int dtype, int stride, const float* z, int z_stride, const void* dt_bias, const void* a_log,
+                            const void* skip, int vec_dtype, float* state, const int* query_start_loc, const int* state_slots, int num_slots,
+                            int num_requests, int num_tokens, float* out, int H, int G, int P, int N, int chunks, cudaStream_t stream) {
+    CIB_REQUIRE(H > 0 && G > 0 && H % G == 0 && P > 0 && N > 0 && stride >= H * P + 2 * G * N && z_stride >= H, "ssm_scan: bad sizes");
+    CIB_REQUIRE(N <= 256, "ssm_scan: state size %d is beyond 256", N);
+    if (num_requests == 0 || num_tokens == 0) return 0;
+    AnyVec db{dt_bias, vec_dtype == kBF16}, al{a_log, vec_dtype == kBF16}, sk{skip, vec_dtype == kBF16};
+    if (chunks) {
+        CIB_REQUIRE(dtype == kBF16 && cib_ssm_chunk_supports(H, G, P, N) && stride % 8 == 0 && (uintptr_t)rows % 16 == 0 && (uintptr_t)state % 16 == 0,
+                    "ssm_scan: the rows do not fit the tensor-core form");
+        CIB_REQUIRE(num_requests <= 65535, "ssm_scan: too many requests");
+        // two warps (32 rows of S) a CTA while four would leave SMs without work
+        const bool narrow = P <= 32 || (long long)num_requests * H * ((P + 63) / 64) < 148;
+#define CIB_SSM(NP)                                                                                                                       \
+    return narrow ? launch_ssm_chunk<NP, 2>(rows, stride, z, z_stride, db, al, sk, state, query_start_loc, state_slots, num_slots,           \
+                                            num_requests, out, H, G, P, N, stream)                                                     \
+                  : launch_ssm_chunk<NP, 4>(rows, stride, z, z_stride, db, al, sk, state, query_start_loc, state_slots, num_slots,           \
+                                            num_requests, out, H, G, P, N, stream)
+        if (N <= 32) CIB_SSM(32);
+        if (N <= 64) CIB_SSM(64);
+        if (N <= 128) CIB_SSM(128);
+        CIB_SSM(256);
+#undef CIB_SSM
+    }
+    const dim3 grid(num_requests, H, (P + kSsmWarps * kSsmRows - 1) / (kSsmWarps * kSsmRows));
+    const bool pdl = prompt_pdl();
+#define CIB_WALK(T, C)                                                                                                                    \
+    launch_pdl(ssm_walk_kernel<T, C>, grid, dim3(kSsmWarps * 32), 0, stream, pdl, (const T*)rows, stride, z, z_stride, db, al, sk, state,      \
+               query_start_loc, state_slots, num_slots, out, H, G, P, N)
+#define CIB_WALK_N(T)                         \
+    do {                                      \
+        if (N <= 32) CIB_WALK(T, 1);          \
+        else if (N <= 64) CIB_WALK(T, 2);     \
+        else if (N <= 128) CIB_WALK(T, 4);    \
+        else CIB_WALK(T, 8);                  \
+    } while (0)
+    if (dtype == kF32) CIB_WALK_N(float);
+    else if (dtype == kBF16) CIB_WALK_N(__nv_bfloat16);
+    else CIB_REQUIRE(false, "ssm_scan: bad dtype %d", dtype);
+#undef CIB_WALK_N
+#undef CIB_WALK
+    CIB_LAUNCH_CHECK("ssm_scan");
+    return 0;
+}
+
+// y float32 [tokens][groups * width]; z rows `z_stride` apart; gain [groups * width]; out [tokens][groups * width].
+extern "C" int cib_gated_group_rms(const float* y, const void* z, int z_dtype, int z_stride, const void* gain, int gain_dtype, float eps,
+                                   void* out, int out_dtype, int groups, int width, int num_tokens, cudaStream_t stream) {
+    CIB_REQUIRE(groups > 0 && width > 0 && z_stride >= groups * width && num_tokens >= 0, "gated_group_rms: bad sizes");
+    CIB_REQUIRE(width <= 12 * 1024, "gated_group_rms: groups of %d values are beyond this kernel", width);
+    CIB_REQUIRE((long long)num_tokens * groups < (1ll << 31), "gated_group_rms: too many rows");
+    if (num_tokens == 0) return 0;
+    AnyVec gv{gain, gain_dtype == kBF16};
+    const bool v4 = width % 4 == 0 && z_stride % 4 == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)z % (z_dtype == kF32 ? 16 : 8) == 0 &&
+                    (uintptr_t)out % 16 == 0;
+    int threads = 32;
+    while (threads < 256 && threads * (v4 ? 4 : 1) < width) threads <<= 1;
+    const size_t smem = (size_t)width * sizeof(float);
+    const bool pdl = prompt_pdl();
+#define CIB_GATED(TZ, TO, V)                                                                                                            \
+    launch_pdl(gated_group_rms_kernel<TZ, TO, V>, dim3((unsigned)(num_tokens * groups)), dim3(threads), smem, stream, pdl, y, (const TZ*)z,   \
+               z_stride, gv, eps, (TO*)out, groups, width)
+    if (z_dtype == kF32 && out_dtype == kF32) { if (v4) CIB_GATED(float, float, 4); else CIB_GATED(float, float, 1); }
+    else if (z_dtype == kF32 && out_dtype == kBF16) { if (v4) CIB_GATED(float, __nv_bfloat16, 4); else CIB_GATED(float, __nv_bfloat16, 1); }
+    else if (z_dtype == kBF16 && out_dtype == kBF16) { if (v4) CIB_GATED(__nv_bfloat16, __nv_bfloat16, 4); else CIB_GATED(__nv_bfloat16, __nv_bfloat16, 1); }
+    else CIB_REQUIRE(false, "gated_group_rms: bad dtypes %d -> %d", z_dtype, out_dtype);
+#undef CIB_GATED
+    CIB_LAUNCH_CHECK("gated_group_rms");
+    return 0;
+}

@@ -71,6 +71,14 @@ def _declare(lib: ctypes.CDLL) -> None:
         "cib_embedding_gather": [_P, _P, _I, _P, _I, _I, _I, _P, _F, _I, _P],
         "cib_sandwich_layernorm": [_P, _P, _I, _P, _P, _F, _P, _P, _P, _F, _I, _P, _I, _I, _I, _P],
         "cib_relu_squared": [_P, _P, _I, ctypes.c_longlong, _P],
+        "cib_bias_rows": [_P, _P, _P, _I, _I, _I, _I, _P],
+        "cib_pair_sum": [_P, _P, _F, _F, _P, _I, ctypes.c_longlong, _P],
+        "cib_short_conv": [_P, _I, _I, _P, _I, _P, _P, _I, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _P],
+        "cib_ssm_scan": [_P, _I, _I, _P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _P, _I, _I, _I, _I, _I, _P],
+        "cib_gated_group_rms": [_P, _P, _I, _I, _P, _I, _F, _P, _I, _I, _I, _I, _P],
+        "cib_lru_gates": [_P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _P],
+        "cib_lru_scan": [_P, _P, _I, _I, _P, _F, _P, _P, _P, _I, _I, _I, _P, _I, _I, _P],
+        "cib_lru_decode": [_P, _I, _I, _P, _P, _P, _P, _I, _P, _F, _P, _P, _I, _P, _I, _I, _I, _P],
         "cib_sigmoid_gate": [_P, _I, _P, _I, _P, _I, _I, _I, _P],
         "cib_latent_prep": [_P, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _F, _P, _P, _I, _F, _P, _P, ctypes.c_longlong, _P, _I, _I, _P],
         "cib_latent_attention_generic": [_P, _I, _I, _P, _I, _I, _I, _P, _I, _P, _I, _I, _P, _I, _P, _P, _P, _P, _P, _I, _F, _P, _I,
@@ -80,10 +88,10 @@ def _declare(lib: ctypes.CDLL) -> None:
         "cib_gemm_generic_batched": [_P, _I, ctypes.c_longlong, _P, _I, ctypes.c_longlong, _I, _P, _I, ctypes.c_longlong, _I,
                                      _I, _I, _I, _I, _P],
         "cib_moe_table_gate_up": [_P, _I, _I, _P, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _F, _P],
-        "cib_moe_table_grouped": [_P, _I, _P, _P, _I, _I, _I, _P, _P, _P, _I, _F, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _F, _P],
-        "cib_moe_table_down": [_P, _I, _P, _P, _I, _I, _I, _P, _P, _I, _F, _P, _P, _I, _I, _P, _I, _I, _I, _P],
+        "cib_moe_table_grouped": [_P, _I, _P, _P, _I, _I, _I, _P, _P, _P, _I, _F, _P, _P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _P],
+        "cib_moe_table_down": [_P, _I, _P, _P, _I, _I, _I, _P, _P, _I, _F, _P, _P, _I, _P, _I, _P, _P, _I, _I, _I, _P],
         "cib_window_attention_prep": [_P, _I, _I, _P, _I, _P, _P, _P, _I, _F, _I, _I, _I, _I, _P, _I, _P, _I, _P, ctypes.c_longlong, _I, _I,
-                                      _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _F, _I, _P, _I, _P, _P, _P, _P, _I, _I, _P],
+                                      _P, _P, _P, _I, _I, _I, _I, _F, _I, _I, _F, _I, _P, _I, _P, _P, _P, _P, _I, _I, _I, _P],
         "cib_conv_state_update": [_P, _I, _I, _I, _P, _P, _P, _I, _I, _I, _P, _P],
         "cib_channel_delta_scan": [_P, _I, _I, _P, _I, _P, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _P, _P, _P, _I, _I, _I, _P],
         "cib_wkv_scan": [_P, _P, _P, _I, _I, _P, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _P, _P, _P, _I, _I, _I, _P],
@@ -100,7 +108,7 @@ def _declare(lib: ctypes.CDLL) -> None:
         "cib_delta_scan": [_P, _I, _P, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _P, _I, _I, _I, _P],
         "cib_head_rms_gate": [_P, _P, _I, _I, _P, _I, _I, _F, _I, _P, _I, _I, _I, _P],
         "cib_router_topk": [_P, _I, _I, _I, _P, _P, _I, _P],
-        "cib_router_scored_topk": [_P, _I, _I, _I, _P, _I, _I, _F, _I, _I, _P, _P, _P, _I, _P],
+        "cib_router_scored_topk": [_P, _I, _I, _I, _P, _I, _I, _F, _I, _I, _I, _P, _P, _P, _I, _P],
         "cib_rms_stream": [_P, _P, _I, _P, _I, _F, _P, _I, _F, _P, _P, _I, _I, _I, _P],
         "cib_gelu_tanh": [_P, _P, _I, _P, _I, _P, _I, _I, _I, _P],
         "cib_add_rmsnorm": [_P, _P, _I, _P, _I, _F, _P, _I, _I, _I, _P],
@@ -128,6 +136,10 @@ def _declare(lib: ctypes.CDLL) -> None:
     lib.cib_moe_table_grouped_supports.restype = _I
     lib.cib_moe_table_grouped_workspace_ints.argtypes = [_I, _I, _I]
     lib.cib_moe_table_grouped_workspace_ints.restype = ctypes.c_longlong
+    lib.cib_ssm_chunk_supports.argtypes = [_I, _I, _I, _I]
+    lib.cib_ssm_chunk_supports.restype = _I
+    lib.cib_lru_mma_supports.argtypes = [_I]
+    lib.cib_lru_mma_supports.restype = _I
     lib.cib_window_attention_mma_supports.argtypes = [_I, _I, _I, _I]
     lib.cib_window_attention_mma_supports.restype = _I
     lib.cib_latent_attention_mma_supports.argtypes = [_I, _I, _I]
@@ -262,6 +274,26 @@ def relu_squared(x: torch.Tensor, out: torch.Tensor) -> None:
         raise KernelError("relu_squared: out does not fit x")
     rc = library().cib_relu_squared(_cuda(x, "x"), _cuda(out, "out"), _code(x, "x"), x.numel(), _stream())
     _check(rc, "relu_squared")
+    _count()
+
+
+def bias_rows(x: torch.Tensor, bias: torch.Tensor, out: torch.Tensor, squared_relu: bool = False) -> None:
+    """out = x + bias (float32 [cols]), or ``max(x + bias, 0) ** 2``; ``out`` may be ``x``."""
+    rows, cols = x.shape
+    if out.shape != x.shape or out.dtype != x.dtype:
+        raise KernelError("bias_rows: out does not fit x")
+    rc = library().cib_bias_rows(_cuda(x, "x"), _f32_vec(bias, cols, "bias"), _cuda(out, "out"), _code(x, "x"), rows, cols,
+                                 1 if squared_relu else 0, _stream())
+    _check(rc, "bias_rows")
+    _count()
+
+
+def pair_sum(a: torch.Tensor, b: torch.Tensor, scale_a: float, scale_b: float, out: torch.Tensor) -> None:
+    """out = scale_a * a + scale_b * b, element by element."""
+    if b.shape != a.shape or out.shape != a.shape or not (a.dtype == b.dtype == out.dtype):
+        raise KernelError("pair_sum: a, b and out must have one shape and dtype")
+    rc = library().cib_pair_sum(_cuda(a, "a"), _cuda(b, "b"), float(scale_a), float(scale_b), _cuda(out, "out"), _code(a, "a"), a.numel(), _stream())
+    _check(rc, "pair_sum")
     _count()
 
 
@@ -733,15 +765,15 @@ MOE_GROUPED_MIN_ROWS = 128
 def moe_table_feed_forward(h: torch.Tensor, ids: torch.Tensor | None, table: torch.Tensor, gate_up: torch.Tensor,
                            down: torch.Tensor, base: torch.Tensor | None, out: torch.Tensor,
                            weights: torch.Tensor | None = None, clamp_limit: float | None = None, activation: str | None = None,
-                           base_gate: torch.Tensor | None = None, base_gate_plain: bool = False) -> None:
+                           base_gate: torch.Tensor | None = None, self_weight: torch.Tensor | None = None) -> None:
     """out[t] = base[t] + (1/top) * sum over k of expert(table[ids[t], k])(h[t]) with gated experts
     (``ids`` None: the table has a row per row of ``h`` — experts chosen by a router; ``weights`` float32 [T, top]:
     a weight per choice instead of 1/top; ``clamp_limit``: the experts' activation is
     ``g * sigmoid(1.702 g) * (u + 1)`` with ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``)
     ``down_e(silu(gate_e h) * up_e h)``; ``gate_up[E, 2 ff, W]`` (gate rows first), ``down[E, W, ff]``, ``table[V, top]``.
     ``activation="relu2"``: experts without a gate, ``down_e(relu(up_e h) ** 2)``, whose first matrix is ``[E, ff, W]``.
-    ``base_gate`` float32 [T] (any stride): ``base[t]`` is multiplied by ``sigmoid(base_gate[t])`` as it is added, or with
-    ``base_gate_plain`` by ``base_gate[t]`` itself.
+    ``base_gate`` float32 [T] (any stride): ``base[t]`` is multiplied by ``sigmoid(base_gate[t])`` as it is added.
+    ``self_weight`` float32 [T]: ``self_weight[t] * h[t]`` is added as well (experts that give back their input).
     Few rows, 32-bit, or sizes that are not multiples of 32: two launches (a matrix-vector product per token and
     choice).  Many bfloat16 rows: grouped by expert (see ``MOE_GROUPED_MIN_ROWS``)."""
     T, W = h.shape
@@ -767,7 +799,9 @@ def moe_table_feed_forward(h: torch.Tensor, ids: torch.Tensor | None, table: tor
         raise KernelError("moe_table: a gate for base needs base and one number per row")
     p_bg = _cuda(base_gate, "base_gate", torch.float32, contiguous=False) if base_gate is not None else None
     bg_stride = base_gate.stride(0) if base_gate is not None else 0
-    bg_plain = 1 if base_gate_plain else 0
+    if self_weight is not None and self_weight.shape != (T,):
+        raise KernelError("moe_table: self_weight must be [rows]")
+    p_self = _cuda(self_weight, "self_weight", torch.float32) if self_weight is not None else None
     lib = library()
     if (h.dtype == torch.bfloat16 and T * top >= MOE_GROUPED_MIN_ROWS and h.stride(0) % 8 == 0
             and lib.cib_moe_table_grouped_supports(W, ff, E)):
@@ -778,7 +812,7 @@ def moe_table_feed_forward(h: torch.Tensor, ids: torch.Tensor | None, table: tor
         rc = lib.cib_moe_table_grouped(
             _cuda(h, "h", contiguous=False), h.stride(0), p_ids, _cuda(table, "table", torch.int32), V, top, E,
             _cuda(gate_up, "gate_up"), _cuda(down, "down"), _cuda(base, "base", contiguous=False) if base is not None else None,
-            base.stride(0) if base is not None else 0, 1.0 / top, p_w, p_bg, bg_stride, bg_plain, _cuda(out, "out"), _cuda(act, "act"), _cuda(y, "y"),
+            base.stride(0) if base is not None else 0, 1.0 / top, p_w, p_bg, bg_stride, p_self, _cuda(out, "out"), _cuda(act, "act"), _cuda(y, "y"),
             _cuda(ints, "ints"), T, W, ff, act_kind, limit, _stream())
         _check(rc, "moe_table_grouped")
         for _ in range(4):
@@ -791,7 +825,8 @@ def moe_table_feed_forward(h: torch.Tensor, ids: torch.Tensor | None, table: tor
     _check(rc, "moe_table_gate_up")
     rc = lib.cib_moe_table_down(_cuda(act, "act"), _code(act, "act"), p_ids, _cuda(table, "table", torch.int32),
                                 V, top, E, _cuda(down, "down"), _cuda(base, "base", contiguous=False) if base is not None else None,
-                                base.stride(0) if base is not None else 0, 1.0 / top, p_w, p_bg, bg_stride, bg_plain, _cuda(out, "out"), T, W, ff, _stream())
+                                base.stride(0) if base is not None else 0, 1.0 / top, p_w, p_bg, bg_stride, _cuda(h, "h", contiguous=False), h.stride(0), p_self,
+                                _cuda(out, "out"), T, W, ff, _stream())
     _check(rc, "moe_table_down")
     _count()
     _count()
@@ -1108,11 +1143,12 @@ def router_topk(logits: torch.Tensor, top: int, choice: torch.Tensor, weight: to
 
 def router_scored_topk(logits: torch.Tensor, top: int, choice: torch.Tensor, weight: torch.Tensor, *,
                        correction: torch.Tensor | None = None, groups: int = 1, keep: int = 1, scale: float = 1.0,
-                       softmax: bool = False, identity_from: int | None = None, identity_weight: torch.Tensor | None = None) -> None:
+                       softmax: bool = False, renorm: bool = False, identity_from: int | None = None,
+                       identity_weight: torch.Tensor | None = None) -> None:
     """From float32 logits [T, E] with scores ``s = sigmoid(logits)`` (``softmax``: the softmax over all E): ``choice`` int32 [T, top], the experts with the
     largest ``s + correction`` (float32 [E], None: no correction; the lower index wins a tie) among the ``keep`` of
     ``groups`` equal groups of neighbouring experts whose two largest ``s + correction`` sum highest; ``weight`` float32
-    [T, top] = ``scale * s`` of the chosen, not renormalised.  ``identity_weight`` float32 [T] gets the sum of a token's
+    [T, top] = ``scale * s`` of the chosen, not renormalised or, with ``renorm``, ``s`` over the sum of the chosen ``s`` (+ 1e-20).  ``identity_weight`` float32 [T] gets the sum of a token's
     weights of chosen experts from index ``identity_from`` on."""
     T, E = logits.shape
     if choice.shape != (T, top) or weight.shape != (T, top) or logits.stride(1) != 1:
@@ -1123,7 +1159,7 @@ def router_scored_topk(logits: torch.Tensor, top: int, choice: torch.Tensor, wei
         raise KernelError("router_scored_topk: identity_weight must be [tokens] and identity_from given")
     rc = library().cib_router_scored_topk(_cuda(logits, "logits", torch.float32, contiguous=False), logits.stride(0), E, top,
                                           _cuda(correction, "correction") if correction is not None else None, int(groups),
-                                          int(keep), float(scale), 1 if softmax else 0, E if identity_from is None else int(identity_from),
+                                          int(keep), float(scale), 1 if softmax else 0, 1 if renorm else 0, E if identity_from is None else int(identity_from),
                                           _cuda(choice, "choice", torch.int32), _cuda(weight, "weight", torch.float32),
                                           _cuda(identity_weight, "identity_weight", torch.float32) if identity_weight is not None else None,
                                           T, _stream())
@@ -1148,7 +1184,8 @@ def window_attention_prep(qkv: torch.Tensor, positions: torch.Tensor, slot_mappi
                           bias: torch.Tensor | None = None, norm: bool = True, q_gain: torch.Tensor | None = None,
                           k_gain: torch.Tensor | None = None, norm_first: bool = False, rot_half: bool = False,
                           q_temp: tuple | None = None, value_from_key: bool = False, rot_gain: float = 1.0, q_only: bool = False,
-                          q_out: torch.Tensor | None = None, conv: "ShortConv | None" = None) -> None:
+                          q_out: torch.Tensor | None = None, conv: "ShortConv | None" = None,
+                          norm_rows: bool = False) -> None:
     """On the packed rows ``[q | k | v]``: ``bias`` (float32, one value per column) is added; rotary encoding of the
     first ``rot_dims`` values of every query and key head (32-bit angle ``pos * freq[i]``; neighbouring pairs, or with
     ``rot_half`` the pairs (i, i + rot_dims / 2)); with ``norm`` every query and key head is divided by its root mean
@@ -1158,7 +1195,8 @@ def window_attention_prep(qkv: torch.Tensor, positions: torch.Tensor, slot_mappi
     its key as it stands before norm and rotation (``vdim == dim``).  ``rot_gain``: a factor on the rotation's cosine and
     sine.  ``q_only``: the rows hold queries only (keys and values are those another layer has cached).  ``conv``: a short
     causal convolution over time of every column (biases included in its input) before anything else, whose state is read
-    and, after this launch or in it, moved on; the queries then go to ``q_out`` [T, H * dim].  Queries are otherwise
+    and, after this launch or in it, moved on; the queries then go to ``q_out`` [T, H * dim].  ``norm_rows``: one root mean square
+    over all of a token's queries (and one over its keys), gains of a value per column.  Queries are otherwise
     rewritten in place; keys and values
     (``(1 - mix) * v + mix * v_first`` when both are given) go to ``cache[page, 0, kv head, slot, dim + vdim]``."""
     T, stride = qkv.shape
@@ -1193,10 +1231,11 @@ def window_attention_prep(qkv: torch.Tensor, positions: torch.Tensor, slot_mappi
         _cuda(mix, "mix") if mix is not None else None, _code(mix, "mix") if mix is not None else 0,
         _cuda(cache, "cache") if cache is not None else None, cache.shape[0] * cache.shape[3] if cache is not None else 0,
         cache.shape[3] if cache is not None else 1, T,
-        _f32_vec(bias, columns, "bias"), _f32_vec(q_gain, dim, "q_gain"), _f32_vec(k_gain, dim, "k_gain"), 1 if norm else 0,
+        _f32_vec(bias, columns, "bias"), _f32_vec(q_gain, num_heads * dim if norm_rows else dim, "q_gain"),
+        _f32_vec(k_gain, num_kv_heads * dim if norm_rows else dim, "k_gain"), 1 if norm else 0,
         1 if norm_first else 0, 1 if rot_half else 0, 1 if q_temp else 0, float(q_temp[0]) if q_temp else 0.0,
         int(q_temp[1]) if q_temp else 1, 1 if value_from_key else 0, float(rot_gain), 1 if q_only else 0,
-        *(conv.arguments() if conv is not None else (None, 0, None, None, None, None, 0, 0)), _stream())
+        *(conv.arguments() if conv is not None else (None, 0, None, None, None, None, 0, 0)), 1 if norm_rows else 0, _stream())
     _check(rc, "window_attention_prep")
     _count()
     if conv is not None and conv.taps.shape[0] > 1 and not conv.one_token_each:
@@ -1482,6 +1521,134 @@ def token_shift(x: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, query_st
         _cuda(query_start_loc, "query_start_loc", torch.int32), _cuda(token_request, "token_request", torch.int32),
         _cuda(state_slots, "state_slots", torch.int32), state.shape[0], _cuda(out, "out"), W, T, _stream())
     _check(rc, "token_shift")
+    _count()
+
+
+# ---- a short convolution of its own, the state-space scan, the gated linear recurrence ------------------------------------------
+
+def short_conv(x: torch.Tensor, conv: ShortConv, out: torch.Tensor, *, in_bias: torch.Tensor | None = None,
+               bias: torch.Tensor | None = None, silu: bool = False) -> None:
+    """``out`` [T, C] = the causal convolution of ``conv`` over the rows ``x[:, :C] + in_bias`` (any row stride), plus
+    ``bias``, then SiLU; biases float32 [C].  Two launches, or one when every request brings one token."""
+    T, C = out.shape
+    conv.check(C)
+    if x.shape[0] != T or x.shape[1] < C or x.stride(1) != 1 or out.stride(1) != 1:
+        raise KernelError("short_conv: rows or out do not fit")
+    taps, K, state, qsl, treq, slots, num_slots, one_each = conv.arguments()
+    rc = library().cib_short_conv(_cuda(x, "x", contiguous=False), _code(x, "x"), x.stride(0), taps, K, _f32_vec(in_bias, C, "in_bias"),
+                                  _f32_vec(bias, C, "bias"), 1 if silu else 0, state, qsl, treq, slots, num_slots,
+                                  _cuda(out, "out", contiguous=False), _code(out, "out"), out.stride(0), C, T, one_each, _stream())
+    _check(rc, "short_conv")
+    _count()
+    if K > 1 and not conv.one_token_each:
+        conv_state_update(x, K, conv.state, conv.query_start_loc, conv.state_slots, C, in_bias)
+
+
+def ssm_chunk_supports(rows: torch.Tensor, num_heads: int, groups: int, vdim: int, state_size: int) -> bool:
+    """Whether the state-space scan runs in chunks on the tensor cores for these rows and sizes."""
+    return (rows.dtype == torch.bfloat16 and rows.stride(0) % 8 == 0 and rows.data_ptr() % 16 == 0
+            and bool(library().cib_ssm_chunk_supports(num_heads, groups, vdim, state_size)))
+
+
+def ssm_scan(rows: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, skip: torch.Tensor, state: torch.Tensor,
+             query_start_loc: torch.Tensor, state_slots: torch.Tensor, out: torch.Tensor, num_heads: int, groups: int, vdim: int,
+             state_size: int, chunks: bool = False) -> None:
+    """The state-space recurrence with a scalar decay per head over every request's rows ``[x (H P) | B (G N) | C (G N)]``:
+    ``S <- exp(-exp(a_log) step) S + step x B^T``, ``out = S C + skip x`` with ``step = softplus(dt + dt_bias)``; ``dt`` float32
+    [T, >= H] (any row stride), ``state`` float32 [slots, H, P * N], ``out`` float32 [T, H * P].  ``chunks``: 64 tokens at a
+    time on the tensor cores (see ``ssm_chunk_supports``); else token after token in 32 bits."""
+    T = out.shape[0]
+    H, G, P, N = num_heads, groups, vdim, state_size
+    if (rows.shape[0] != T or rows.shape[1] < H * P + 2 * G * N or rows.stride(1) != 1 or out.shape != (T, H * P)
+            or state.shape[1:] != (H, P * N)):
+        raise KernelError("ssm_scan: rows, state or out do not fit")
+    if dt.shape[0] != T or dt.shape[1] < H or dt.stride(1) != 1:
+        raise KernelError("ssm_scan: dt does not fit")
+    if len({v.dtype for v in (dt_bias, a_log, skip)}) != 1 or any(v.numel() != H for v in (dt_bias, a_log, skip)):
+        raise KernelError("ssm_scan: dt_bias, a_log and skip have a number per head, in one dtype")
+    rc = library().cib_ssm_scan(
+        _cuda(rows, "rows", contiguous=False), _code(rows, "rows"), rows.stride(0), _cuda(dt, "dt", torch.float32, contiguous=False), dt.stride(0),
+        _cuda(dt_bias, "dt_bias"), _cuda(a_log, "a_log"), _cuda(skip, "skip"), _code(a_log, "a_log"), _cuda(state, "state", torch.float32),
+        _cuda(query_start_loc, "query_start_loc", torch.int32), _cuda(state_slots, "state_slots", torch.int32), state.shape[0],
+        state_slots.numel(), T, _cuda(out, "out", torch.float32), H, G, P, N, 1 if chunks else 0, _stream())
+    _check(rc, "ssm_scan")
+    _count()
+
+
+def gated_group_rms(y: torch.Tensor, z: torch.Tensor, gain: torch.Tensor, eps: float, groups: int, out: torch.Tensor) -> None:
+    """out = the rows ``y * silu(z)`` split into ``groups`` equal parts, each divided by its root mean square, times the gain;
+    ``y`` float32 [T, C], ``z`` rows of any stride."""
+    T, C = y.shape
+    if out.shape != y.shape or z.shape != y.shape or z.stride(1) != 1 or gain.numel() != C or C % groups:
+        raise KernelError("gated_group_rms: shapes do not fit")
+    rc = library().cib_gated_group_rms(_cuda(y, "y", torch.float32), _cuda(z, "z", contiguous=False), _code(z, "z"), z.stride(0),
+                                       _cuda(gain, "gain"), _code(gain, "gain"), float(eps), _cuda(out, "out"), _code(out, "out"), groups,
+                                       C // groups, T, _stream())
+    _check(rc, "gated_group_rms")
+    _count()
+
+
+LRU_DECODE_MAX_BLOCK = 1536       # channels of a block whose rows of eight tokens fit the decode kernel's shared memory
+
+
+def lru_mma_supports(u: torch.Tensor, block: int) -> bool:
+    """Whether the gates of blocks of so many channels are multiplied on the tensor cores."""
+    return (u.dtype == torch.bfloat16 and u.stride(0) % 8 == 0 and u.data_ptr() % 16 == 0 and bool(library().cib_lru_mma_supports(block)))
+
+
+def _lru_vectors(gates: torch.Tensor, u: torch.Tensor, bias: torch.Tensor, sp: torch.Tensor) -> tuple:
+    blocks, two_b, b = gates.shape
+    C = blocks * b
+    if two_b != 2 * b or u.shape[1] < C or u.stride(1) != 1 or gates.dtype != u.dtype:
+        raise KernelError("lru: the gates' matrices must be [blocks, 2 b, b] of the rows' dtype")
+    return C, blocks, _f32_vec(bias, 2 * C, "gate biases"), _f32_vec(sp, C, "softplus(lam)")
+
+
+def lru_gates(u: torch.Tensor, gates: torch.Tensor, bias: torch.Tensor, sp: torch.Tensor, pairs: torch.Tensor,
+              logits: torch.Tensor | None = None) -> None:
+    """``pairs`` float32 [T, C, 2] = decay ``a = exp(-8 r sp)`` (as ``a - 1`` where ``a >= exp(-1/2)``, which is never positive;
+    as ``a`` below) and input ``sqrt(1 - a^2) i u`` of every token and channel, with
+    ``r = sigmoid(Ra u + ra)``, ``i = sigmoid(Ri u + ri)`` block by block; ``gates`` [blocks, 2 b, b] holds a block's Ra then
+    Ri, ``bias`` float32 [2 C] all ra then all ri.  ``logits`` float32 [T, blocks * 2 b]: the products, taken elsewhere."""
+    C, blocks, p_bias, p_sp = _lru_vectors(gates, u, bias, sp)
+    T = u.shape[0]
+    if pairs.shape != (T, C, 2) or (logits is not None and logits.shape != (T, 2 * C)):
+        raise KernelError("lru_gates: pairs or logits do not fit")
+    rc = library().cib_lru_gates(_cuda(u, "u", contiguous=False), _code(u, "u"), u.stride(0), _cuda(gates, "gates"),
+                                 _cuda(logits, "logits", torch.float32) if logits is not None else None, p_bias, p_sp,
+                                 _cuda(pairs, "pairs", torch.float32), C, blocks, T, _stream())
+    _check(rc, "lru_gates")
+    _count()
+
+
+def lru_scan(pairs: torch.Tensor, y: torch.Tensor, y_bias: torch.Tensor, out_scale: float, state: torch.Tensor, query_start_loc: torch.Tensor,
+             state_slots: torch.Tensor, longest: int, out: torch.Tensor) -> None:
+    """``S <- a S + c`` over every request's ``pairs`` (a, c), from and to its slot of ``state`` (float32 [slots, C]); ``out``
+    [T, C] = ``out_scale * S * gelu_tanh(y + y_bias)``.  ``longest``: tokens of the longest request, or a bound."""
+    T, C, _ = pairs.shape
+    if out.shape != (T, C) or y.shape[0] != T or y.shape[1] < C or y.stride(1) != 1 or y.dtype != out.dtype or state.shape[1:] != (C,):
+        raise KernelError("lru_scan: y, state or out do not fit")
+    rc = library().cib_lru_scan(_cuda(pairs, "pairs", torch.float32), _cuda(y, "y", contiguous=False), _code(y, "y"), y.stride(0),
+                                _f32_vec(y_bias, C, "y_bias"), float(out_scale), _cuda(state, "state", torch.float32),
+                                _cuda(query_start_loc, "query_start_loc", torch.int32), _cuda(state_slots, "state_slots", torch.int32),
+                                state.shape[0], state_slots.numel(), int(longest), _cuda(out, "out"), C, T, _stream())
+    _check(rc, "lru_scan")
+    _count()
+
+
+def lru_decode(u: torch.Tensor, gates: torch.Tensor, bias: torch.Tensor, sp: torch.Tensor, y: torch.Tensor, y_bias: torch.Tensor,
+               out_scale: float, state: torch.Tensor, state_slots: torch.Tensor, out: torch.Tensor) -> None:
+    """Gates, recurrence and output of ``lru_gates`` and ``lru_scan`` in one launch, for a step in which row t is request
+    t's single token."""
+    C, blocks, p_bias, p_sp = _lru_vectors(gates, u, bias, sp)
+    T = u.shape[0]
+    if out.shape != (T, C) or y.shape[0] != T or y.shape[1] < C or y.stride(1) != 1 or y.dtype != out.dtype or state.shape[1:] != (C,) or state_slots.numel() != T:
+        raise KernelError("lru_decode: y, state or out do not fit")
+    rc = library().cib_lru_decode(_cuda(u, "u", contiguous=False), _code(u, "u"), u.stride(0), _cuda(gates, "gates"), p_bias, p_sp,
+                                  _cuda(y, "y", contiguous=False), y.stride(0), _f32_vec(y_bias, C, "y_bias"), float(out_scale),
+                                  _cuda(state, "state", torch.float32), _cuda(state_slots, "state_slots", torch.int32), state.shape[0],
+                                  _cuda(out, "out"), C, blocks, T, _stream())
+    _check(rc, "lru_decode")
     _count()
 
 

@@ -116,6 +116,22 @@ class ResidualStream:
             kernels.sandwich_layernorm(self.residual, None, None, self.extra, None, None)
             self.extra = None
 
+    def rows(self, dtype: torch.dtype) -> torch.Tensor:
+        """The stream of every token in ``dtype``, everything outstanding folded in (nothing is pending afterwards): what a
+        sub-layer without a norm on its input reads.  In 32 bits that is the residual itself, good until the next fold."""
+        from .. import kernels
+        if self.residual.dim() != 2:
+            raise RuntimeError("a residual of several streams has no rows of its own")
+        raw = None if dtype == torch.float32 else torch.empty(self.residual.shape, dtype=dtype, device=self.residual.device)
+        if self.pending_norm is not None and self.extra is None and self.writer is None:
+            self.pending_norm.fold(self, raw)
+        else:
+            self.settle()
+            if raw is not None or self.pending is not None:
+                kernels.rms_stream(self.residual, self.pending, None, None, None, raw)
+                self.pending = None
+        return self.residual if raw is None else raw
+
     def spare(self) -> torch.Tensor:
         """A second buffer of the residual's shape, for kernels that write the new residual beside the old."""
         if self._spare is None:
@@ -197,9 +213,10 @@ class Norm(Part):
     def norm_rows(self, rows: torch.Tensor) -> torch.Tensor:
         raise NotImplementedError
 
-    def fold(self, stream: ResidualStream) -> None:
+    def fold(self, stream: ResidualStream, raw: Optional[torch.Tensor] = None) -> None:
         """``stream.residual += self(stream.pending)`` (and ``stream.extra``, if the norm can add it in the same pass);
-        nothing is pending afterwards.  Only a norm that a block uses on a sub-layer's OUTPUT needs this."""
+        nothing is pending afterwards.  Only a norm that a block uses on a sub-layer's OUTPUT needs this.  ``raw``: rows
+        that get the new residual in their own dtype (see ``ResidualStream.rows``)."""
         raise NotImplementedError(f"{type(self).__name__} cannot norm a sub-layer's output")
 
     def fusable_rms(self) -> Optional[tuple]:

@@ -119,3 +119,31 @@ class SandwichBlock(Block):
             h = self.feed_forward_norm.add_norm(stream)
             stream.pending = self.feed_forward.forward(h, ctx)
             stream.pending_norm = self.feed_forward_out_norm
+
+
+@BLOCKS.register("postnorm")
+class PostNormBlock(Block):
+    """``x += norm1(mixer(x)); x += norm2(feed_forward(x))``: norms on the sub-layers' outputs only, which read the stream
+    itself.  Spec: ``PartSpec("postnorm", norm_names=(first, second))``.  A layer whose feed-forward is of kind ``none`` has
+    the first norm only.
+
+    A sub-layer's output stays pending with its norm; the next sub-layer's input (``ResidualStream.rows``) applies the norm,
+    adds, stores the 32-bit residual and rounds it for the products in one kernel."""
+
+    def __init__(self, spec: PartSpec, *, mixer: Mixer, feed_forward: FeedForward,
+                 make_norm: Callable[[str], Norm], prefix: str) -> None:
+        super().__init__(spec, mixer=mixer, feed_forward=feed_forward, make_norm=make_norm, prefix=prefix)
+        first, second = spec.get("norm_names", ("norm1", "norm2"))
+        self.mixer_norm = make_norm(f"{prefix}.{first}")
+        self.has_feed_forward = not getattr(feed_forward, "absent", False)
+        self.feed_forward_norm = make_norm(f"{prefix}.{second}") if self.has_feed_forward else None
+
+    def parts(self) -> List[Part]:
+        return [self.mixer, self.mixer_norm] + ([self.feed_forward, self.feed_forward_norm] if self.has_feed_forward else [])
+
+    def forward(self, stream: ResidualStream, ctx: StepContext, run: int) -> None:
+        stream.pending = self.mixer.forward(stream.rows(self.mixer.dtype), ctx, run)
+        stream.pending_norm = self.mixer_norm
+        if self.has_feed_forward:
+            stream.pending = self.feed_forward.forward(stream.rows(self.feed_forward.dtype), ctx)
+            stream.pending_norm = self.feed_forward_norm

@@ -74,8 +74,9 @@ class NoFeedForward(FeedForward):
 
 @FEED_FORWARDS.register("relu2")
 class SquaredReluFeedForward(FeedForward):
-    """``down( relu(up(x)) ** 2 )``, no gate, no biases.  Spec: ``PartSpec("relu2", intermediate_size=I,
-    names=(up, down))`` with tensor names relative to the part's prefix."""
+    """``down( relu(up(x)) ** 2 )``, no gate; with ``bias`` both products have one (the tensor's name plus
+    ``bias_suffix``), added in 32 bits.  Spec: ``PartSpec("relu2", intermediate_size=I, names=(up, down), bias=False,
+    bias_suffix=".b")`` with tensor names relative to the part's prefix."""
 
     def __init__(self, spec: PartSpec, *, hidden_size: int, prefix: str, dtype: torch.dtype) -> None:
         super().__init__(spec, hidden_size=hidden_size, prefix=prefix, dtype=dtype)
@@ -83,14 +84,21 @@ class SquaredReluFeedForward(FeedForward):
         up, down = spec.get("names", ("up_proj.weight", "down_proj.weight"))
         self.up = Linear([f"{prefix}.{up}"], [self.intermediate_size], hidden_size, dtype)
         self.down = Linear([f"{prefix}.{down}"], [hidden_size], self.intermediate_size, dtype)
+        suffix = spec.get("bias_suffix", ".b")
+        self._bias_specs = [TensorSpec(f"{prefix}.{n}{suffix}", (size,), keep_stored_precision=True, init="zeros")
+                            for n, size in ((up, self.intermediate_size), (down, hidden_size))] if spec.get("bias", False) else []
+        self.up_bias: Optional[torch.Tensor] = None       # 32-bit
+        self.down_bias: Optional[torch.Tensor] = None
 
     def tensors(self) -> List[TensorSpec]:
-        return self.up.tensors() + self.down.tensors()
+        return self.up.tensors() + self.down.tensors() + self._bias_specs
 
     def load(self, store) -> None:
         self.up.load(store)
         self.down.load(store)
         self.up.warm_next = self.down.weight
+        if self._bias_specs:
+            self.up_bias, self.down_bias = (store.get(s).float().contiguous() for s in self._bias_specs)
 
     def first_weight(self) -> Optional[torch.Tensor]:
         return self.up.weight
@@ -103,6 +111,11 @@ class SquaredReluFeedForward(FeedForward):
 
     def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
         y = self.up.forward(x)
+        if self.up_bias is not None:
+            kernels.bias_rows(y, self.up_bias, y, squared_relu=True)
+            out = self.down.forward(y)
+            kernels.bias_rows(out, self.down_bias, out)
+            return out
         act = torch.empty_like(y)
         kernels.relu_squared(y, act)
         return self.down.forward(act)
@@ -205,7 +218,7 @@ class RoutedExperts(FeedForward):
       tensor ``correction_name``; None: no correction) among the ``groups = (count, keep)`` best groups — the experts form
       ``count`` equal groups of neighbours, a group's mark is the sum of its two largest choice scores, and only experts
       of the ``keep`` best groups can be chosen; the weights are the chosen experts' ``s`` times ``route_scale``, not
-      renormalised;
+      renormalised or, with ``renorm``, over the sum of the chosen ``s`` (+ 1e-20);
     * ``"softmax"``: the same with ``s`` the softmax over all logits.
 
     ``identity`` n > 0 (with a scored choice): the router has n more rows, whose experts have no matrices and give back
@@ -220,7 +233,7 @@ class RoutedExperts(FeedForward):
     token and is added, multiplied by ``sigmoid(g . h)`` when ``shared_gate_name`` names a row ``[1, W]``.
 
     Spec: ``PartSpec("moe_routed", experts=E, top=k, intermediate_size=I, activation, limit, score, correction_name, groups,
-    route_scale, identity=0, router_name="router", expert_names=("e{}.gate", "e{}.up", "e{}.down"), shared_size, shared_names,
+    route_scale, renorm=False, identity=0, router_name="router", expert_names=("e{}.gate", "e{}.up", "e{}.down"), shared_size, shared_names,
     shared_gate_name)``.  The experts' matrices are stacked at load as for the table-routed mixture, whose kernels run
     the experts here too (rows by token and choice for few rows, grouped by expert on the tensor cores for many)."""
 
@@ -246,13 +259,14 @@ class RoutedExperts(FeedForward):
         groups = spec.get("groups") or (1, 1)
         self.groups, self.keep = int(groups[0]), int(groups[1])
         self.route_scale = float(spec.get("route_scale", 1.0))
+        self.renorm = bool(spec.get("renorm", False))
         if self.score != "softmax_chosen":
             if self.groups <= 0 or routes % self.groups or not 0 < self.keep <= self.groups:
                 raise ValueError(f"moe_routed: {self.groups} groups ({self.keep} kept) of {routes} experts")
             if self.keep * (routes // self.groups) < self.top:
                 raise ValueError(f"moe_routed: {self.keep} groups of {routes // self.groups} experts cannot give {self.top}")
-        elif (self.groups, self.keep) != (1, 1) or spec.get("correction_name") or self.route_scale != 1.0:
-            raise ValueError("moe_routed: groups, a correction and a scale belong to a scored choice")
+        elif (self.groups, self.keep) != (1, 1) or spec.get("correction_name") or self.route_scale != 1.0 or self.renorm:
+            raise ValueError("moe_routed: groups, a correction, a scale and weights over their sum belong to a scored choice")
         p = prefix
         names = spec.get("expert_names", ("e{}.gate", "e{}.up", "e{}.down") if self.gated else ("e{}.up", "e{}.down"))
         if len(names) != (3 if self.gated else 2):
@@ -279,8 +293,6 @@ class RoutedExperts(FeedForward):
             self.shared_down = Linear([f"{p}.{shared[-1]}"], [hidden_size], self.shared_size, dtype)
             if self.activation == "clamped":
                 raise ValueError("moe_routed: a shared expert with the clamped gate is not built")
-            if self.identity:
-                raise ValueError("moe_routed: identity experts beside a shared expert are not built")
         self.gate_up: Optional[torch.Tensor] = None
         self.down: Optional[torch.Tensor] = None
         self.correction: Optional[torch.Tensor] = None
@@ -333,14 +345,14 @@ class RoutedExperts(FeedForward):
         kept = torch.empty(T, dtype=torch.float32, device=x.device) if self.identity else None
         if self.score != "softmax_chosen":
             kernels.router_scored_topk(logits, self.top, choice, weight, correction=self.correction, groups=self.groups,
-                                       keep=self.keep, scale=self.route_scale, softmax=self.score == "softmax",
+                                       keep=self.keep, scale=self.route_scale, softmax=self.score == "softmax", renorm=self.renorm,
                                        identity_from=self.experts if self.identity else None, identity_weight=kept)
         else:
             kernels.router_topk(logits, self.top, choice, weight)
-        base = self._shared(x) if self.shared_size else x if self.identity else None
-        base_gate = routed[:, self.experts] if self.has_shared_gate else kept
+        base = self._shared(x) if self.shared_size else None
+        base_gate = routed[:, self.experts + self.identity] if self.has_shared_gate else None
         out = torch.empty((T, self.hidden_size), dtype=x.dtype, device=x.device)
         kernels.moe_table_feed_forward(x, None, choice, self.gate_up, self.down, base, out, weights=weight,
                                        clamp_limit=self.limit, activation="relu2" if self.activation == "relu2" else None,
-                                       base_gate=base_gate, base_gate_plain=bool(self.identity))
+                                       base_gate=base_gate, self_weight=kept)
         return out

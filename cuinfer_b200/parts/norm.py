@@ -65,10 +65,10 @@ class RMSNorm(Norm):
         stream.pending = None
         return out
 
-    def fold(self, stream: ResidualStream) -> None:
+    def fold(self, stream: ResidualStream, raw=None) -> None:
         if self.groups > 1:
             raise NotImplementedError("rmsnorm: a norm in groups on a sub-layer's output is not built")
-        kernels.rms_stream(stream.residual, stream.pending, (self.weight, self.eps), None, None)
+        kernels.rms_stream(stream.residual, stream.pending, (self.weight, self.eps), None, None, raw)
         stream.pending = stream.pending_norm = None
 
     def norm_rows(self, rows: torch.Tensor) -> torch.Tensor:
@@ -128,9 +128,11 @@ class LayerNorm(Norm):
         stream.pending = stream.pending_norm = stream.extra = None
         return out
 
-    def fold(self, stream: ResidualStream) -> None:
+    def fold(self, stream: ResidualStream, raw=None) -> None:
         kernels.sandwich_layernorm(stream.residual, stream.pending, self._triple(), stream.extra, None, None)
         stream.pending = stream.pending_norm = stream.extra = None
+        if raw is not None:
+            kernels.rms_stream(stream.residual, None, None, None, None, raw)
 
     def norm_rows(self, rows: torch.Tensor) -> torch.Tensor:
         out = torch.empty(rows.shape, dtype=self.dtype, device=rows.device)

@@ -1,4 +1,5 @@
-"""Mixers that carry a matrix per head from token to token instead of a cache of keys, and a pair of mixers side by side.
+"""Mixers that carry a state (a matrix per head, or a number per channel) from token to token instead of a cache of keys,
+and a pair of mixers side by side.
 
 The recurrent ones keep their state in 32 bits in the request's state slot (zero when the request is admitted), read it at the start
 of a step and write it back at the end, so a prompt may be cut anywhere.  What enters the recurrence besides the
@@ -39,8 +40,28 @@ row h and the row h' of the token before (zeros before a sequence's first), mix_
 then each head's o divided by its root mean square, times a gain over all heads, times the gate, then ``Wo``.  The previous
 h is state too.  Spec: ``PartSpec("wkv", num_heads, dim, eps, rank, names={...})``.
 
-``side_by_side`` — two mixers on the same input: ``(rms(left) * left.out + rms(right) * right.out) / 2``, norms of whole rows.
-Spec: ``PartSpec("side_by_side", left=PartSpec(...), right=PartSpec(...), eps, names={"left": "left", "right": "right",
+``state_space`` — the state-space recurrence with a scalar decay per head (Mamba-2).  One projection ``W_in h`` gives
+``[z (H P) | x (H P) | B (G N) | C (G N) | dt (H)]``; x, B and C pass a short causal convolution per channel (with a bias;
+its last ``taps - 1`` inputs are state too) and SiLU; ``dt = softplus(dt + dt_bias)``; head i uses B and C of group
+``i // (H / G)``::
+
+    S <- exp(-exp(A_log) dt) S + dt x B^T;  y = S C + D x
+
+then ``y * silu(z)``, each of ``norm_groups`` equal parts over its own root mean square, times a gain, then ``Wo``.  Spec:
+``PartSpec("state_space", num_heads, vdim, state_size, groups, taps, norm_groups, eps, names={...})``.
+
+``gated_linear`` — a linear recurrence with one number of state per channel (Griffin's block with the RG-LRU).  Two branches
+of ``width`` channels with biases: ``y = gelu_tanh(Wy h + by)`` and ``u = conv(Wx h + bx)``, a short causal convolution per
+channel with a bias; u in ``blocks`` equal parts, each with two square matrices: ``r = sigmoid(Ra u + ra)``,
+``i = sigmoid(Ri u + ri)``::
+
+    a = exp(-8 r softplus(lam));  S <- a S + sqrt(1 - a^2) i u
+
+then ``Wo (out_scale * S * y)``.  Spec: ``PartSpec("gated_linear", width, blocks, taps, out_scale=1.0, names={...})``.
+
+``side_by_side`` — two mixers on the same input.  Without ``scales``: ``(rms(left) * left.out + rms(right) * right.out) / 2``,
+norms of whole rows; with ``scales = (a, b)``: ``a * left + b * right``.
+Spec: ``PartSpec("side_by_side", left=PartSpec(...), right=PartSpec(...), eps, scales=None, names={"left": "left", "right": "right",
 "out": "out"})``: the mixers' tensors lie under ``left`` and ``right``, the norms' gains are ``left.out`` and ``right.out``.  One of
 the two may keep a paged cache; both may keep state.
 """
@@ -54,12 +75,14 @@ import torch
 from .. import kernels
 from .base import Mixer
 from .context import StepContext
-from .linear import Linear, dense_operand, per_head_products
+from .linear import Linear, dense_operand, padded_rows, per_head_products
 from .registry import MIXERS
 from .spec import PartSpec, StateNeed, TensorSpec
 
 MLSTM_FLOOR = 1e-6          # added to the read-out's denominator
 DELTA_UNIT_EPS = 1e-6       # inside the root of the unit norm of queries and keys
+FEW_ROWS = 16               # rows up to which the state-space mixer's projections are one product in 32 bits
+LRU_DECODE_MAX_ROWS = 64    # rows up to which a step of single tokens takes the gated linear recurrence in one launch
 
 
 def _names(spec: PartSpec, defaults: Dict[str, str]) -> Dict[str, str]:
@@ -352,11 +375,169 @@ class TimeMixing(Mixer):
         return self.o.forward(out)
 
 
+@MIXERS.register("state_space")
+class StateSpace(Mixer):
+    def __init__(self, spec: PartSpec, *, hidden_size: int, prefix: str, dtype: torch.dtype) -> None:
+        super().__init__(spec, hidden_size=hidden_size, prefix=prefix, dtype=dtype)
+        self.num_heads, self.vdim, self.state_size = int(spec.num_heads), int(spec.vdim), int(spec.state_size)
+        self.groups, self.taps, self.norm_groups = int(spec.groups), int(spec.taps), int(spec.get("norm_groups", 1))
+        self.eps = float(spec.get("eps", 1e-6))
+        if min(self.num_heads, self.vdim, self.state_size, self.groups, self.taps, self.norm_groups) <= 0 or self.num_heads % self.groups:
+            raise ValueError("state_space: sizes must be positive and num_heads a multiple of groups")
+        if self.state_size > 256:
+            raise ValueError(f"state_space: state size {self.state_size} is beyond what the scan kernels keep in registers (256)")
+        self.inner = self.num_heads * self.vdim
+        if self.inner % self.norm_groups:
+            raise ValueError(f"state_space: {self.inner} values do not split into {self.norm_groups} groups")
+        n = _names(spec, {"in": "in", "conv": "conv", "conv_bias": "conv.b", "dt_bias": "dt_bias", "A_log": "A_log", "D": "D", "norm": "norm",
+                          "o": "o"})
+        p, H = prefix, self.num_heads
+        self.channels = self.inner + 2 * self.groups * self.state_size
+        # one matrix [z | x | B | C | dt].  Steps of many rows multiply its two parts apart, so that the step sizes come out in
+        # 32 bits beside rows in the engine's dtype; steps of few rows take all of it in 32 bits at once
+        self.all = Linear([f"{p}.{n['in']}"], [self.inner + self.channels + H], hidden_size, dtype, pad=True)
+        self.main = Linear([f"{p}.{n['in']}"], [self.inner + self.channels], hidden_size, dtype)
+        self.steps = Linear([f"{p}.{n['in']}"], [H], hidden_size, dtype)
+        self.o = Linear([f"{p}.{n['o']}"], [hidden_size], self.inner, dtype)
+        self._tap_spec = TensorSpec(f"{p}.{n['conv']}", (self.channels, self.taps))
+        self._conv_bias_spec = TensorSpec(f"{p}.{n['conv_bias']}", (self.channels,), keep_stored_precision=True, init="zeros")
+        self._vec_specs = [TensorSpec(f"{p}.{n[v]}", (H,), keep_stored_precision=True, init="ones" if v == "D" else "zeros")
+                           for v in ("dt_bias", "A_log", "D")]
+        self._gain_spec = TensorSpec(f"{p}.{n['norm']}", (self.inner,), keep_stored_precision=True, init="ones")
+        self.conv_taps = self.conv_bias = self.dt_bias = self.a_log = self.skip = self.gain = None
+
+    def tensors(self) -> List[TensorSpec]:
+        return self.all.tensors() + self.o.tensors() + [self._tap_spec, self._conv_bias_spec, *self._vec_specs, self._gain_spec]
+
+    def load(self, store) -> None:
+        self.all.load(store)
+        self.o.load(store)
+        rows = self.inner + self.channels
+        self.main.weight = self.all.weight[:rows]
+        self.steps.weight = padded_rows(self.all.weight[rows:rows + self.num_heads].clone())
+        self.conv_taps = store.get(self._tap_spec).float().t().contiguous()
+        self.conv_bias = store.get(self._conv_bias_spec).float().contiguous()
+        self.dt_bias, self.a_log, self.skip = (store.get(s).float().contiguous() for s in self._vec_specs)
+        self.gain = store.get(self._gain_spec)
+
+    def first_weight(self) -> Optional[torch.Tensor]:
+        return self.all.weight
+
+    def warm_after(self, weight: Optional[torch.Tensor]) -> None:
+        self.o.warm_next = weight
+
+    def state_need(self):
+        return (StateNeed((self.num_heads, self.vdim * self.state_size), "float32", name="memory"),
+                StateNeed((max(self.taps - 1, 1), self.channels), "float32", name="conv"))
+
+    def workspace_bytes(self, tokens: int) -> int:
+        width = 2 if self.dtype == torch.bfloat16 else 4
+        return (self.main.workspace_bytes(tokens) + tokens * (self.num_heads + 8) * 4 + tokens * self.channels * width
+                + tokens * self.inner * (4 + width) + self.o.workspace_bytes(tokens))
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, run: int) -> torch.Tensor:
+        H, G, P, N, T = self.num_heads, self.groups, self.vdim, self.state_size, x.shape[0]
+        state = ctx.run_state(run)
+        if T <= FEW_ROWS or self.dtype == torch.float32:
+            rows = self.all.forward(x, out_dtype=torch.float32)
+            dt = rows[:, self.inner + self.channels:]
+        else:
+            rows = self.main.forward(x)
+            dt = self.steps.forward(x, out_dtype=torch.float32)
+        xbc = torch.empty((T, self.channels), dtype=self.dtype, device=x.device)
+        conv = kernels.ShortConv(self.conv_taps, state["conv"], ctx.query_start_loc, ctx.token_request, ctx.state_slots,
+                                 one_token_each=ctx.decode_only)
+        kernels.short_conv(rows[:, self.inner:], conv, xbc, bias=self.conv_bias, silu=True)
+        y = torch.empty((T, self.inner), dtype=torch.float32, device=x.device)
+        kernels.ssm_scan(xbc, dt, self.dt_bias, self.a_log, self.skip, state["memory"], ctx.query_start_loc, ctx.state_slots, y, H, G, P, N,
+                         chunks=not ctx.decode_only and kernels.ssm_chunk_supports(xbc, H, G, P, N))
+        out = torch.empty((T, self.inner), dtype=self.dtype, device=x.device)
+        kernels.gated_group_rms(y, rows[:, :self.inner], self.gain, self.eps, self.norm_groups, out)
+        return self.o.forward(out)
+
+
+@MIXERS.register("gated_linear")
+class GatedLinear(Mixer):
+    def __init__(self, spec: PartSpec, *, hidden_size: int, prefix: str, dtype: torch.dtype) -> None:
+        super().__init__(spec, hidden_size=hidden_size, prefix=prefix, dtype=dtype)
+        self.width, self.blocks, self.taps = int(spec.width), int(spec.blocks), int(spec.taps)
+        self.out_scale = float(spec.get("out_scale", 1.0))
+        if min(self.width, self.blocks, self.taps) <= 0 or self.width % self.blocks:
+            raise ValueError("gated_linear: sizes must be positive and width a multiple of blocks")
+        self.block = self.width // self.blocks
+        n = _names(spec, {"y": "y", "x": "x", "y_bias": "y.b", "x_bias": "x.b", "conv": "conv", "conv_bias": "conv.b", "ra": "ra", "ri": "ri",
+                          "ra_bias": "ra.b", "ri_bias": "ri.b", "lam": "lam", "o": "o"})
+        p, C, b = prefix, self.width, self.block
+        self.main = Linear([f"{p}.{n['y']}", f"{p}.{n['x']}"], [C, C], hidden_size, dtype)
+        self.o = Linear([f"{p}.{n['o']}"], [hidden_size], C, dtype)
+        self._gate_specs = [TensorSpec(f"{p}.{n[r]}", (self.blocks, b, b)) for r in ("ra", "ri")]
+        self._gate_bias_specs = [TensorSpec(f"{p}.{n[r]}", (self.blocks, b), keep_stored_precision=True, init="zeros")
+                                 for r in ("ra_bias", "ri_bias")]
+        self._tap_spec = TensorSpec(f"{p}.{n['conv']}", (C, self.taps))
+        self._vec_specs = [TensorSpec(f"{p}.{n[v]}", (C,), keep_stored_precision=True, init="zeros")
+                           for v in ("y_bias", "x_bias", "conv_bias", "lam")]
+        self.gates: Optional[torch.Tensor] = None             # [blocks, 2 b, b]: a block's Ra, then its Ri
+        self.gate_bias: Optional[torch.Tensor] = None         # 32-bit [2 C]
+        self.conv_taps = self.y_bias = self.x_bias = self.conv_bias = None
+        self.rate: Optional[torch.Tensor] = None              # softplus(lam), 32-bit [C]
+
+    def tensors(self) -> List[TensorSpec]:
+        return self.main.tensors() + self.o.tensors() + self._gate_specs + self._gate_bias_specs + [self._tap_spec] + self._vec_specs
+
+    def load(self, store) -> None:
+        self.main.load(store)
+        self.o.load(store)
+        self.gates = torch.cat([store.get(s) for s in self._gate_specs], dim=1).to(self.dtype).contiguous()
+        self.gate_bias = torch.cat([store.get(s).float().reshape(-1) for s in self._gate_bias_specs]).contiguous()
+        self.conv_taps = store.get(self._tap_spec).float().t().contiguous()
+        self.y_bias, self.x_bias, self.conv_bias, lam = (store.get(s).float().contiguous() for s in self._vec_specs)
+        self.rate = torch.nn.functional.softplus(lam.double()).float().contiguous()
+
+    def first_weight(self) -> Optional[torch.Tensor]:
+        return self.main.weight
+
+    def warm_after(self, weight: Optional[torch.Tensor]) -> None:
+        self.o.warm_next = weight
+
+    def state_need(self):
+        return (StateNeed((self.width,), "float32", name="memory"),
+                StateNeed((max(self.taps - 1, 1), self.width), "float32", name="conv"))
+
+    def workspace_bytes(self, tokens: int) -> int:
+        width = 2 if self.dtype == torch.bfloat16 else 4
+        return (self.main.workspace_bytes(tokens) + tokens * self.width * (2 * width + 8) + tokens * self.width * 8
+                + self.o.workspace_bytes(tokens))
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, run: int) -> torch.Tensor:
+        C, b, T = self.width, self.block, x.shape[0]
+        state = ctx.run_state(run)
+        rows = self.main.forward(x)
+        u = torch.empty((T, C), dtype=self.dtype, device=x.device)
+        conv = kernels.ShortConv(self.conv_taps, state["conv"], ctx.query_start_loc, ctx.token_request, ctx.state_slots,
+                                 one_token_each=ctx.decode_only)
+        kernels.short_conv(rows[:, C:], conv, u, in_bias=self.x_bias, bias=self.conv_bias)
+        out = torch.empty((T, C), dtype=self.dtype, device=x.device)
+        if ctx.decode_only and T <= LRU_DECODE_MAX_ROWS and b <= kernels.LRU_DECODE_MAX_BLOCK:
+            kernels.lru_decode(u, self.gates, self.gate_bias, self.rate, rows, self.y_bias, self.out_scale, state["memory"], ctx.state_slots, out)
+            return self.o.forward(out)
+        pairs = torch.empty((T, C, 2), dtype=torch.float32, device=x.device)
+        if kernels.lru_mma_supports(u, b):
+            kernels.lru_gates(u, self.gates, self.gate_bias, self.rate, pairs)
+        else:
+            logits = torch.empty((T, 2 * C), dtype=torch.float32, device=x.device)
+            per_head_products(u.view(T, self.blocks, b).transpose(0, 1), self.gates, logits.view(T, self.blocks, 2 * b).transpose(0, 1))
+            kernels.lru_gates(u, self.gates, self.gate_bias, self.rate, pairs, logits=logits)
+        kernels.lru_scan(pairs, rows, self.y_bias, self.out_scale, state["memory"], ctx.query_start_loc, ctx.state_slots, ctx.max_query_len, out)
+        return self.o.forward(out)
+
+
 @MIXERS.register("side_by_side")
 class SideBySide(Mixer):
     def __init__(self, spec: PartSpec, *, hidden_size: int, prefix: str, dtype: torch.dtype) -> None:
         super().__init__(spec, hidden_size=hidden_size, prefix=prefix, dtype=dtype)
         self.eps = float(spec.get("eps", 1e-6))
+        scales = spec.get("scales")
+        self.scales = (float(scales[0]), float(scales[1])) if scales is not None else None
         n = _names(spec, {"left": "left", "right": "right", "out": "out"})
         self.sides: Dict[str, Mixer] = {}
         for side in ("left", "right"):
@@ -366,7 +547,7 @@ class SideBySide(Mixer):
             raise ValueError("side_by_side: one of the two mixers may keep a paged cache")
         self.capturable = all(m.capturable for m in self.sides.values())
         self._gain_specs = [TensorSpec(f"{prefix}.{n[side]}.{n['out']}", (hidden_size,), keep_stored_precision=True, init="ones")
-                            for side in ("left", "right")]
+                            for side in ("left", "right")] if self.scales is None else []
         self.gains: Optional[List[torch.Tensor]] = None
 
     def tensors(self) -> List[TensorSpec]:
@@ -376,7 +557,7 @@ class SideBySide(Mixer):
         for m in self.sides.values():
             m.load(store)
         self.gains = [store.get(s) for s in self._gain_specs]
-        if self.gains[0].dtype != self.gains[1].dtype:
+        if self.gains and self.gains[0].dtype != self.gains[1].dtype:
             self.gains = [g.float() for g in self.gains]
 
     def first_weight(self) -> Optional[torch.Tensor]:
@@ -415,5 +596,8 @@ class SideBySide(Mixer):
     def forward(self, x: torch.Tensor, ctx: StepContext, run: int) -> torch.Tensor:
         left, right = (self.sides[side].forward(x, self._context(side, ctx, run), run) for side in ("left", "right"))
         out = torch.empty_like(left)
+        if self.scales is not None:
+            kernels.pair_sum(left, right, self.scales[0], self.scales[1], out)
+            return out
         kernels.pair_rms_mean(left, right, self.gains[0], self.gains[1], self.eps, out)
         return out

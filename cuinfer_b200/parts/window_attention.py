@@ -15,8 +15,9 @@ and key size ``dim``, value size ``vdim``:
 * ``own_kv`` False: the layer has no keys and values of its own (nor their biases and convolutions); it reads those that
   an earlier layer of the same head counts, sizes and rotation has cached (``ModelSpec.cache_source`` names it);
 * ``qk_norm``: ``"unit"`` divides each head of q and k by its root mean square over ``dim`` (``eps`` inside the root),
-  ``"gain"`` also multiplies by a gain of ``dim`` values shared by all heads (one for q, one for k), ``"none"`` leaves
-  them; the norm comes after the position encoding or, with ``norm_first``, before it;
+  ``"gain"`` also multiplies by a gain of ``dim`` values shared by all heads (one for q, one for k), ``"row"`` divides
+  all of a token's queries by their common root mean square (and its keys by theirs) and multiplies by a gain per
+  column, ``"none"`` leaves them; the norm comes after the position encoding or, with ``norm_first``, before it;
 * the position encoding (rotary, on the first ``rotary_dim`` values of each head; ``rope_interleaved`` pairs
   neighbours, ``rope_half`` pairs i with ``i + rotary_dim / 2``) on q and k;
 * ``q_temp = (coef, every)``: the query at position p is multiplied by ``1 + coef * ln(floor((p + 1) / every) + 1)``;
@@ -82,8 +83,8 @@ class WindowAttention(Mixer):
             raise ValueError("window_attention: a mask of chunks keeps no first tokens")
         self.eps = float(spec.get("eps", 1e-6))
         self.qk_norm = spec.get("qk_norm") or ("unit" if spec.get("qk_unit_norm", True) else "none")
-        if self.qk_norm not in ("unit", "gain", "none"):
-            raise ValueError(f"window_attention: qk_norm must be 'unit', 'gain' or 'none', got {self.qk_norm!r}")
+        if self.qk_norm not in ("unit", "gain", "row", "none"):
+            raise ValueError(f"window_attention: qk_norm must be 'unit', 'gain', 'row' or 'none', got {self.qk_norm!r}")
         self.norm_first = bool(spec.get("norm_first", False))
         self.has_bias = bool(spec.get("bias", False))
         temp = spec.get("q_temp")
@@ -116,6 +117,8 @@ class WindowAttention(Mixer):
             raise ValueError(f"window_attention: gate must be None, 'value' or 'head', got {self.gate!r}")
         if self.conv < 0 or (self.conv and (self.value_mix or self.value_from_key)):
             raise ValueError("window_attention: a convolution beside mixed values or values taken from keys is not built")
+        if self.qk_norm == "row" and (self.conv or self.value_mix or self.value_from_key or not self.own_kv):
+            raise ValueError("window_attention: a norm over whole rows beside a convolution, shared keys, mixed values or values taken from keys is not built")
         if not self.own_kv and (self.value_mix or self.value_from_key):
             raise ValueError("window_attention: a layer that reads another's keys and values has no values to mix")
         pos_spec: PartSpec = spec.get("position") or PartSpec("none")
@@ -150,6 +153,9 @@ class WindowAttention(Mixer):
                            for n in spec.get("log_bias_names", ("r1", "r2"))] if self.has_log_bias else []
         self._gain_specs = [TensorSpec(f"{p}.{n}", (self.dim,), keep_stored_precision=True, init="ones")
                             for n in (q_norm, k_norm)] if self.qk_norm == "gain" else []
+        if self.qk_norm == "row":
+            self._gain_specs = [TensorSpec(f"{p}.{n}", (size,), keep_stored_precision=True, init="ones")
+                                for n, size in ((q_norm, self.q_size), (k_norm, self.k_size))]
         self._sink_spec = TensorSpec(f"{p}.{sink}", (self.num_heads,), keep_stored_precision=True, init="zeros") if self.sink == "learned" else None
         self.bias: Optional[torch.Tensor] = None          # 32-bit [q | k | v] biases
         self.q_gain: Optional[torch.Tensor] = None
@@ -236,7 +242,7 @@ class WindowAttention(Mixer):
                                       bias=self.bias, norm=self.qk_norm != "none", q_gain=self.q_gain, k_gain=self.k_gain,
                                       norm_first=self.norm_first, rot_half=getattr(self.position, "layout", "") == "half",
                                       q_temp=self.q_temp, value_from_key=self.value_from_key, rot_gain=self.rot_gain,
-                                      q_only=not self.own_kv, q_out=q if self.conv else None, conv=conv)
+                                      q_only=not self.own_kv, q_out=q if self.conv else None, conv=conv, norm_rows=self.qk_norm == "row")
         out = torch.empty((qkv.shape[0], self.num_heads * self.vdim), dtype=qkv.dtype, device=qkv.device)
         gate = qkv[:, self.columns:self.columns + self._gate_size] if self.gate else None
         attention_dispatch.window_attention(q, out, kv, ctx, self.num_heads, self.num_kv_heads, self.dim, self.vdim,

@@ -419,7 +419,7 @@ def test_experts_that_give_back_their_input(dtype, W, ff, E, identity, top, T):
             want[t] += float(weights[t, k]) * (plain.gated_ff(h[t:t + 1], gate[e], up[e], down[e])[0] if e < E else h[t])
     out = torch.empty(T, W, dtype=dtype, device="cuda")
     kernels.moe_table_feed_forward(_dev(h, dtype), None, choice.cuda(), _dev(torch.cat([gate, up], 1), dtype), _dev(down, dtype),
-                                   _dev(h, dtype), out, weights=weights.cuda(), base_gate=kept.cuda(), base_gate_plain=True)
+                                   None, out, weights=weights.cuda(), self_weight=kept.cuda())
     _close(out, want, dtype, "experts beside identity experts", tol=3e-5 if dtype == torch.float32 else 3e-2)
 
 
