@@ -198,3 +198,104 @@ def greedy(config: dict, weights: Dict[str, torch.Tensor], prompt, steps: int) -
         out.append(nxt)
         toks.append(nxt)
     return out
+
+
+# ---- how safe the routers' choices are ------------------------------------------------------------------------------------
+def choice_margins(scores, top: int):
+    """For rows of choice scores [N, E]: how far the last chosen lies above the first rejected, per row."""
+    if top >= scores.shape[1]:
+        return torch.full((scores.shape[0],), math.inf, dtype=scores.dtype)
+    ranked = scores.sort(-1, descending=True).values
+    return ranked[:, top - 1] - ranked[:, top]
+
+
+# ---- random weights for the tests -------------------------------------------------------------------------------------------
+def random_model(config: dict, seed: int, dtype=torch.float32) -> Dict[str, torch.Tensor]:
+    """Weights whose values are bfloat16 numbers.  The routers are made robust against rounding, so that a bfloat16
+    engine and this implementation choose the same experts: the first columns of the embedding carry, per token id, the
+    router's logits (a router's row e reads column e, plus a little of everything else), drawn again until every layer's
+    choice has a safe margin; the norms' gains are zero in those columns, so nothing is ever added there."""
+    g = torch.Generator().manual_seed(seed)
+    W, V = config["width"], config["vocab"]
+    own = [(i, L) for i, L in enumerate(config["layers"]) if L.get("weights_of") is None]
+    mixtures = [(i, L["mlp"]) for i, L in own if L.get("mlp") and L["mlp"]["kind"] == "moe"]
+    routes = {i: f["router"]["experts"] + int(f["router"].get("identity") or 0) for i, f in mixtures}
+    E_max = max(list(routes.values()) + [0])
+    assert E_max <= W // 2
+
+    def mat(o, i, gain=1.0):
+        return (torch.randn(o, i, generator=g) * gain / math.sqrt(i)).bfloat16().to(dtype)
+
+    def vec(n, around=0.0, spread=0.1):
+        return (around + spread * torch.randn(n, generator=g)).bfloat16().to(dtype)
+
+    def taps(n, K):
+        return (torch.randn(n, K, generator=g) * 0.6).bfloat16().to(dtype)
+
+    def out_gain():
+        v = vec(W, 0.5)
+        v[:E_max] = 0.0
+        return v
+
+    t: Dict[str, torch.Tensor] = {"final.norm": vec(W, 1.0)}
+    corrections = {}
+    for i, f in mixtures:
+        corrections[i] = (0.1 * torch.randn(routes[i], generator=g)).bfloat16().double()
+        t[f"l{i}.mlp.correction"] = corrections[i].to(dtype)
+    embed = torch.randn(V, W, generator=g)
+    if E_max:
+        accepted = torch.zeros(0, E_max, dtype=torch.float64)
+        for _ in range(400):
+            if len(accepted) >= V:
+                break
+            cand = ((torch.rand(4096, E_max, generator=g) * 2 - 1) * 1.5).bfloat16().double()
+            for i, f in mixtures:
+                cand = cand[choice_margins(torch.softmax(2.0 * cand[:, :routes[i]], -1) + corrections[i], f["router"]["top"]) > 0.02]
+            accepted = torch.cat([accepted, cand])
+        assert len(accepted) >= V, "no safe logits found for some token ids"
+        embed[:, :E_max] = accepted[:V].float()
+    t["embed"] = embed.bfloat16().to(dtype)
+    for i, L in own:
+        p, m = f"l{i}.", L["mixer"]
+        t[p + "norm1"] = out_gain()
+        q = p + "mix."
+        if L["type"] == "mamba2":
+            H, P, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
+            inner = H * P
+            C = inner + 2 * G * N
+            t[q + "in"] = mat(inner + C + H, W, 1.5)
+            t[q + "conv"], t[q + "conv.b"] = taps(C, m["conv"]), vec(C, 0.0, 0.3)
+            t[q + "dt_bias"], t[q + "A_log"], t[q + "D"] = vec(H, -2.0, 1.0), vec(H, -1.0, 1.5), vec(H, 0.7, 0.4)
+            t[q + "norm"], t[q + "o"] = vec(inner, 1.0), mat(W, inner)
+        else:
+            a, b = m["left"], m["right"]
+            H, G, d, dv = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            t[q + "left.q"], t[q + "left.k"], t[q + "left.v"] = mat(H * d, W), mat(G * d, W), mat(G * dv, W)
+            t[q + "left.q.norm"], t[q + "left.k.norm"], t[q + "left.o"] = vec(H * d, 1.3, 0.3), vec(G * d, 1.3, 0.3), mat(W, H * dv)
+            n, K, blocks = b["width"], b["conv"], b["blocks"]
+            q += "right."
+            t[q + "y"], t[q + "y.b"], t[q + "x"], t[q + "x.b"] = mat(n, W), vec(n, 0.0, 0.5), mat(n, W), vec(n, 0.0, 0.5)
+            t[q + "conv"], t[q + "conv.b"], t[q + "lam"], t[q + "o"] = taps(n, K), vec(n, 0.0, 0.3), vec(n, -2.0, 2.0), mat(W, n)
+            size = n // blocks
+            for r in ("ra", "ri"):
+                t[q + r] = (torch.randn(blocks, size, size, generator=g) * 1.5 / math.sqrt(size)).bfloat16().to(dtype)
+                t[q + r + ".b"] = vec(n, 0.0, 0.7).view(blocks, size)
+        f = L.get("mlp")
+        if not f:
+            continue
+        t[p + "norm2"] = out_gain()
+        q = p + "mlp."
+        if f["kind"] == "dense":
+            t[q + "up"], t[q + "up.b"], t[q + "down"], t[q + "down.b"] = mat(f["ff"], W), vec(f["ff"], 0.0, 0.3), mat(W, f["ff"]), vec(W, 0.0, 0.5)
+            continue
+        sizes = {f"e{e}": f["expert"]["ff"] for e in range(f["router"]["experts"])}
+        if f.get("shared"):
+            sizes["shared"] = f["shared"]["ff"]
+        for name, ff in sizes.items():
+            t[f"{q}{name}.gate"], t[f"{q}{name}.up"], t[f"{q}{name}.down"] = mat(ff, W), mat(ff, W), mat(W, ff)
+        router = torch.randn(routes[i], W, generator=g) * 0.004 / math.sqrt(W)
+        router[:, :E_max] = 0.0
+        for e in range(routes[i]):
+            router[e, e] = 2.0
+        t[q + "router"] = router.bfloat16().to(dtype)
+    return t
