@@ -1,4 +1,4 @@
-"""Bilolorn, Kusolorn, Desilorn, Zinunex and Nugolorn beside the Qwen3 dense decoder at equal layer sizes: prefill and decode throughput
+"""Bilolorn, Kusolorn, Desilorn, Zinunex, Nugolorn and Neburax beside the Qwen3 dense decoder at equal layer sizes: prefill and decode throughput
 through the model runner, and the time of every kernel of a step with the share of its roofline that it reaches.
 
 ``bench.py --designs`` runs this (``--design-names kusolorn,qwen3`` chooses the designs; ``kusolorn_attention`` is
@@ -137,6 +137,23 @@ def nugolorn_config(s: dict) -> dict:
             "residual_mult": 0.5, "logit_scale": 0.5, "layers": layers}
 
 
+def neburax_config(s: dict) -> dict:
+    """Four layers: three of the state-space recurrence (twice the width in heads of 64, a state of 128) and one pair of chunked
+    attention (the Qwen3 arm's head counts and head size, chunks as long as Kusolorn's window) and the gated linear
+    recurrence (as wide as the model, blocks of 256); a dense feed-forward first and experts of Kusolorn's sizes, of which an
+    eighth more give back their input, with a shared one after it."""
+    ssm = {"heads": 2 * s["width"] // 64, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1}
+    pair = {"left": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["head_dim"], "vdim": s["head_dim"], "scale": s["head_dim"] ** -0.5,
+                     "mask": {"size": s["window"]}},
+            "right": {"width": s["width"], "blocks": s["width"] // 256, "conv": 4}, "left_scale": 1.1, "right_scale": 0.9}
+    dense = {"kind": "dense", "ff": s["ff"]}
+    moe = {"kind": "moe", "router": {"experts": s["experts"], "top": s["top"], "identity": s["experts"] // 8}, "expert": {"ff": s["expert_ff"]},
+           "shared": {"ff": s["shared_ff"]}}
+    kinds = [("mamba2", ssm, dense), ("mamba2", ssm, moe), ("parallel", pair, moe), ("mamba2", ssm, moe)]
+    layers = [{"type": t, "mixer": m, "mlp": f} for t, m, f in (kinds * ((s["layers"] + 3) // 4))[:s["layers"]]]
+    return {"architecture": "Neburax", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "layers": layers}
+
+
 def qwen3_config(s: dict) -> dict:
     return dict(architectures=["Qwen3ForCausalLM"], num_hidden_layers=s["layers"], hidden_size=s["width"],
                 num_attention_heads=s["heads"], num_key_value_heads=s["kv_heads"], head_dim=s["head_dim"],
@@ -158,7 +175,13 @@ def make_runner(config: dict, pages: int, max_seqs: int, graphs: bool):
     from .weights import write_random_model
 
     folder = tempfile.mkdtemp(prefix="cuinfer_b200_designs_")
-    write_random_model(folder, config, 7, std=0.02, gain_std=0.02, dtype="bfloat16", generator="counter", materialize=False)
+    # A router's corrections stay small beside its scores: drawn like the gains they would send every token to the same
+    # experts.  A design whose sub-layers read the stream itself gets an embedding of unit size, or the convolutions' biases
+    # would outweigh the tokens.
+    gains = {".correction": 0.01}
+    if config.get("architecture") == "Neburax":
+        gains["embed"] = 50.0
+    write_random_model(folder, config, 7, std=0.02, gain_std=0.02, dtype="bfloat16", generator="counter", materialize=False, gains=gains)
     cfg = EngineConfig(model_path=folder, block_size=16, dtype="bfloat16", num_blocks=pages, max_num_seqs=max_seqs,
                        max_num_scheduled_tokens=1 << 20, enable_cuda_graph=graphs)
     return ModelRunner(folder, cfg)
@@ -264,6 +287,14 @@ class KernelTimes:
             "token_shift": lambda x, mu, state, qsl, tr, slots, out: (0.0, _nbytes(x, out, mu)),
             "channel_delta_scan": lambda qkv, beta, decay, al, db, state, qsl, slots, out, G, H, d, dv, **k: scan(out.shape[0], H, d, dv, 7, state),
             "wkv_scan": lambda r, k, v, decay, w0, u, state, qsl, slots, out, H, d, dv, **kw: scan(out.shape[0], H, d, dv, 5, state),
+            "bias_rows": rowwise, "pair_sum": rowwise, "gated_group_rms": rowwise,
+            "short_conv": lambda x, conv, out, **k: (0.0, _nbytes(out) + out.numel() * x.element_size()),
+            "ssm_scan": lambda rows, dt, db, al, sk, state, qsl, slots, out, H, G, P, N, **k:
+                (5.0 * out.shape[0] * H * P * N, _nbytes(rows, out) + out.shape[0] * H * 4 + 2 * _nbytes(state) * len(lq) // max(1, state.shape[0])),
+            "lru_gates": lambda u, gates, bias, sp, pairs, **k: (4.0 * u.shape[0] * gates.shape[0] * gates.shape[2] ** 2, _nbytes(u, gates, pairs)),
+            "lru_scan": lambda pairs, y, yb, sc, state, qsl, slots, longest, out: (0.0, _nbytes(pairs) + 2 * _nbytes(out)),
+            "lru_decode": lambda u, gates, bias, sp, y, yb, sc, state, slots, out:
+                (4.0 * u.shape[0] * gates.shape[0] * gates.shape[2] ** 2, _nbytes(gates) + 3 * _nbytes(out) + 8 * out.numel()),
             "latent_prep": lambda proj, q_off, rq, kv_off, rk, dr, *a, **k: (0.0, proj.shape[0] * (2 * rq + 2 * (rk + dr)) * 2),
             "qk_norm_rope_kv_write": lambda qkv, *a, **k: (0.0, 2 * _nbytes(qkv)),
             "latent_attention_mma": lambda q_abs, q, out, cache, bt, qsl, sl, ql, freq, rd, sinks, H, dn, rk, dr, *a, **k:
@@ -316,7 +347,7 @@ def measure(design: str, size: str, prefill_tokens: int, batch: int, context: in
 
     s = SIZES[size]
     config = {"bilolorn": bilolorn_config, "kusolorn": kusolorn_config, "kusolorn_attention": kusolorn_attention_config,
-              "desilorn": desilorn_config, "zinunex": zinunex_config, "nugolorn": nugolorn_config, "qwen3": qwen3_config}[design](s)
+              "desilorn": desilorn_config, "zinunex": zinunex_config, "nugolorn": nugolorn_config, "neburax": neburax_config, "qwen3": qwen3_config}[design](s)
     pages = (batch * (context + steps + 64) + prefill_tokens) // 16 + 64
     runner = make_runner(config, pages, max_seqs=max(batch, 8), graphs=True)
     gen = torch.Generator().manual_seed(5)

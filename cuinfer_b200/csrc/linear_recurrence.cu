@@ -49,12 +49,19 @@ lru_gates_mma_kernel(const __nv_bfloat16* __restrict__ u, int u_stride, const __
                      const float* __restrict__ sp, float2* __restrict__ pairs, int C, int b, int num_tokens) {
     __shared__ __align__(16) __nv_bfloat16 sA[kLStages][kLM][kLLd];
     __shared__ __align__(16) __nv_bfloat16 sB[kLStages][2][kLN][kLLd];
+    __shared__ __align__(8) float s_bias[2][kLN], s_sp[kLN];       // of this tile's channels
     griddep_launch();
     griddep_wait();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int tiles = (b + kLN - 1) / kLN;
     const int block = blockIdx.y / tiles, n0 = (blockIdx.y % tiles) * kLN, m0 = blockIdx.x * kLM;
     const int rows = min(kLM, num_tokens - m0);
+    if (tid < kLN) {
+        const int c = block * b + min(n0 + tid, b - 1);
+        s_bias[0][tid] = bias[c];
+        s_bias[1][tid] = bias[C + c];
+        s_sp[tid] = sp[c];
+    }
     const __nv_bfloat16* wb = w + (size_t)block * 2 * b * b;
     const __nv_bfloat16* a = u + (size_t)m0 * u_stride + (size_t)block * b;
     auto load = [&](int stage, int k0) {
@@ -111,16 +118,21 @@ lru_gates_mma_kernel(const __nv_bfloat16* __restrict__ u, int u_stride, const __
         const int row = warp * 16 + qrow + 8 * half;
         if (row >= rows) continue;
         const size_t t = (size_t)(m0 + row);
+        const __nv_bfloat16* ur = u + t * u_stride + (size_t)block * b + n0;
+        float4* dst = reinterpret_cast<float4*>(pairs + t * C + (size_t)block * b + n0);
+        __nv_bfloat162 uv[kLN / 8];                      // all of the row's inputs are on their way before the first is used
+#pragma unroll
+        for (int j = 0; j < kLN / 8; ++j)
+            if (n0 + j * 8 < b) uv[j] = *reinterpret_cast<const __nv_bfloat162*>(ur + j * 8 + quad * 2);
 #pragma unroll
         for (int j = 0; j < kLN / 8; ++j) {
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int col = n0 + j * 8 + quad * 2 + e;
-                if (col >= b) continue;
-                const int c = block * b + col;
-                pairs[t * C + c] = lru_pair(acc[0][j][2 * half + e] + bias[c], acc[1][j][2 * half + e] + bias[C + c],
-                                            __bfloat162float(u[t * u_stride + c]), sp[c]);
-            }
+            const int col = j * 8 + quad * 2;            // b is a multiple of 32: a pair of columns is inside or outside
+            if (n0 + col >= b) continue;
+            const float2 br = *reinterpret_cast<const float2*>(&s_bias[0][col]), bi = *reinterpret_cast<const float2*>(&s_bias[1][col]);
+            const float2 rate = *reinterpret_cast<const float2*>(&s_sp[col]);
+            const float2 p = lru_pair(acc[0][j][2 * half] + br.x, acc[1][j][2 * half] + bi.x, __low2float(uv[j]), rate.x);
+            const float2 q = lru_pair(acc[0][j][2 * half + 1] + br.y, acc[1][j][2 * half + 1] + bi.y, __high2float(uv[j]), rate.y);
+            dst[col / 2] = make_float4(p.x, p.y, q.x, q.y);
         }
     }
 }
@@ -194,9 +206,11 @@ lru_scan_kernel(const float2* __restrict__ pairs, const T* __restrict__ y, int y
     if (end == t1 && st) *st = S;                        // every warp has read the state before the exchange
 }
 
-constexpr int kLruTokens = 8, kLruDecodeWarps = 8, kLruPerWarp = 2;
+constexpr int kLruTokens = 8, kLruDecodeWarps = 8;
 
-// One token per request (token t is request t's).  grid (blocks, channel tiles of a block).
+// One token per request (token t is request t's).  grid (blocks, channel tiles of a block): a warp a channel.  The sixteen sums
+// of a channel over eight tokens are reduced by halves: at every step a lane gives one half of its sums away and adds to
+// the other, so that lane l ends with sum l / 2.
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(kLruDecodeWarps * 32)
 lru_decode_kernel(const T* __restrict__ u, int u_stride, const T* __restrict__ w, const float* __restrict__ bias, const float* __restrict__ sp,
@@ -205,72 +219,87 @@ lru_decode_kernel(const T* __restrict__ u, int u_stride, const T* __restrict__ w
     extern __shared__ __align__(16) float us[];          // [kLruTokens][b]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int block = blockIdx.x;
-    const T* wb = w + (size_t)block * 2 * b * b;
+    const int col = blockIdx.y * kLruDecodeWarps + warp, c = block * b + min(col, b - 1);
+    const T* wr = w + (size_t)block * 2 * b * b + (size_t)min(col, b - 1) * b;
+    const T* wi = wr + (size_t)b * b;
     griddep_launch();
+    // weights: not written by the kernel before this one
+    uint4 first_r = make_uint4(0, 0, 0, 0), first_i = first_r;
+    if (VEC && lane * 8 < b) {
+        first_r = *reinterpret_cast<const uint4*>(wr + lane * 8);
+        first_i = *reinterpret_cast<const uint4*>(wi + lane * 8);
+    }
+    const float br = bias[c], bi = bias[C + c], rate = sp[c], yb = y_bias[c];
     griddep_wait();
     for (int tb = 0; tb < num_tokens; tb += kLruTokens) {
         const int count = min(kLruTokens, num_tokens - tb);
+        // lane 4 tt takes token tt: what it needs is on its way before the products
+        const int mine = tb + (lane >> 2);
+        const bool finish = (lane & 3) == 0 && mine < num_tokens && col < b;
+        float* st = nullptr;
+        float before = 0.f, gate = 0.f;
+        if (finish) {
+            const int slot = state_slots[mine];
+            st = slot >= 0 && slot < num_slots ? state + (size_t)slot * C + c : nullptr;
+            before = st ? *st : 0.f;
+            gate = to_f32(y[(size_t)mine * y_stride + c]);
+        }
         __syncthreads();
         for (int idx = threadIdx.x; idx < kLruTokens * b; idx += blockDim.x) {
             const int tt = idx / b, k = idx - tt * b;
             us[idx] = tt < count ? to_f32(u[(size_t)(tb + tt) * u_stride + (size_t)block * b + k]) : 0.f;
         }
         __syncthreads();
-        for (int q = 0; q < kLruPerWarp; ++q) {
-            const int col = (blockIdx.y * kLruDecodeWarps + warp) * kLruPerWarp + q;
-            if (col >= b) continue;                      // a whole warp; the barriers lie outside
-            float zr[kLruTokens], zi[kLruTokens];
+        float v[2 * kLruTokens];                         // [token][Ra, Ri]
 #pragma unroll
-            for (int tt = 0; tt < kLruTokens; ++tt) zr[tt] = zi[tt] = 0.f;
-            const T* wr = wb + (size_t)col * b;
-            const T* wi = wb + (size_t)(b + col) * b;
-            if constexpr (VEC) {                         // bfloat16, b a multiple of 8: 16 bytes of each row a lane
-                for (int k = lane * 8; k < b; k += 256) {
-                    const uint4 vr = *reinterpret_cast<const uint4*>(wr + k), vi = *reinterpret_cast<const uint4*>(wi + k);
-                    const __nv_bfloat162* hr = reinterpret_cast<const __nv_bfloat162*>(&vr);
-                    const __nv_bfloat162* hi = reinterpret_cast<const __nv_bfloat162*>(&vi);
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        const float2 fr = __bfloat1622float2(hr[e]), fi = __bfloat1622float2(hi[e]);
-#pragma unroll
-                        for (int tt = 0; tt < kLruTokens; ++tt) {
-                            const float2 x = *reinterpret_cast<const float2*>(us + tt * b + k + 2 * e);
-                            zr[tt] = fmaf(fr.x, x.x, fmaf(fr.y, x.y, zr[tt]));
-                            zi[tt] = fmaf(fi.x, x.x, fmaf(fi.y, x.y, zi[tt]));
-                        }
-                    }
+        for (int i = 0; i < 2 * kLruTokens; ++i) v[i] = 0.f;
+        if constexpr (VEC) {                             // bfloat16, b a multiple of 8: 16 bytes of each row a lane
+            for (int k = lane * 8; k < b; k += 256) {
+                uint4 vr = first_r, vi = first_i;
+                if (k >= 256) {
+                    vr = *reinterpret_cast<const uint4*>(wr + k);
+                    vi = *reinterpret_cast<const uint4*>(wi + k);
                 }
-            } else {
-                for (int k = lane; k < b; k += 32) {
-                    const float fr = to_f32(wr[k]), fi = to_f32(wi[k]);
+                const __nv_bfloat162* hr = reinterpret_cast<const __nv_bfloat162*>(&vr);
+                const __nv_bfloat162* hi = reinterpret_cast<const __nv_bfloat162*>(&vi);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float2 fr = __bfloat1622float2(hr[e]), fi = __bfloat1622float2(hi[e]);
 #pragma unroll
                     for (int tt = 0; tt < kLruTokens; ++tt) {
-                        const float x = us[tt * b + k];
-                        zr[tt] = fmaf(fr, x, zr[tt]);
-                        zi[tt] = fmaf(fi, x, zi[tt]);
+                        const float2 x = *reinterpret_cast<const float2*>(us + tt * b + k + 2 * e);
+                        v[2 * tt] = fmaf(fr.x, x.x, fmaf(fr.y, x.y, v[2 * tt]));
+                        v[2 * tt + 1] = fmaf(fi.x, x.x, fmaf(fi.y, x.y, v[2 * tt + 1]));
                     }
                 }
             }
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1)
+        } else {
+            for (int k = lane; k < b; k += 32) {
+                const float fr = to_f32(wr[k]), fi = to_f32(wi[k]);
 #pragma unroll
                 for (int tt = 0; tt < kLruTokens; ++tt) {
-                    zr[tt] += __shfl_xor_sync(0xffffffffu, zr[tt], o);
-                    zi[tt] += __shfl_xor_sync(0xffffffffu, zi[tt], o);
+                    const float x = us[tt * b + k];
+                    v[2 * tt] = fmaf(fr, x, v[2 * tt]);
+                    v[2 * tt + 1] = fmaf(fi, x, v[2 * tt + 1]);
                 }
-            float mr = 0.f, mi = 0.f;                    // lane tt takes token tt
-#pragma unroll
-            for (int tt = 0; tt < kLruTokens; ++tt)
-                if (lane == tt) { mr = zr[tt]; mi = zi[tt]; }
-            if (lane < count) {
-                const int t = tb + lane, c = block * b + col;
-                const int slot = state_slots[t];
-                float* st = slot >= 0 && slot < num_slots ? state + (size_t)slot * C + c : nullptr;
-                const float2 p = lru_pair(mr + bias[c], mi + bias[C + c], us[lane * b + col], sp[c]);
-                const float S = lru_apply(p.x, st ? *st : 0.f, p.y);
-                if (st) *st = S;
-                out[(size_t)t * C + c] = from_f32<T>(out_scale * S * gelu_tanhf_(to_f32(y[(size_t)t * y_stride + c]) + y_bias[c]));
             }
+        }
+#pragma unroll
+        for (int half = kLruTokens, o = 16; half >= 1; half >>= 1, o >>= 1) {
+            const bool upper = (lane & o) != 0;
+#pragma unroll
+            for (int i = 0; i < half; ++i) {
+                const float give = upper ? v[i] : v[i + half], keep = upper ? v[i + half] : v[i];
+                v[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+            }
+        }
+        v[0] += __shfl_xor_sync(0xffffffffu, v[0], 1);   // lane l: sum l / 2, that is token l / 4, Ra (even) or Ri (odd)
+        const float zi = __shfl_down_sync(0xffffffffu, v[0], 2);
+        if (finish) {
+            const float2 p = lru_pair(v[0] + br, zi + bi, us[(lane >> 2) * b + col], rate);
+            const float S = lru_apply(p.x, before, p.y);
+            if (st) *st = S;
+            out[(size_t)mine * C + c] = from_f32<T>(out_scale * S * gelu_tanhf_(gate + yb));
         }
     }
 }
@@ -333,7 +362,7 @@ extern "C" int cib_lru_decode(const void* u, int dtype, int u_stride, const void
                               void* out, int C, int blocks, int num_tokens, cudaStream_t stream) {
     CIB_REQUIRE(C > 0 && blocks > 0 && C % blocks == 0 && u_stride >= C && y_stride >= C && num_tokens >= 0, "lru_decode: bad sizes");
     if (num_tokens == 0) return 0;
-    const int b = C / blocks, per = kLruDecodeWarps * kLruPerWarp;
+    const int b = C / blocks, per = kLruDecodeWarps;
     const size_t smem = (size_t)kLruTokens * b * sizeof(float);
     CIB_REQUIRE(smem <= 48 * 1024, "lru_decode: blocks of %d channels are beyond this kernel", b);
     const dim3 grid(blocks, (b + per - 1) / per);

@@ -83,7 +83,7 @@ router_scored_topk_kernel(const float* __restrict__ logits, int stride, int expe
         z_inv = 1.f / warp_sum(sum);
     }
     auto score = [&](int e) { return softmax ? expf(z[e] - z_max) * z_inv : 1.f / (1.f + expf(-z[e])); };
-    float identity = 0.f;
+    float identity = 0.f, total = 0.f;
     for (int e = lane; e < experts; e += 32) {
         const float s = score(e);
         float c = s + (correction ? correction[e] : 0.f);
@@ -142,16 +142,15 @@ router_scored_topk_kernel(const float* __restrict__ logits, int stride, int expe
             choice[(size_t)t * top + k] = at;
             const float w = at >= 0 ? scale * score(at) : 0.f;
             weight[(size_t)t * top + k] = w;
+            total += w;
             if (at >= identity_from) identity += w;
             if (at >= 0) cs[at] = -INFINITY;
         }
         __syncwarp();
     }
-    if (renorm && lane == 0) {                                    // the lane that has written the weights
-        float sum = 0.f;
-        for (int k = 0; k < top; ++k) sum += weight[(size_t)t * top + k];
-        const float inv = scale / (sum + scale * 1e-20f);
-        for (int k = 0; k < top; ++k) weight[(size_t)t * top + k] *= inv;
+    if (renorm) {                                                 // after the loop's last __syncwarp every weight is in place
+        const float inv = scale / (__shfl_sync(0xffffffffu, total, 0) + scale * 1e-20f);
+        for (int k = lane; k < top; k += 32) weight[(size_t)t * top + k] *= inv;
         identity *= inv;
     }
     if (identity_weight && lane == 0) identity_weight[t] = identity;

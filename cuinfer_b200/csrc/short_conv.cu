@@ -5,7 +5,7 @@
 // Requests, slots and the order of tokens as in recurrent.cu.  Inputs before a step's rows come from the request's state
 // ([K - 1][C], oldest first, input bias included); before the start of a sequence they are zero (the state of a new
 // request is).  A thread walks a few consecutive tokens of V neighbouring channels with the last inputs in registers,
-// so that a row is read once; at a request's first row the registers are filled from its state.  With
+// so that a row is read once (a step of few tokens gives every token a thread of its own); at a request's first row the registers are filled from its state.  With
 // `one_token_each` the thread that reads a request's state also moves it on; otherwise `conv_state_update_kernel`
 // (recurrent.cu) does that after this launch.  Sums and activation 32-bit, one rounding at the end.
 #include <algorithm>
@@ -14,7 +14,8 @@
 
 namespace cib {
 
-constexpr int kConvTokens = 8;           // tokens a thread walks
+constexpr int kConvTokens = 8;           // tokens a thread walks (one in a step of few tokens)
+constexpr int kConvFewTokens = 256;
 constexpr int kConvMaxTaps = 16;
 
 template <typename T, int V> __device__ __forceinline__ void load_row(const T* p, float (&v)[V]) {
@@ -41,14 +42,14 @@ template <> __device__ __forceinline__ void store_row<__nv_bfloat16, 4>(__nv_bfl
     *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
 }
 
-// KT: taps held in registers, K <= KT (a tap beyond K is zero).
-template <typename TI, typename TO, int V, int KT>
+// KT: taps held in registers, K <= KT (a tap beyond K is zero); TB: tokens a thread walks.
+template <typename TI, typename TO, int V, int KT, int TB>
 __global__ void __launch_bounds__(128)
 short_conv_kernel(const TI* __restrict__ x, int stride, const float* __restrict__ taps, int K, const float* __restrict__ in_bias,
                   const float* __restrict__ bias, int silu, float* __restrict__ state, const int* __restrict__ query_start_loc,
                   const int* __restrict__ token_request, const int* __restrict__ state_slots, int num_slots, TO* __restrict__ out,
                   int out_stride, int C, int num_tokens, int one_token_each) {
-    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+    const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
     griddep_launch();
     if (c >= C) return;
     float w[KT][V], ib[V], ob[V];                     // weights: not written by the kernel before this one
@@ -62,7 +63,34 @@ short_conv_kernel(const TI* __restrict__ x, int stride, const float* __restrict_
         ob[k] = bias ? bias[c + k] : 0.f;
     }
     griddep_wait();
-    const int t0 = blockIdx.y * kConvTokens, t1 = min(num_tokens, t0 + kConvTokens);
+    const int t0 = blockIdx.x * TB, t1 = min(num_tokens, t0 + TB);
+    if constexpr (TB > 1) {
+        // all of the tokens and what precedes them in one request: every row is asked for before the first is used
+        const int r = token_request[t0];
+        if (t1 == t0 + TB && t0 - (KT - 1) >= query_start_loc[r] && t1 <= query_start_loc[r + 1]) {
+            float u[TB + KT - 1][V];
+#pragma unroll
+            for (int i = 0; i < TB + KT - 1; ++i) load_row<TI, V>(x + (size_t)(t0 - (KT - 1) + i) * stride + c, u[i]);
+#pragma unroll
+            for (int i = 0; i < TB + KT - 1; ++i)
+#pragma unroll
+                for (int k = 0; k < V; ++k) u[i][k] += ib[k];
+#pragma unroll
+            for (int i = 0; i < TB; ++i) {
+                float y[V];
+#pragma unroll
+                for (int k = 0; k < V; ++k) {
+                    float s = 0.f;
+#pragma unroll
+                    for (int j = 0; j < KT; ++j) s = fmaf(w[j][k], u[i + KT - 1 - j][k], s);
+                    s += ob[k];
+                    y[k] = silu ? s / (1.f + expf(-s)) : s;
+                }
+                store_row<TO, V>(out + (size_t)(t0 + i) * out_stride + c, y);
+            }
+            return;
+        }
+    }
     float win[KT][V];                                 // win[j]: the input j tokens back
     for (int t = t0; t < t1; ++t) {
         const int r = token_request[t];
@@ -127,16 +155,19 @@ extern "C" int cib_short_conv(const void* x, int dtype, int stride, const float*
     const bool v4 = C % 4 == 0 && stride % 4 == 0 && out_stride % 4 == 0 && (uintptr_t)x % in_bytes == 0 && (uintptr_t)out % out_bytes == 0 &&
                     (uintptr_t)state % 16 == 0;
     const int per = v4 ? 4 : 1;
-    const dim3 grid((unsigned)((C / per + 127) / 128 + (C % per ? 1 : 0)), (unsigned)((num_tokens + kConvTokens - 1) / kConvTokens));
+    const int walk = num_tokens <= kConvFewTokens || K > 4 ? 1 : kConvTokens;
+    const dim3 grid((unsigned)((num_tokens + walk - 1) / walk), (unsigned)((C / per + 127) / 128));
+    CIB_REQUIRE(grid.y <= 65535, "short_conv: %d channels are beyond this kernel", C);
     const bool pdl = prompt_pdl();
     cudaError_t e = cudaErrorInvalidValue;
-#define CIB_CONV(TI, TO, V, KT)                                                                                                       \
-    e = launch_pdl(short_conv_kernel<TI, TO, V, KT>, grid, dim3(128), 0, stream, pdl, (const TI*)x, stride, taps, K, in_bias, bias, silu,  \
+#define CIB_CONV(TI, TO, V, KT, TB)                                                                                                   \
+    e = launch_pdl(short_conv_kernel<TI, TO, V, KT, TB>, grid, dim3(128), 0, stream, pdl, (const TI*)x, stride, taps, K, in_bias, bias, silu,  \
                    state, query_start_loc, token_request, state_slots, num_slots, (TO*)out, out_stride, C, num_tokens, one_token_each)
 #define CIB_CONV_K(TI, TO, V)                       \
     do {                                            \
-        if (K <= 4) CIB_CONV(TI, TO, V, 4);         \
-        else CIB_CONV(TI, TO, V, kConvMaxTaps);     \
+        if (walk > 1) CIB_CONV(TI, TO, V, 4, kConvTokens);      \
+        else if (K <= 4) CIB_CONV(TI, TO, V, 4, 1);             \
+        else CIB_CONV(TI, TO, V, kConvMaxTaps, 1);              \
     } while (0)
 #define CIB_CONV_V(TI, TO)                          \
     do {                                            \

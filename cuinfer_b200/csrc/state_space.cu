@@ -102,6 +102,8 @@ ssm_walk_kernel(const T* __restrict__ rows, int stride, const float* __restrict_
 // ---- chunks of 64 tokens on the tensor cores -----------------------------------------------------------------------------
 constexpr int kChunk = 64;
 constexpr int kChunkLd = kChunk + 8;
+constexpr int kChunkRows = 64;                   // rows of S a CTA owns: sixteen a consumer warp
+constexpr int kChunkThreads = 256;
 
 __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint32_t& lo) {
     hi = pack_bf16(a, b);
@@ -109,75 +111,92 @@ __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint3
     lo = pack_bf16(a - __low2float(h), b - __high2float(h));
 }
 
-template <int NP, int NW> constexpr size_t ssm_chunk_smem() {
-    constexpr int PT = NW * 16;
-    return (size_t)2 * (2 * kChunk * (NP + 8) + kChunk * (PT + 8)) * 2      // two stages of C, B, x
-           + (size_t)2 * kChunk * (PT + 8) * 2                              // weighted x, value and remainder
-           + (size_t)2 * kChunk * kChunkLd * 2                              // the weights of a chunk's pairs, likewise
-           + (size_t)4 * kChunk * 4;                                        // L, dt, exp(L), weights of the update
+template <int NP> constexpr int ssm_stages() { return NP <= 128 ? 3 : 2; }
+template <int NP> constexpr size_t ssm_chunk_smem() {
+    return (size_t)ssm_stages<NP>() * (2 * kChunk * (NP + 8) + kChunk * (kChunkRows + 8)) * 2      // C, B, x of a chunk
+           + (size_t)2 * 2 * kChunk * (kChunkRows + 8) * 2                  // two chunks' weighted x, value and remainder
+           + (size_t)2 * 2 * kChunk * kChunkLd * 2                          // two chunks' weights of pairs, likewise
+           + (size_t)3 * 4 * kChunk * 4;                                    // three chunks' L, dt, exp(L), weights of the update
 }
 
-// A CTA of NW warps walks the chunks of one request for 16 NW rows of one head's S; each warp owns 16 rows, and
-// 64 / NW rows of the chunk's pairs.
-template <int NP, int NW>
-__global__ void __launch_bounds__(NW * 32)
+// A CTA walks the chunks of one request for 64 rows of one head's S.  Only the state links one chunk to the next, so the
+// warps divide: four producers make the next chunk's weighted x and pair weights (16 tokens each, and the first of them
+// the step sizes of the chunk after it), four consumers take the current chunk's products with S, 16 rows of it each.
+// One barrier a chunk.
+template <int NP>
+__global__ void __launch_bounds__(kChunkThreads)
 ssm_chunk_kernel(const __nv_bfloat16* __restrict__ rows, int stride, const float* __restrict__ z, int z_stride, AnyVec dt_bias, AnyVec a_log,
                  AnyVec skip, float* __restrict__ state, const int* __restrict__ query_start_loc, const int* __restrict__ state_slots,
                  int num_slots, float* __restrict__ out, int H, int G, int P, int N) {
-    constexpr int PT = NW * 16, LDN = NP + 8, LDP = PT + 8, MT = 4 / NW;
+    constexpr int PT = kChunkRows, LDN = NP + 8, LDP = PT + 8, STAGES = ssm_stages<NP>();
     constexpr int kStage = 2 * kChunk * LDN + kChunk * LDP;
     extern __shared__ __align__(16) unsigned char ssm_raw[];
     __nv_bfloat16* stages = reinterpret_cast<__nv_bfloat16*>(ssm_raw);
-    __nv_bfloat16* xw_hi = stages + 2 * kStage;
-    __nv_bfloat16* xw_lo = xw_hi + kChunk * LDP;
-    __nv_bfloat16* w_hi = xw_lo + kChunk * LDP;
-    __nv_bfloat16* w_lo = w_hi + kChunk * kChunkLd;
-    float* Ls = reinterpret_cast<float*>(w_lo + kChunk * kChunkLd);
-    float* dts = Ls + kChunk;
-    float* eL = dts + kChunk;
-    float* wu = eL + kChunk;
+    __nv_bfloat16* xw = stages + STAGES * kStage;               // [2 chunks][value, remainder][kChunk][LDP]
+    __nv_bfloat16* pw = xw + 4 * kChunk * LDP;                  // [2 chunks][value, remainder][kChunk][kChunkLd]
+    float* steps = reinterpret_cast<float*>(pw + 4 * kChunk * kChunkLd);      // [3 chunks][L, dt, exp(L), update][kChunk]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const bool producer = warp >= 4;
     const int r = blockIdx.z, h = blockIdx.x, p_base = blockIdx.y * PT;
     const int t0 = query_start_loc[r], t1 = query_start_loc[r + 1];
     if (t1 <= t0) return;
+    const int chunks = (t1 - t0 + kChunk - 1) / kChunk;
     const int slot = state_slots[r];
     const bool has = slot >= 0 && slot < num_slots;
     const int qrow = lane >> 2, quad = lane & 3, mat = lane >> 3, rr = lane & 7;
-    const int p_lo = p_base + warp * 16 + qrow, p_hi = p_lo + 8;
     const float a = -expf(a_log[h]), bias = dt_bias[h], dskip = skip[h];
     const __nv_bfloat16* x_ = rows + (size_t)h * P + p_base;
     const __nv_bfloat16* b_ = rows + (size_t)H * P + (size_t)(h / (H / G)) * N;
     const __nv_bfloat16* c_ = b_ + (size_t)G * N;
 
-    auto load = [&](int stage, int base) {
-        const int count = min(kChunk, t1 - base);
-        __nv_bfloat16* cs = stages + stage * kStage;
+    auto load = [&](int c) {                                    // a token or column beyond the rows becomes zero
+        const int base = t0 + c * kChunk, count = min(kChunk, t1 - base);
+        __nv_bfloat16* cs = stages + (c % STAGES) * kStage;
         __nv_bfloat16 *bs = cs + kChunk * LDN, *xs = bs + kChunk * LDN;
-        for (int idx = tid; idx < kChunk * (NP / 8); idx += NW * 32) {
+        for (int idx = tid; idx < kChunk * (NP / 8); idx += kChunkThreads) {
             const int s = idx / (NP / 8), n = (idx % (NP / 8)) * 8;
             const bool ok = s < count && n < N;
             const size_t at = ok ? (size_t)(base + s) * stride + n : 0;
             cp_async16(cs + s * LDN + n, c_ + at, ok);
             cp_async16(bs + s * LDN + n, b_ + at, ok);
         }
-        for (int idx = tid; idx < kChunk * (PT / 8); idx += NW * 32) {
+        for (int idx = tid; idx < kChunk * (PT / 8); idx += kChunkThreads) {
             const int s = idx / (PT / 8), p = (idx % (PT / 8)) * 8;
             const bool ok = s < count && p_base + p < P;
             cp_async16(xs + s * LDP + p, x_ + (ok ? (size_t)(base + s) * stride + p : 0), ok);
         }
     };
-    // the two step sizes of a chunk that this lane of the first warp takes care of: tokens 2 lane and 2 lane + 1
-    auto raw_step = [&](int base, int s) { return base + s < t1 ? z[(size_t)(base + s) * z_stride + h] : 0.f; };
+    // the step sizes of a chunk, by one warp: tokens 2 lane and 2 lane + 1; a token beyond the rows has a step of zero
+    auto raw_step = [&](int c, int s) {
+        const int t = t0 + c * kChunk + s;
+        return t < t1 ? z[(size_t)t * z_stride + h] : 0.f;
+    };
+    auto step_sizes = [&](int c, float z0, float z1) {
+        const int count = min(kChunk, t1 - (t0 + c * kChunk));
+        float* Ls = steps + (c % 3) * 4 * kChunk;
+        float *dts = Ls + kChunk, *eL = dts + kChunk, *wu = eL + kChunk;
+        const float d0 = 2 * lane < count ? softplusf_(z0 + bias) : 0.f, d1 = 2 * lane + 1 < count ? softplusf_(z1 + bias) : 0.f;
+        const float l1 = a * d1;
+        float sum = fmaf(a, d0, l1);                            // inclusive over the lanes' pairs
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float v = __shfl_up_sync(0xffffffffu, sum, o);
+            if (lane >= o) sum += v;
+        }
+        const float end = __shfl_sync(0xffffffffu, sum, 31), first = sum - l1;
+        *reinterpret_cast<float2*>(Ls + 2 * lane) = make_float2(first, sum);
+        *reinterpret_cast<float2*>(dts + 2 * lane) = make_float2(d0, d1);
+        *reinterpret_cast<float2*>(eL + 2 * lane) = make_float2(expf(first), expf(sum));
+        *reinterpret_cast<float2*>(wu + 2 * lane) = make_float2(expf(end - first) * d0, expf(end - sum) * d1);
+    };
 
-    load(0, t0);
+    load(0);
     cp_async_commit();
-    float z0 = 0.f, z1 = 0.f;
-    if (warp == 0) {
-        z0 = raw_step(t0, 2 * lane);
-        z1 = raw_step(t0, 2 * lane + 1);
-    }
+    if (warp == 4) step_sizes(0, raw_step(0, 2 * lane), raw_step(0, 2 * lane + 1));
+    const int p_lo = p_base + warp * 16 + qrow, p_hi = p_lo + 8;             // a consumer's rows
+    const bool mine = !producer && p_base + warp * 16 < P;
     float S[NP / 8][4];                                          // rows p_lo, p_hi; columns 8 j + 2 quad, + 1
-    {
+    if (mine) {
         const float* st = has ? state + ((size_t)slot * H + h) * P * N : nullptr;
 #pragma unroll
         for (int j = 0; j < NP / 8; ++j) {
@@ -187,160 +206,165 @@ ssm_chunk_kernel(const __nv_bfloat16* __restrict__ rows, int stride, const float
             S[j][0] = lo.x; S[j][1] = lo.y; S[j][2] = hi.x; S[j][3] = hi.y;
         }
     }
-    int stage = 0;
-    for (int base = t0; base < t1; base += kChunk, stage ^= 1) {
-        const int count = min(kChunk, t1 - base), next = base + kChunk;
-        if (next < t1) load(stage ^ 1, next);
+    for (int c = -1; c < chunks; ++c) {                          // producers are one chunk ahead
+        cp_async_wait<0>();                                      // this thread's copies of chunk c + 1
+        __syncthreads();                                         // everyone's, and everyone is done with chunk c - 1
+        if (STAGES == 3 && c + 2 < chunks) load(c + 2);
+        if (STAGES == 2 && c == -1 && chunks > 1) load(1);
         cp_async_commit();
-        if (warp == 0) {
-            const bool ok0 = 2 * lane < count, ok1 = 2 * lane + 1 < count;
-            const float d0 = ok0 ? softplusf_(z0 + bias) : 0.f, d1 = ok1 ? softplusf_(z1 + bias) : 0.f;
-            if (next < t1) {
-                z0 = raw_step(next, 2 * lane);
-                z1 = raw_step(next, 2 * lane + 1);
-            }
-            const float l0 = a * d0, l1 = a * d1;
-            float sum = l0 + l1;                                 // inclusive over the lanes' pairs
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const float v = __shfl_up_sync(0xffffffffu, sum, o);
-                if (lane >= o) sum += v;
-            }
-            const float end = __shfl_sync(0xffffffffu, sum, 31);
-            const float first = sum - l1;
-            Ls[2 * lane] = first;
-            Ls[2 * lane + 1] = sum;
-            dts[2 * lane] = d0;
-            dts[2 * lane + 1] = d1;
-            eL[2 * lane] = expf(first);
-            eL[2 * lane + 1] = expf(sum);
-            wu[2 * lane] = expf(end - first) * d0;
-            wu[2 * lane + 1] = expf(end - sum) * d1;
-        }
-        cp_async_wait<1>();
-        __syncthreads();
-        const __nv_bfloat16* cs = stages + stage * kStage;
-        const __nv_bfloat16 *bs = cs + kChunk * LDN, *xs = bs + kChunk * LDN;
-
-        // x weighted for the update
-        for (int idx = tid; idx < kChunk * (PT / 2); idx += NW * 32) {
-            const int s = idx / (PT / 2), p = (idx % (PT / 2)) * 2;
-            const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(xs + s * LDP + p);
-            uint32_t hi, lo;
-            split_bf16(wu[s] * __low2float(v), wu[s] * __high2float(v), hi, lo);
-            *reinterpret_cast<uint32_t*>(xw_hi + s * LDP + p) = hi;
-            *reinterpret_cast<uint32_t*>(xw_lo + s * LDP + p) = lo;
-        }
-        // this warp's rows of C B^T, weighted; tiles above the diagonal are zero and never read
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-            const int tr = (warp * MT + m) * 16;
-            float g[kChunk / 8][4];
-#pragma unroll
-            for (int j = 0; j < kChunk / 8; ++j) g[j][0] = g[j][1] = g[j][2] = g[j][3] = 0.f;
+        if (producer) {
+            if (c + 1 < chunks) {
+                const int pc = c + 1, w4 = warp - 4, ptid = tid - 128;
+                const bool ahead = w4 == 0 && pc + 1 < chunks;
+                float z0 = 0.f, z1 = 0.f;
+                if (ahead) {
+                    z0 = raw_step(pc + 1, 2 * lane);
+                    z1 = raw_step(pc + 1, 2 * lane + 1);
+                }
+                const __nv_bfloat16* cs = stages + (pc % STAGES) * kStage;
+                const __nv_bfloat16 *bs = cs + kChunk * LDN, *xs = bs + kChunk * LDN;
+                const float* Ls = steps + (pc % 3) * 4 * kChunk;
+                const float *dts = Ls + kChunk, *wu = Ls + 3 * kChunk;
+                __nv_bfloat16 *xw_hi = xw + (pc & 1) * 2 * kChunk * LDP, *xw_lo = xw_hi + kChunk * LDP;
+                __nv_bfloat16 *w_hi = pw + (pc & 1) * 2 * kChunk * kChunkLd, *w_lo = w_hi + kChunk * kChunkLd;
 #pragma unroll 4
+                for (int idx = ptid; idx < kChunk * (PT / 4); idx += 128) {
+                    const int s = idx / (PT / 4), p = (idx % (PT / 4)) * 4;
+                    const uint2 v = *reinterpret_cast<const uint2*>(xs + s * LDP + p);
+                    const float2 v0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
+                    const float2 v1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+                    const float f = wu[s];
+                    uint2 hi, lo;
+                    split_bf16(f * v0.x, f * v0.y, hi.x, lo.x);
+                    split_bf16(f * v1.x, f * v1.y, hi.y, lo.y);
+                    *reinterpret_cast<uint2*>(xw_hi + s * LDP + p) = hi;
+                    *reinterpret_cast<uint2*>(xw_lo + s * LDP + p) = lo;
+                }
+                // this warp's rows of C B^T, weighted; tiles above the diagonal are never read
+                const int tr = w4 * 16;
+                float g[kChunk / 8][4];
+#pragma unroll
+                for (int j = 0; j < kChunk / 8; ++j) g[j][0] = g[j][1] = g[j][2] = g[j][3] = 0.f;
+#pragma unroll 4
+                for (int kk = 0; kk < NP / 16; ++kk) {
+                    uint32_t af[4];
+                    ldmatrix_x4(af, smem_u32(cs + (tr + (mat & 1) * 8 + rr) * LDN + kk * 16 + (mat >> 1) * 8));
+#pragma unroll
+                    for (int np = 0; np < kChunk / 16; ++np) {
+                        if (np > w4) continue;
+                        uint32_t bf[4];
+                        ldmatrix_x4(bf, smem_u32(bs + (np * 16 + (mat >> 1) * 8 + rr) * LDN + kk * 16 + (mat & 1) * 8));
+                        mma_bf16_16816(g[2 * np], af, bf[0], bf[1]);
+                        mma_bf16_16816(g[2 * np + 1], af, bf[2], bf[3]);
+                    }
+                }
+                const int ta = tr + qrow, tb = ta + 8;
+                const float La = Ls[ta], Lb = Ls[tb];
+#pragma unroll
+                for (int j = 0; j < kChunk / 8; ++j) {
+                    if (j > 2 * w4 + 1) continue;
+                    const int s = j * 8 + quad * 2;
+                    const float2 ls = *reinterpret_cast<const float2*>(Ls + s), d = *reinterpret_cast<const float2*>(dts + s);
+                    uint32_t hi, lo;
+                    split_bf16(s <= ta ? g[j][0] * expf(La - ls.x) * d.x : 0.f, s + 1 <= ta ? g[j][1] * expf(La - ls.y) * d.y : 0.f, hi, lo);
+                    *reinterpret_cast<uint32_t*>(w_hi + ta * kChunkLd + s) = hi;
+                    *reinterpret_cast<uint32_t*>(w_lo + ta * kChunkLd + s) = lo;
+                    split_bf16(s <= tb ? g[j][2] * expf(Lb - ls.x) * d.x : 0.f, s + 1 <= tb ? g[j][3] * expf(Lb - ls.y) * d.y : 0.f, hi, lo);
+                    *reinterpret_cast<uint32_t*>(w_hi + tb * kChunkLd + s) = hi;
+                    *reinterpret_cast<uint32_t*>(w_lo + tb * kChunkLd + s) = lo;
+                }
+                if (ahead) step_sizes(pc + 1, z0, z1);
+            }
+        } else if (c >= 0 && mine) {
+            const __nv_bfloat16* cs = stages + (c % STAGES) * kStage;
+            const __nv_bfloat16 *bs = cs + kChunk * LDN, *xs = bs + kChunk * LDN;
+            const float* eL = steps + (c % 3) * 4 * kChunk + 2 * kChunk;
+            const __nv_bfloat16 *xw_hi = xw + (c & 1) * 2 * kChunk * LDP, *xw_lo = xw_hi + kChunk * LDP;
+            const __nv_bfloat16 *w_hi = pw + (c & 1) * 2 * kChunk * kChunkLd, *w_lo = w_hi + kChunk * kChunkLd;
+            // y = S0 C^T: rows of S from the registers
+            float y[kChunk / 8][4];
+#pragma unroll
+            for (int j = 0; j < kChunk / 8; ++j) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
+#pragma unroll
             for (int kk = 0; kk < NP / 16; ++kk) {
-                uint32_t af[4];
-                ldmatrix_x4(af, smem_u32(cs + (tr + (mat & 1) * 8 + rr) * LDN + kk * 16 + (mat >> 1) * 8));
+                uint32_t hi[4], lo[4];
+                split_bf16(S[2 * kk][0], S[2 * kk][1], hi[0], lo[0]);
+                split_bf16(S[2 * kk][2], S[2 * kk][3], hi[1], lo[1]);
+                split_bf16(S[2 * kk + 1][0], S[2 * kk + 1][1], hi[2], lo[2]);
+                split_bf16(S[2 * kk + 1][2], S[2 * kk + 1][3], hi[3], lo[3]);
+                uint32_t bf[kChunk / 16][4];
+#pragma unroll
+                for (int np = 0; np < kChunk / 16; ++np)
+                    ldmatrix_x4(bf[np], smem_u32(cs + (np * 16 + (mat >> 1) * 8 + rr) * LDN + kk * 16 + (mat & 1) * 8));
 #pragma unroll
                 for (int np = 0; np < kChunk / 16; ++np) {
-                    if (np * 16 > tr) continue;
-                    uint32_t bf[4];
-                    ldmatrix_x4(bf, smem_u32(bs + (np * 16 + (mat >> 1) * 8 + rr) * LDN + kk * 16 + (mat & 1) * 8));
-                    mma_bf16_16816(g[2 * np], af, bf[0], bf[1]);
-                    mma_bf16_16816(g[2 * np + 1], af, bf[2], bf[3]);
+                    mma_bf16_16816(y[2 * np], hi, bf[np][0], bf[np][1]);
+                    mma_bf16_16816(y[2 * np + 1], hi, bf[np][2], bf[np][3]);
+                }
+#pragma unroll
+                for (int np = 0; np < kChunk / 16; ++np) {
+                    mma_bf16_16816(y[2 * np], lo, bf[np][0], bf[np][1]);
+                    mma_bf16_16816(y[2 * np + 1], lo, bf[np][2], bf[np][3]);
                 }
             }
-            const int ta = tr + qrow, tb = ta + 8;
-            const float La = Ls[ta], Lb = Ls[tb];
 #pragma unroll
             for (int j = 0; j < kChunk / 8; ++j) {
-                if (j * 8 >= tr + 16) continue;
-                const int s = j * 8 + quad * 2;
-                const float ls0 = Ls[s], ls1 = Ls[s + 1], d0 = dts[s], d1 = dts[s + 1];
-                uint32_t hi, lo;
-                split_bf16(s <= ta ? g[j][0] * expf(La - ls0) * d0 : 0.f, s + 1 <= ta ? g[j][1] * expf(La - ls1) * d1 : 0.f, hi, lo);
-                *reinterpret_cast<uint32_t*>(w_hi + ta * kChunkLd + s) = hi;
-                *reinterpret_cast<uint32_t*>(w_lo + ta * kChunkLd + s) = lo;
-                split_bf16(s <= tb ? g[j][2] * expf(Lb - ls0) * d0 : 0.f, s + 1 <= tb ? g[j][3] * expf(Lb - ls1) * d1 : 0.f, hi, lo);
-                *reinterpret_cast<uint32_t*>(w_hi + tb * kChunkLd + s) = hi;
-                *reinterpret_cast<uint32_t*>(w_lo + tb * kChunkLd + s) = lo;
+                const float2 e = *reinterpret_cast<const float2*>(eL + j * 8 + quad * 2);
+                y[j][0] *= e.x; y[j][1] *= e.y; y[j][2] *= e.x; y[j][3] *= e.y;
+            }
+            const float e_end = eL[kChunk - 1];
+#pragma unroll
+            for (int j = 0; j < NP / 8; ++j) { S[j][0] *= e_end; S[j][1] *= e_end; S[j][2] *= e_end; S[j][3] *= e_end; }
+#pragma unroll
+            for (int kk = 0; kk < kChunk / 16; ++kk) {
+                const int s0 = kk * 16;
+                uint32_t xa[4], wa_hi[4], wa_lo[4];
+                const int at = (s0 + (mat >> 1) * 8 + rr) * LDP + warp * 16 + (mat & 1) * 8;
+                ldmatrix_x4_trans(xa, smem_u32(xs + at));
+                ldmatrix_x4_trans(wa_hi, smem_u32(xw_hi + at));
+                ldmatrix_x4_trans(wa_lo, smem_u32(xw_lo + at));
+#pragma unroll
+                for (int np = 0; np < kChunk / 16; ++np) {
+                    if (np < kk) continue;                       // tokens before s0 do not see it
+                    uint32_t bh[4], bl[4];
+                    ldmatrix_x4(bh, smem_u32(w_hi + (np * 16 + (mat >> 1) * 8 + rr) * kChunkLd + s0 + (mat & 1) * 8));
+                    ldmatrix_x4(bl, smem_u32(w_lo + (np * 16 + (mat >> 1) * 8 + rr) * kChunkLd + s0 + (mat & 1) * 8));
+                    mma_bf16_16816(y[2 * np], xa, bh[0], bh[1]);
+                    mma_bf16_16816(y[2 * np + 1], xa, bh[2], bh[3]);
+                    mma_bf16_16816(y[2 * np], xa, bl[0], bl[1]);
+                    mma_bf16_16816(y[2 * np + 1], xa, bl[2], bl[3]);
+                }
+#pragma unroll
+                for (int nj = 0; nj < NP / 16; ++nj) {
+                    uint32_t bf[4];
+                    ldmatrix_x4_trans(bf, smem_u32(bs + (s0 + (mat & 1) * 8 + rr) * LDN + nj * 16 + (mat >> 1) * 8));
+                    mma_bf16_16816(S[2 * nj], wa_hi, bf[0], bf[1]);
+                    mma_bf16_16816(S[2 * nj + 1], wa_hi, bf[2], bf[3]);
+                    mma_bf16_16816(S[2 * nj], wa_lo, bf[0], bf[1]);
+                    mma_bf16_16816(S[2 * nj + 1], wa_lo, bf[2], bf[3]);
+                }
+            }
+            const int base = t0 + c * kChunk, count = min(kChunk, t1 - base);
+            const int xl = warp * 16 + qrow;                     // this lane's rows within x's columns
+#pragma unroll
+            for (int j = 0; j < kChunk / 8; ++j) {
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int s = j * 8 + quad * 2 + e;
+                    if (s >= count) continue;
+                    float* dst = out + ((size_t)(base + s) * H + h) * P;
+                    if (p_lo < P) dst[p_lo] = fmaf(dskip, __bfloat162float(xs[s * LDP + xl]), y[j][e]);
+                    if (p_hi < P) dst[p_hi] = fmaf(dskip, __bfloat162float(xs[s * LDP + xl + 8]), y[j][2 + e]);
+                }
             }
         }
-        // y = S0 C^T: rows of S from the registers
-        float y[kChunk / 8][4];
-#pragma unroll
-        for (int j = 0; j < kChunk / 8; ++j) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
-#pragma unroll
-        for (int kk = 0; kk < NP / 16; ++kk) {
-            uint32_t hi[4], lo[4];
-            split_bf16(S[2 * kk][0], S[2 * kk][1], hi[0], lo[0]);
-            split_bf16(S[2 * kk][2], S[2 * kk][3], hi[1], lo[1]);
-            split_bf16(S[2 * kk + 1][0], S[2 * kk + 1][1], hi[2], lo[2]);
-            split_bf16(S[2 * kk + 1][2], S[2 * kk + 1][3], hi[3], lo[3]);
-#pragma unroll
-            for (int np = 0; np < kChunk / 16; ++np) {
-                uint32_t bf[4];
-                ldmatrix_x4(bf, smem_u32(cs + (np * 16 + (mat >> 1) * 8 + rr) * LDN + kk * 16 + (mat & 1) * 8));
-                mma_bf16_16816(y[2 * np], hi, bf[0], bf[1]);
-                mma_bf16_16816(y[2 * np + 1], hi, bf[2], bf[3]);
-                mma_bf16_16816(y[2 * np], lo, bf[0], bf[1]);
-                mma_bf16_16816(y[2 * np + 1], lo, bf[2], bf[3]);
-            }
+        if (STAGES == 2 && c >= 0 && c + 2 < chunks) {           // the stage of chunk c is free only now
+            __syncthreads();
+            load(c + 2);
+            cp_async_commit();
         }
-#pragma unroll
-        for (int j = 0; j < kChunk / 8; ++j) {
-            const float e0 = eL[j * 8 + quad * 2], e1 = eL[j * 8 + quad * 2 + 1];
-            y[j][0] *= e0; y[j][1] *= e1; y[j][2] *= e0; y[j][3] *= e1;
-        }
-        const float e_end = eL[kChunk - 1];                      // a token beyond the chunk's count has a step of zero
-#pragma unroll
-        for (int j = 0; j < NP / 8; ++j) { S[j][0] *= e_end; S[j][1] *= e_end; S[j][2] *= e_end; S[j][3] *= e_end; }
-        __syncthreads();                                         // weighted x and pair weights are in place
-#pragma unroll
-        for (int kk = 0; kk < kChunk / 16; ++kk) {
-            const int s0 = kk * 16;
-            uint32_t xa[4], wa_hi[4], wa_lo[4];
-            const int at = (s0 + (mat >> 1) * 8 + rr) * LDP + warp * 16 + (mat & 1) * 8;
-            ldmatrix_x4_trans(xa, smem_u32(xs + at));
-            ldmatrix_x4_trans(wa_hi, smem_u32(xw_hi + at));
-            ldmatrix_x4_trans(wa_lo, smem_u32(xw_lo + at));
-#pragma unroll
-            for (int np = 0; np < kChunk / 16; ++np) {
-                if (np < kk) continue;                           // tokens before s0 do not see it
-                uint32_t bf[4];
-                ldmatrix_x4(bf, smem_u32(w_hi + (np * 16 + (mat >> 1) * 8 + rr) * kChunkLd + s0 + (mat & 1) * 8));
-                mma_bf16_16816(y[2 * np], xa, bf[0], bf[1]);
-                mma_bf16_16816(y[2 * np + 1], xa, bf[2], bf[3]);
-                ldmatrix_x4(bf, smem_u32(w_lo + (np * 16 + (mat >> 1) * 8 + rr) * kChunkLd + s0 + (mat & 1) * 8));
-                mma_bf16_16816(y[2 * np], xa, bf[0], bf[1]);
-                mma_bf16_16816(y[2 * np + 1], xa, bf[2], bf[3]);
-            }
-#pragma unroll
-            for (int nj = 0; nj < NP / 16; ++nj) {
-                uint32_t bf[4];
-                ldmatrix_x4_trans(bf, smem_u32(bs + (s0 + (mat & 1) * 8 + rr) * LDN + nj * 16 + (mat >> 1) * 8));
-                mma_bf16_16816(S[2 * nj], wa_hi, bf[0], bf[1]);
-                mma_bf16_16816(S[2 * nj + 1], wa_hi, bf[2], bf[3]);
-                mma_bf16_16816(S[2 * nj], wa_lo, bf[0], bf[1]);
-                mma_bf16_16816(S[2 * nj + 1], wa_lo, bf[2], bf[3]);
-            }
-        }
-        const int xl = warp * 16 + qrow;                         // this lane's rows within x's columns
-#pragma unroll
-        for (int j = 0; j < kChunk / 8; ++j) {
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int s = j * 8 + quad * 2 + e;
-                if (s >= count) continue;
-                float* dst = out + ((size_t)(base + s) * H + h) * P;
-                if (p_lo < P) dst[p_lo] = fmaf(dskip, __bfloat162float(xs[s * LDP + xl]), y[j][e]);
-                if (p_hi < P) dst[p_hi] = fmaf(dskip, __bfloat162float(xs[s * LDP + xl + 8]), y[j][2 + e]);
-            }
-        }
-        __syncthreads();                                         // the stage and the scratch are free
     }
-    if (!has) return;
+    if (!has || !mine) return;
     float* st = state + ((size_t)slot * H + h) * P * N;
 #pragma unroll
     for (int j = 0; j < NP / 8; ++j) {
@@ -409,16 +433,17 @@ extern "C" int cib_ssm_chunk_supports(int H, int G, int P, int N) {
     return H > 0 && G > 0 && P % 8 == 0 && N % 8 == 0 && N <= 256 && H % G == 0;
 }
 
-template <int NP, int NW>
+template <int NP>
 static int launch_ssm_chunk(const void* rows, int stride, const float* z, int z_stride, AnyVec db, AnyVec al, AnyVec sk, float* state,
                             const int* query_start_loc, const int* state_slots, int num_slots, int num_requests, float* out, int H, int G, int P,
                             int N, cudaStream_t stream) {
-    constexpr size_t smem = ssm_chunk_smem<NP, NW>();
+    constexpr size_t smem = ssm_chunk_smem<NP>();
+    static_assert(smem <= 227 * 1024, "a chunk's working set does not fit");
     static SmemLimit limit;
-    if (int rc = raise_smem_limit(limit, ssm_chunk_kernel<NP, NW>, smem, "ssm_chunk")) return rc;
-    const dim3 grid(H, (P + NW * 16 - 1) / (NW * 16), num_requests);
-    ssm_chunk_kernel<NP, NW><<<grid, NW * 32, smem, stream>>>((const __nv_bfloat16*)rows, stride, z, z_stride, db, al, sk, state, query_start_loc,
-                                                             state_slots, num_slots, out, H, G, P, N);
+    if (int rc = raise_smem_limit(limit, ssm_chunk_kernel<NP>, smem, "ssm_chunk")) return rc;
+    const dim3 grid(H, (P + kChunkRows - 1) / kChunkRows, num_requests);
+    ssm_chunk_kernel<NP><<<grid, kChunkThreads, smem, stream>>>((const __nv_bfloat16*)rows, stride, z, z_stride, db, al, sk, state, query_start_loc,
+                                                               state_slots, num_slots, out, H, G, P, N);
     CIB_LAUNCH_CHECK("ssm_chunk");
     return 0;
 }
@@ -437,13 +462,8 @@ extern "C" int cib_ssm_scan(const void* rows, int dtype, int stride, const float
         CIB_REQUIRE(dtype == kBF16 && cib_ssm_chunk_supports(H, G, P, N) && stride % 8 == 0 && (uintptr_t)rows % 16 == 0 && (uintptr_t)state % 16 == 0,
                     "ssm_scan: the rows do not fit the tensor-core form");
         CIB_REQUIRE(num_requests <= 65535, "ssm_scan: too many requests");
-        // two warps (32 rows of S) a CTA while four would leave SMs without work
-        const bool narrow = P <= 32 || (long long)num_requests * H * ((P + 63) / 64) < 148;
 #define CIB_SSM(NP)                                                                                                                       \
-    return narrow ? launch_ssm_chunk<NP, 2>(rows, stride, z, z_stride, db, al, sk, state, query_start_loc, state_slots, num_slots,           \
-                                            num_requests, out, H, G, P, N, stream)                                                     \
-                  : launch_ssm_chunk<NP, 4>(rows, stride, z, z_stride, db, al, sk, state, query_start_loc, state_slots, num_slots,           \
-                                            num_requests, out, H, G, P, N, stream)
+    return launch_ssm_chunk<NP>(rows, stride, z, z_stride, db, al, sk, state, query_start_loc, state_slots, num_slots, num_requests, out, H, G, P, N, stream)
         if (N <= 32) CIB_SSM(32);
         if (N <= 64) CIB_SSM(64);
         if (N <= 128) CIB_SSM(128);
