@@ -216,6 +216,8 @@ class KernelTimes:
             rep_args = args
             if name in ("sandwich_layernorm", "add_rmsnorm", "rms_stream", "group_rms"):           # they add into their first argument
                 rep_args = (args[0].clone(),) + tuple(args[1:])
+            if name == "bias_rows":                                                                # may run in place
+                rep_args = (args[0], args[1], torch.empty_like(args[2]))
             # the repeats are recorded into a CUDA graph and the graph is timed: the device's time, not Python's
             torch.cuda.synchronize()
             graph = torch.cuda.CUDAGraph()

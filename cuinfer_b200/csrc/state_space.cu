@@ -7,7 +7,8 @@
 //
 // Requests, slots and the order of tokens as in recurrent.cu.  Step sizes, decays, state and read-out are 32-bit.
 //
-// Two kernels.
+// Two kernels.  A step of several requests runs both: requests of up to kSsmFewTokens tokens walk (a decoded token beside a
+// prompt's portion would cost a whole chunk), longer ones go in chunks.
 //  * ssm_walk: token after token in 32-bit FMA, any sizes; a warp holds four rows of S over its lanes.  Steps of single tokens,
 //    the 32-bit engine, sizes the other does not take.
 //  * ssm_chunk (bfloat16 rows): 64 tokens at a time on the tensor cores.  With L_t the sum of the log decays of a chunk's tokens
@@ -22,20 +23,21 @@
 
 namespace cib {
 
+constexpr int kSsmFewTokens = 16;
 constexpr int kSsmWarps = 4, kSsmRows = 4;       // a block walks kSsmWarps * kSsmRows rows of a head's state
 
 template <typename T, int C>
 __global__ void __launch_bounds__(kSsmWarps * 32)
 ssm_walk_kernel(const T* __restrict__ rows, int stride, const float* __restrict__ z, int z_stride, AnyVec dt_bias, AnyVec a_log, AnyVec skip,
                 float* __restrict__ state, const int* __restrict__ query_start_loc, const int* __restrict__ state_slots, int num_slots,
-                float* __restrict__ out, int H, int G, int P, int N) {
+                float* __restrict__ out, int H, int G, int P, int N, int few) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int r = blockIdx.x, h = blockIdx.y, p0 = (blockIdx.z * kSsmWarps + warp) * kSsmRows;
     griddep_launch();
     const float a = -expf(a_log[h]), bias = dt_bias[h], dskip = skip[h];          // weights
     griddep_wait();
     const int t0 = query_start_loc[r], t1 = query_start_loc[r + 1];
-    if (t1 <= t0 || p0 >= P) return;
+    if (t1 <= t0 || p0 >= P || (few > 0 && t1 - t0 > few)) return;
     const int slot = state_slots[r];
     const bool has = slot >= 0 && slot < num_slots;
     float* st = has ? state + (((size_t)slot * H + h) * P + p0) * N : nullptr;
@@ -127,7 +129,7 @@ template <int NP>
 __global__ void __launch_bounds__(kChunkThreads)
 ssm_chunk_kernel(const __nv_bfloat16* __restrict__ rows, int stride, const float* __restrict__ z, int z_stride, AnyVec dt_bias, AnyVec a_log,
                  AnyVec skip, float* __restrict__ state, const int* __restrict__ query_start_loc, const int* __restrict__ state_slots,
-                 int num_slots, float* __restrict__ out, int H, int G, int P, int N) {
+                 int num_slots, float* __restrict__ out, int H, int G, int P, int N, int few) {
     constexpr int PT = kChunkRows, LDN = NP + 8, LDP = PT + 8, STAGES = ssm_stages<NP>();
     constexpr int kStage = 2 * kChunk * LDN + kChunk * LDP;
     extern __shared__ __align__(16) unsigned char ssm_raw[];
@@ -139,7 +141,7 @@ ssm_chunk_kernel(const __nv_bfloat16* __restrict__ rows, int stride, const float
     const bool producer = warp >= 4;
     const int r = blockIdx.z, h = blockIdx.x, p_base = blockIdx.y * PT;
     const int t0 = query_start_loc[r], t1 = query_start_loc[r + 1];
-    if (t1 <= t0) return;
+    if (t1 - t0 <= few) return;
     const int chunks = (t1 - t0 + kChunk - 1) / kChunk;
     const int slot = state_slots[r];
     const bool has = slot >= 0 && slot < num_slots;
@@ -436,14 +438,14 @@ extern "C" int cib_ssm_chunk_supports(int H, int G, int P, int N) {
 template <int NP>
 static int launch_ssm_chunk(const void* rows, int stride, const float* z, int z_stride, AnyVec db, AnyVec al, AnyVec sk, float* state,
                             const int* query_start_loc, const int* state_slots, int num_slots, int num_requests, float* out, int H, int G, int P,
-                            int N, cudaStream_t stream) {
+                            int N, int few, cudaStream_t stream) {
     constexpr size_t smem = ssm_chunk_smem<NP>();
     static_assert(smem <= 227 * 1024, "a chunk's working set does not fit");
     static SmemLimit limit;
     if (int rc = raise_smem_limit(limit, ssm_chunk_kernel<NP>, smem, "ssm_chunk")) return rc;
     const dim3 grid(H, (P + kChunkRows - 1) / kChunkRows, num_requests);
     ssm_chunk_kernel<NP><<<grid, kChunkThreads, smem, stream>>>((const __nv_bfloat16*)rows, stride, z, z_stride, db, al, sk, state, query_start_loc,
-                                                               state_slots, num_slots, out, H, G, P, N);
+                                                               state_slots, num_slots, out, H, G, P, N, few);
     CIB_LAUNCH_CHECK("ssm_chunk");
     return 0;
 }
@@ -458,23 +460,27 @@ extern "C" int cib_ssm_scan(const void* rows, int dtype, int stride, const float
     CIB_REQUIRE(N <= 256, "ssm_scan: state size %d is beyond 256", N);
     if (num_requests == 0 || num_tokens == 0) return 0;
     AnyVec db{dt_bias, vec_dtype == kBF16}, al{a_log, vec_dtype == kBF16}, sk{skip, vec_dtype == kBF16};
+    const int few = chunks && num_requests > 1 ? kSsmFewTokens : 0;
     if (chunks) {
         CIB_REQUIRE(dtype == kBF16 && cib_ssm_chunk_supports(H, G, P, N) && stride % 8 == 0 && (uintptr_t)rows % 16 == 0 && (uintptr_t)state % 16 == 0,
                     "ssm_scan: the rows do not fit the tensor-core form");
         CIB_REQUIRE(num_requests <= 65535, "ssm_scan: too many requests");
+        int rc;
 #define CIB_SSM(NP)                                                                                                                       \
-    return launch_ssm_chunk<NP>(rows, stride, z, z_stride, db, al, sk, state, query_start_loc, state_slots, num_slots, num_requests, out, H, G, P, N, stream)
+    rc = launch_ssm_chunk<NP>(rows, stride, z, z_stride, db, al, sk, state, query_start_loc, state_slots, num_slots, num_requests, out, H, G, P, \
+                              N, few, stream)
         if (N <= 32) CIB_SSM(32);
-        if (N <= 64) CIB_SSM(64);
-        if (N <= 128) CIB_SSM(128);
-        CIB_SSM(256);
+        else if (N <= 64) CIB_SSM(64);
+        else if (N <= 128) CIB_SSM(128);
+        else CIB_SSM(256);
 #undef CIB_SSM
+        if (rc != 0 || few == 0) return rc;
     }
     const dim3 grid(num_requests, H, (P + kSsmWarps * kSsmRows - 1) / (kSsmWarps * kSsmRows));
     const bool pdl = prompt_pdl();
 #define CIB_WALK(T, C)                                                                                                                    \
     launch_pdl(ssm_walk_kernel<T, C>, grid, dim3(kSsmWarps * 32), 0, stream, pdl, (const T*)rows, stride, z, z_stride, db, al, sk, state,      \
-               query_start_loc, state_slots, num_slots, out, H, G, P, N)
+               query_start_loc, state_slots, num_slots, out, H, G, P, N, few)
 #define CIB_WALK_N(T)                         \
     do {                                      \
         if (N <= 32) CIB_WALK(T, 1);          \

@@ -1556,7 +1556,8 @@ def ssm_scan(rows: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log:
     """The state-space recurrence with a scalar decay per head over every request's rows ``[x (H P) | B (G N) | C (G N)]``:
     ``S <- exp(-exp(a_log) step) S + step x B^T``, ``out = S C + skip x`` with ``step = softplus(dt + dt_bias)``; ``dt`` float32
     [T, >= H] (any row stride), ``state`` float32 [slots, H, P * N], ``out`` float32 [T, H * P].  ``chunks``: 64 tokens at a
-    time on the tensor cores (see ``ssm_chunk_supports``); else token after token in 32 bits."""
+    time on the tensor cores (see ``ssm_chunk_supports``), with a second launch for the requests of a few tokens when there
+    are several requests; else token after token in 32 bits."""
     T = out.shape[0]
     H, G, P, N = num_heads, groups, vdim, state_size
     if (rows.shape[0] != T or rows.shape[1] < H * P + 2 * G * N or rows.stride(1) != 1 or out.shape != (T, H * P)
@@ -1573,6 +1574,8 @@ def ssm_scan(rows: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log:
         state_slots.numel(), T, _cuda(out, "out", torch.float32), H, G, P, N, 1 if chunks else 0, _stream())
     _check(rc, "ssm_scan")
     _count()
+    if chunks and state_slots.numel() > 1:
+        _count()
 
 
 def gated_group_rms(y: torch.Tensor, z: torch.Tensor, gain: torch.Tensor, eps: float, groups: int, out: torch.Tensor) -> None:

@@ -602,6 +602,31 @@ def test_state_space_scan(H, G, P, N, form):
 
 
 @pytest.mark.parametrize("chunks", [False, True])
+def test_state_space_scan_of_one_request_in_short_portions(chunks):
+    """Portions of one to 70 tokens of a request that is alone in its steps: every one goes through the form asked for."""
+    from cuinfer_b200 import kernels
+
+    g = torch.Generator().manual_seed(3)
+    H, G, P, N = 3, 3, 24, 40
+    portions = [2, 3, 1, 16, 17, 63, 2, 64, 65, 5, 70]
+    n = sum(portions)
+    xbc, dt = torch.randn(n, H * P + 2 * G * N, generator=g).bfloat16(), (torch.randn(n, H, generator=g) - 1).float()
+    a_log, dt_bias, skip = torch.tensor([-3.0, 0.0, 1.0]), torch.zeros(H), torch.ones(H)
+    x, B, C = torch.split(xbc.double(), [H * P, G * N, G * N], 1)
+    want, S = plain.state_space_scan(x.reshape(n, H, P), B.reshape(n, G, N), C.reshape(n, G, N), plain.softplus(dt.double()), a_log.double(), skip.double())
+    state = torch.zeros(2, H, P * N, device="cuda")
+    at = 0
+    for k in portions:
+        out = torch.empty(k, H * P, device="cuda")
+        kernels.ssm_scan(xbc[at:at + k].cuda(), dt[at:at + k].cuda(), dt_bias.cuda(), a_log.cuda(), skip.cuda(), state, _ints([0, k]), _ints([1]),
+                         out, H, G, P, N, chunks=chunks)
+        _close(out.view(k, H, P), want[at:at + k], torch.float32, f"tokens {at}..", tol=2e-4 if chunks else 1e-5)
+        at += k
+    _close(state[1].view(H, P, N), S.transpose(1, 2), torch.float32, "state", tol=2e-4 if chunks else 1e-5)
+    assert not state[0].any()
+
+
+@pytest.mark.parametrize("chunks", [False, True])
 def test_state_space_scan_remembers_a_far_token(chunks):
     """A memory that hardly fades: one early token writes, the other tokens write next to nothing, and the read-out a
     thousand tokens later is that token's value times its decay, to many digits."""
