@@ -104,7 +104,6 @@ ssm_walk_kernel(const T* __restrict__ rows, int stride, const float* __restrict_
 // ---- chunks of 64 tokens on the tensor cores -----------------------------------------------------------------------------
 constexpr int kChunk = 64;
 constexpr int kChunkLd = kChunk + 8;
-constexpr int kChunkRows = 64;                   // rows of S a CTA owns: sixteen a consumer warp
 constexpr int kChunkThreads = 256;
 
 __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint32_t& lo) {
@@ -114,29 +113,35 @@ __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint3
 }
 
 template <int NP> constexpr int ssm_stages() { return NP <= 128 ? 3 : 2; }
-template <int NP> constexpr size_t ssm_chunk_smem() {
-    return (size_t)ssm_stages<NP>() * (2 * kChunk * (NP + 8) + kChunk * (kChunkRows + 8)) * 2      // C, B, x of a chunk
-           + (size_t)2 * 2 * kChunk * (kChunkRows + 8) * 2                  // two chunks' weighted x, value and remainder
+template <int NP, int TILES> constexpr size_t ssm_chunk_smem() {
+    constexpr int PT = TILES * 16;
+    return (size_t)ssm_stages<NP>() * (2 * kChunk * (NP + 8) + kChunk * (PT + 8)) * 2      // C, B, x of a chunk
+           + (size_t)2 * 2 * kChunk * (PT + 8) * 2                          // two chunks' weighted x, value and remainder
            + (size_t)2 * 2 * kChunk * kChunkLd * 2                          // two chunks' weights of pairs, likewise
-           + (size_t)3 * 4 * kChunk * 4;                                    // three chunks' L, dt, exp(L), weights of the update
+           + (size_t)3 * 5 * kChunk * 4                                     // three chunks' L, dt, exp(L), weights of the update, of pairs
+           + (TILES < 4 ? (size_t)4 * 8 * 32 * 16 : 0);                     // the consumers' parts of y
 }
 
-// A CTA walks the chunks of one request for 64 rows of one head's S.  Only the state links one chunk to the next, so the
-// warps divide: four producers make the next chunk's weighted x and pair weights (16 tokens each, and the first of them
-// the step sizes of the chunk after it), four consumers take the current chunk's products with S, 16 rows of it each.
-// One barrier a chunk.
-template <int NP>
+// A CTA walks the chunks of one request for 16 TILES rows of one head's S.  Only the state links one chunk to the next, so
+// the warps divide: four producers make the next chunk's weighted x and pair weights (16 tokens each, and the first of them
+// the step sizes of the chunk after it), four consumers take the current chunk's products with S.  One barrier a chunk.
+// A consumer holds 16 rows and 1 / SPLIT of the columns of S (SPLIT = 4 / TILES: the tensor pipe of a warp's scheduler is what
+// bounds a chunk's time, so a prompt with too few heads to fill the GPU shares a row tile out to several schedulers); the
+// parts of y that its columns and its share of the pairs give are then added through shared memory.
+template <int NP, int TILES>
 __global__ void __launch_bounds__(kChunkThreads)
 ssm_chunk_kernel(const __nv_bfloat16* __restrict__ rows, int stride, const float* __restrict__ z, int z_stride, AnyVec dt_bias, AnyVec a_log,
                  AnyVec skip, float* __restrict__ state, const int* __restrict__ query_start_loc, const int* __restrict__ state_slots,
                  int num_slots, float* __restrict__ out, int H, int G, int P, int N, int few) {
-    constexpr int PT = kChunkRows, LDN = NP + 8, LDP = PT + 8, STAGES = ssm_stages<NP>();
+    constexpr int PT = TILES * 16, LDN = NP + 8, LDP = PT + 8, STAGES = ssm_stages<NP>(), SPLIT = 4 / TILES, NS = NP / SPLIT;
+    static_assert(NS % 16 == 0, "a warp's columns are whole steps of a product");
     constexpr int kStage = 2 * kChunk * LDN + kChunk * LDP;
     extern __shared__ __align__(16) unsigned char ssm_raw[];
     __nv_bfloat16* stages = reinterpret_cast<__nv_bfloat16*>(ssm_raw);
     __nv_bfloat16* xw = stages + STAGES * kStage;               // [2 chunks][value, remainder][kChunk][LDP]
     __nv_bfloat16* pw = xw + 4 * kChunk * LDP;                  // [2 chunks][value, remainder][kChunk][kChunkLd]
-    float* steps = reinterpret_cast<float*>(pw + 4 * kChunk * kChunkLd);      // [3 chunks][L, dt, exp(L), update][kChunk]
+    float* steps = reinterpret_cast<float*>(pw + 4 * kChunk * kChunkLd);      // [3 chunks][L, dt, exp(L), update, pairs][kChunk]
+    float4* parts = reinterpret_cast<float4*>(steps + 3 * 5 * kChunk);        // [consumer][j][lane]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const bool producer = warp >= 4;
     const int r = blockIdx.z, h = blockIdx.x, p_base = blockIdx.y * PT;
@@ -175,8 +180,8 @@ ssm_chunk_kernel(const __nv_bfloat16* __restrict__ rows, int stride, const float
     };
     auto step_sizes = [&](int c, float z0, float z1) {
         const int count = min(kChunk, t1 - (t0 + c * kChunk));
-        float* Ls = steps + (c % 3) * 4 * kChunk;
-        float *dts = Ls + kChunk, *eL = dts + kChunk, *wu = eL + kChunk;
+        float* Ls = steps + (c % 3) * 5 * kChunk;
+        float *dts = Ls + kChunk, *eL = dts + kChunk, *wu = eL + kChunk, *wp = wu + kChunk;
         const float d0 = 2 * lane < count ? softplusf_(z0 + bias) : 0.f, d1 = 2 * lane + 1 < count ? softplusf_(z1 + bias) : 0.f;
         const float l1 = a * d1;
         float sum = fmaf(a, d0, l1);                            // inclusive over the lanes' pairs
@@ -190,19 +195,22 @@ ssm_chunk_kernel(const __nv_bfloat16* __restrict__ rows, int stride, const float
         *reinterpret_cast<float2*>(dts + 2 * lane) = make_float2(d0, d1);
         *reinterpret_cast<float2*>(eL + 2 * lane) = make_float2(expf(first), expf(sum));
         *reinterpret_cast<float2*>(wu + 2 * lane) = make_float2(expf(end - first) * d0, expf(end - sum) * d1);
+        const float edge = __shfl_sync(0xffffffffu, sum, lane | 7);          // at the last of the token's sixteen
+        *reinterpret_cast<float2*>(wp + 2 * lane) = make_float2(expf(edge - first) * d0, expf(edge - sum) * d1);
     };
 
     load(0);
     cp_async_commit();
     if (warp == 4) step_sizes(0, raw_step(0, 2 * lane), raw_step(0, 2 * lane + 1));
-    const int p_lo = p_base + warp * 16 + qrow, p_hi = p_lo + 8;             // a consumer's rows
-    const bool mine = !producer && p_base + warp * 16 < P;
-    float S[NP / 8][4];                                          // rows p_lo, p_hi; columns 8 j + 2 quad, + 1
+    const int tile = warp % TILES, share = (warp / TILES) % SPLIT, n_base = share * NS;      // a consumer's rows and columns
+    const int p_lo = p_base + tile * 16 + qrow, p_hi = p_lo + 8;
+    const bool mine = !producer && p_base + tile * 16 < P;
+    float S[NS / 8][4];                                          // rows p_lo, p_hi; columns n_base + 8 j + 2 quad, + 1
     if (mine) {
         const float* st = has ? state + ((size_t)slot * H + h) * P * N : nullptr;
 #pragma unroll
-        for (int j = 0; j < NP / 8; ++j) {
-            const int n = j * 8 + quad * 2;
+        for (int j = 0; j < NS / 8; ++j) {
+            const int n = n_base + j * 8 + quad * 2;
             const float2 lo = has && n < N && p_lo < P ? *reinterpret_cast<const float2*>(st + (size_t)p_lo * N + n) : make_float2(0.f, 0.f);
             const float2 hi = has && n < N && p_hi < P ? *reinterpret_cast<const float2*>(st + (size_t)p_hi * N + n) : make_float2(0.f, 0.f);
             S[j][0] = lo.x; S[j][1] = lo.y; S[j][2] = hi.x; S[j][3] = hi.y;
@@ -225,8 +233,8 @@ ssm_chunk_kernel(const __nv_bfloat16* __restrict__ rows, int stride, const float
                 }
                 const __nv_bfloat16* cs = stages + (pc % STAGES) * kStage;
                 const __nv_bfloat16 *bs = cs + kChunk * LDN, *xs = bs + kChunk * LDN;
-                const float* Ls = steps + (pc % 3) * 4 * kChunk;
-                const float *dts = Ls + kChunk, *wu = Ls + 3 * kChunk;
+                const float* Ls = steps + (pc % 3) * 5 * kChunk;
+                const float *dts = Ls + kChunk, *wu = Ls + 3 * kChunk, *wp = Ls + 4 * kChunk;
                 __nv_bfloat16 *xw_hi = xw + (pc & 1) * 2 * kChunk * LDP, *xw_lo = xw_hi + kChunk * LDP;
                 __nv_bfloat16 *w_hi = pw + (pc & 1) * 2 * kChunk * kChunkLd, *w_lo = w_hi + kChunk * kChunkLd;
 #pragma unroll 4
@@ -261,102 +269,139 @@ ssm_chunk_kernel(const __nv_bfloat16* __restrict__ rows, int stride, const float
                     }
                 }
                 const int ta = tr + qrow, tb = ta + 8;
+                // exp(L_t - L_s) of tokens in different sixteens goes by way of the earlier sixteen's last token, whose L lies
+                // between the two: one factor a token and sixteen instead of one a pair, neither above one
                 const float La = Ls[ta], Lb = Ls[tb];
 #pragma unroll
-                for (int j = 0; j < kChunk / 8; ++j) {
-                    if (j > 2 * w4 + 1) continue;
-                    const int s = j * 8 + quad * 2;
-                    const float2 ls = *reinterpret_cast<const float2*>(Ls + s), d = *reinterpret_cast<const float2*>(dts + s);
-                    uint32_t hi, lo;
-                    split_bf16(s <= ta ? g[j][0] * expf(La - ls.x) * d.x : 0.f, s + 1 <= ta ? g[j][1] * expf(La - ls.y) * d.y : 0.f, hi, lo);
-                    *reinterpret_cast<uint32_t*>(w_hi + ta * kChunkLd + s) = hi;
-                    *reinterpret_cast<uint32_t*>(w_lo + ta * kChunkLd + s) = lo;
-                    split_bf16(s <= tb ? g[j][2] * expf(Lb - ls.x) * d.x : 0.f, s + 1 <= tb ? g[j][3] * expf(Lb - ls.y) * d.y : 0.f, hi, lo);
-                    *reinterpret_cast<uint32_t*>(w_hi + tb * kChunkLd + s) = hi;
-                    *reinterpret_cast<uint32_t*>(w_lo + tb * kChunkLd + s) = lo;
+                for (int np = 0; np < kChunk / 16; ++np) {
+                    if (np > w4) continue;
+                    const float edge = Ls[np * 16 + 15];
+                    const bool diagonal = np == w4;
+                    const float fa = diagonal ? 1.f : expf(La - edge), fb = diagonal ? 1.f : expf(Lb - edge);
+#pragma unroll
+                    for (int half = 0; half < 2; ++half) {
+                        const int j = 2 * np + half, s = j * 8 + quad * 2;
+                        float2 va, vb;
+                        if (diagonal) {
+                            const float2 ls = *reinterpret_cast<const float2*>(Ls + s), d = *reinterpret_cast<const float2*>(dts + s);
+                            va = make_float2(s <= ta ? expf(La - ls.x) * d.x : 0.f, s + 1 <= ta ? expf(La - ls.y) * d.y : 0.f);
+                            vb = make_float2(s <= tb ? expf(Lb - ls.x) * d.x : 0.f, s + 1 <= tb ? expf(Lb - ls.y) * d.y : 0.f);
+                        } else {
+                            const float2 w = *reinterpret_cast<const float2*>(wp + s);
+                            va = make_float2(fa * w.x, fa * w.y);
+                            vb = make_float2(fb * w.x, fb * w.y);
+                        }
+                        uint32_t hi, lo;
+                        split_bf16(g[j][0] * va.x, g[j][1] * va.y, hi, lo);
+                        *reinterpret_cast<uint32_t*>(w_hi + ta * kChunkLd + s) = hi;
+                        *reinterpret_cast<uint32_t*>(w_lo + ta * kChunkLd + s) = lo;
+                        split_bf16(g[j][2] * vb.x, g[j][3] * vb.y, hi, lo);
+                        *reinterpret_cast<uint32_t*>(w_hi + tb * kChunkLd + s) = hi;
+                        *reinterpret_cast<uint32_t*>(w_lo + tb * kChunkLd + s) = lo;
+                    }
                 }
                 if (ahead) step_sizes(pc + 1, z0, z1);
             }
-        } else if (c >= 0 && mine) {
+        } else if (c >= 0) {
             const __nv_bfloat16* cs = stages + (c % STAGES) * kStage;
             const __nv_bfloat16 *bs = cs + kChunk * LDN, *xs = bs + kChunk * LDN;
-            const float* eL = steps + (c % 3) * 4 * kChunk + 2 * kChunk;
+            const float* eL = steps + (c % 3) * 5 * kChunk + 2 * kChunk;
             const __nv_bfloat16 *xw_hi = xw + (c & 1) * 2 * kChunk * LDP, *xw_lo = xw_hi + kChunk * LDP;
             const __nv_bfloat16 *w_hi = pw + (c & 1) * 2 * kChunk * kChunkLd, *w_lo = w_hi + kChunk * kChunkLd;
             // y = S0 C^T: rows of S from the registers
             float y[kChunk / 8][4];
 #pragma unroll
             for (int j = 0; j < kChunk / 8; ++j) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
+            if (mine) {
 #pragma unroll
-            for (int kk = 0; kk < NP / 16; ++kk) {
-                uint32_t hi[4], lo[4];
-                split_bf16(S[2 * kk][0], S[2 * kk][1], hi[0], lo[0]);
-                split_bf16(S[2 * kk][2], S[2 * kk][3], hi[1], lo[1]);
-                split_bf16(S[2 * kk + 1][0], S[2 * kk + 1][1], hi[2], lo[2]);
-                split_bf16(S[2 * kk + 1][2], S[2 * kk + 1][3], hi[3], lo[3]);
-                uint32_t bf[kChunk / 16][4];
+                for (int kk = 0; kk < NS / 16; ++kk) {
+                    uint32_t hi[4], lo[4];
+                    split_bf16(S[2 * kk][0], S[2 * kk][1], hi[0], lo[0]);
+                    split_bf16(S[2 * kk][2], S[2 * kk][3], hi[1], lo[1]);
+                    split_bf16(S[2 * kk + 1][0], S[2 * kk + 1][1], hi[2], lo[2]);
+                    split_bf16(S[2 * kk + 1][2], S[2 * kk + 1][3], hi[3], lo[3]);
+                    uint32_t bf[kChunk / 16][4];
 #pragma unroll
-                for (int np = 0; np < kChunk / 16; ++np)
-                    ldmatrix_x4(bf[np], smem_u32(cs + (np * 16 + (mat >> 1) * 8 + rr) * LDN + kk * 16 + (mat & 1) * 8));
+                    for (int np = 0; np < kChunk / 16; ++np)
+                        ldmatrix_x4(bf[np], smem_u32(cs + (np * 16 + (mat >> 1) * 8 + rr) * LDN + n_base + kk * 16 + (mat & 1) * 8));
 #pragma unroll
-                for (int np = 0; np < kChunk / 16; ++np) {
-                    mma_bf16_16816(y[2 * np], hi, bf[np][0], bf[np][1]);
-                    mma_bf16_16816(y[2 * np + 1], hi, bf[np][2], bf[np][3]);
+                    for (int np = 0; np < kChunk / 16; ++np) {
+                        mma_bf16_16816(y[2 * np], hi, bf[np][0], bf[np][1]);
+                        mma_bf16_16816(y[2 * np + 1], hi, bf[np][2], bf[np][3]);
+                    }
+#pragma unroll
+                    for (int np = 0; np < kChunk / 16; ++np) {
+                        mma_bf16_16816(y[2 * np], lo, bf[np][0], bf[np][1]);
+                        mma_bf16_16816(y[2 * np + 1], lo, bf[np][2], bf[np][3]);
+                    }
                 }
 #pragma unroll
-                for (int np = 0; np < kChunk / 16; ++np) {
-                    mma_bf16_16816(y[2 * np], lo, bf[np][0], bf[np][1]);
-                    mma_bf16_16816(y[2 * np + 1], lo, bf[np][2], bf[np][3]);
+                for (int j = 0; j < kChunk / 8; ++j) {
+                    const float2 e = *reinterpret_cast<const float2*>(eL + j * 8 + quad * 2);
+                    y[j][0] *= e.x; y[j][1] *= e.y; y[j][2] *= e.x; y[j][3] *= e.y;
+                }
+                const float e_end = eL[kChunk - 1];
+#pragma unroll
+                for (int j = 0; j < NS / 8; ++j) { S[j][0] *= e_end; S[j][1] *= e_end; S[j][2] *= e_end; S[j][3] *= e_end; }
+#pragma unroll
+                for (int kk = 0; kk < kChunk / 16; ++kk) {
+                    const int s0 = kk * 16;
+                    uint32_t xa[4], wa_hi[4], wa_lo[4];
+                    const int at = (s0 + (mat >> 1) * 8 + rr) * LDP + tile * 16 + (mat & 1) * 8;
+                    ldmatrix_x4_trans(wa_hi, smem_u32(xw_hi + at));
+                    ldmatrix_x4_trans(wa_lo, smem_u32(xw_lo + at));
+                    const bool pairs_here = kk % SPLIT == share;     // this consumer's share of the chunk's own pairs
+                    if (pairs_here) ldmatrix_x4_trans(xa, smem_u32(xs + at));
+#pragma unroll
+                    for (int np = 0; np < kChunk / 16; ++np) {
+                        if (np < kk || !pairs_here) continue;        // tokens before s0 do not see it
+                        uint32_t bh[4], bl[4];
+                        ldmatrix_x4(bh, smem_u32(w_hi + (np * 16 + (mat >> 1) * 8 + rr) * kChunkLd + s0 + (mat & 1) * 8));
+                        ldmatrix_x4(bl, smem_u32(w_lo + (np * 16 + (mat >> 1) * 8 + rr) * kChunkLd + s0 + (mat & 1) * 8));
+                        mma_bf16_16816(y[2 * np], xa, bh[0], bh[1]);
+                        mma_bf16_16816(y[2 * np + 1], xa, bh[2], bh[3]);
+                        mma_bf16_16816(y[2 * np], xa, bl[0], bl[1]);
+                        mma_bf16_16816(y[2 * np + 1], xa, bl[2], bl[3]);
+                    }
+#pragma unroll
+                    for (int nj = 0; nj < NS / 16; ++nj) {
+                        uint32_t bf[4];
+                        ldmatrix_x4_trans(bf, smem_u32(bs + (s0 + (mat & 1) * 8 + rr) * LDN + n_base + nj * 16 + (mat >> 1) * 8));
+                        mma_bf16_16816(S[2 * nj], wa_hi, bf[0], bf[1]);
+                        mma_bf16_16816(S[2 * nj + 1], wa_hi, bf[2], bf[3]);
+                        mma_bf16_16816(S[2 * nj], wa_lo, bf[0], bf[1]);
+                        mma_bf16_16816(S[2 * nj + 1], wa_lo, bf[2], bf[3]);
+                    }
                 }
             }
+            if constexpr (SPLIT > 1) {                           // the consumers of a row tile add up: each for its share of the tokens
 #pragma unroll
-            for (int j = 0; j < kChunk / 8; ++j) {
-                const float2 e = *reinterpret_cast<const float2*>(eL + j * 8 + quad * 2);
-                y[j][0] *= e.x; y[j][1] *= e.y; y[j][2] *= e.x; y[j][3] *= e.y;
-            }
-            const float e_end = eL[kChunk - 1];
+                for (int j = 0; j < kChunk / 8; ++j) parts[(warp * 8 + j) * 32 + lane] = make_float4(y[j][0], y[j][1], y[j][2], y[j][3]);
+                asm volatile("bar.sync 1, 128;" ::: "memory");   // the four consumer warps
 #pragma unroll
-            for (int j = 0; j < NP / 8; ++j) { S[j][0] *= e_end; S[j][1] *= e_end; S[j][2] *= e_end; S[j][3] *= e_end; }
+                for (int i = 0; i < kChunk / 8 / SPLIT; ++i) {
+                    const int j = share * (kChunk / 8 / SPLIT) + i;
+                    float4 sum = parts[(tile * 8 + j) * 32 + lane];
 #pragma unroll
-            for (int kk = 0; kk < kChunk / 16; ++kk) {
-                const int s0 = kk * 16;
-                uint32_t xa[4], wa_hi[4], wa_lo[4];
-                const int at = (s0 + (mat >> 1) * 8 + rr) * LDP + warp * 16 + (mat & 1) * 8;
-                ldmatrix_x4_trans(xa, smem_u32(xs + at));
-                ldmatrix_x4_trans(wa_hi, smem_u32(xw_hi + at));
-                ldmatrix_x4_trans(wa_lo, smem_u32(xw_lo + at));
-#pragma unroll
-                for (int np = 0; np < kChunk / 16; ++np) {
-                    if (np < kk) continue;                       // tokens before s0 do not see it
-                    uint32_t bh[4], bl[4];
-                    ldmatrix_x4(bh, smem_u32(w_hi + (np * 16 + (mat >> 1) * 8 + rr) * kChunkLd + s0 + (mat & 1) * 8));
-                    ldmatrix_x4(bl, smem_u32(w_lo + (np * 16 + (mat >> 1) * 8 + rr) * kChunkLd + s0 + (mat & 1) * 8));
-                    mma_bf16_16816(y[2 * np], xa, bh[0], bh[1]);
-                    mma_bf16_16816(y[2 * np + 1], xa, bh[2], bh[3]);
-                    mma_bf16_16816(y[2 * np], xa, bl[0], bl[1]);
-                    mma_bf16_16816(y[2 * np + 1], xa, bl[2], bl[3]);
-                }
-#pragma unroll
-                for (int nj = 0; nj < NP / 16; ++nj) {
-                    uint32_t bf[4];
-                    ldmatrix_x4_trans(bf, smem_u32(bs + (s0 + (mat & 1) * 8 + rr) * LDN + nj * 16 + (mat >> 1) * 8));
-                    mma_bf16_16816(S[2 * nj], wa_hi, bf[0], bf[1]);
-                    mma_bf16_16816(S[2 * nj + 1], wa_hi, bf[2], bf[3]);
-                    mma_bf16_16816(S[2 * nj], wa_lo, bf[0], bf[1]);
-                    mma_bf16_16816(S[2 * nj + 1], wa_lo, bf[2], bf[3]);
+                    for (int o = 1; o < SPLIT; ++o) {
+                        const float4 v = parts[((tile + o * TILES) * 8 + j) * 32 + lane];
+                        sum.x += v.x; sum.y += v.y; sum.z += v.z; sum.w += v.w;
+                    }
+                    y[i][0] = sum.x; y[i][1] = sum.y; y[i][2] = sum.z; y[i][3] = sum.w;
                 }
             }
-            const int base = t0 + c * kChunk, count = min(kChunk, t1 - base);
-            const int xl = warp * 16 + qrow;                     // this lane's rows within x's columns
+            const int base = t0 + c * kChunk, count = mine ? min(kChunk, t1 - base) : 0;
+            const int xl = tile * 16 + qrow;                     // this lane's rows within x's columns
 #pragma unroll
-            for (int j = 0; j < kChunk / 8; ++j) {
+            for (int i = 0; i < kChunk / 8 / SPLIT; ++i) {
+                const int j = share * (kChunk / 8 / SPLIT) + i;
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int s = j * 8 + quad * 2 + e;
                     if (s >= count) continue;
                     float* dst = out + ((size_t)(base + s) * H + h) * P;
-                    if (p_lo < P) dst[p_lo] = fmaf(dskip, __bfloat162float(xs[s * LDP + xl]), y[j][e]);
-                    if (p_hi < P) dst[p_hi] = fmaf(dskip, __bfloat162float(xs[s * LDP + xl + 8]), y[j][2 + e]);
+                    if (p_lo < P) dst[p_lo] = fmaf(dskip, __bfloat162float(xs[s * LDP + xl]), y[i][e]);
+                    if (p_hi < P) dst[p_hi] = fmaf(dskip, __bfloat162float(xs[s * LDP + xl + 8]), y[i][2 + e]);
                 }
             }
         }
@@ -369,8 +414,8 @@ ssm_chunk_kernel(const __nv_bfloat16* __restrict__ rows, int stride, const float
     if (!has || !mine) return;
     float* st = state + ((size_t)slot * H + h) * P * N;
 #pragma unroll
-    for (int j = 0; j < NP / 8; ++j) {
-        const int n = j * 8 + quad * 2;
+    for (int j = 0; j < NS / 8; ++j) {
+        const int n = n_base + j * 8 + quad * 2;
         if (n >= N) continue;
         if (p_lo < P) *reinterpret_cast<float2*>(st + (size_t)p_lo * N + n) = make_float2(S[j][0], S[j][1]);
         if (p_hi < P) *reinterpret_cast<float2*>(st + (size_t)p_hi * N + n) = make_float2(S[j][2], S[j][3]);
@@ -435,19 +480,35 @@ extern "C" int cib_ssm_chunk_supports(int H, int G, int P, int N) {
     return H > 0 && G > 0 && P % 8 == 0 && N % 8 == 0 && N <= 256 && H % G == 0;
 }
 
+template <int NP, int TILES>
+static int launch_ssm_chunk_tiles(const void* rows, int stride, const float* z, int z_stride, AnyVec db, AnyVec al, AnyVec sk, float* state,
+                            const int* query_start_loc, const int* state_slots, int num_slots, int num_requests, float* out, int H, int G, int P,
+                            int N, int few, cudaStream_t stream) {
+    constexpr size_t smem = ssm_chunk_smem<NP, TILES>();
+    static_assert(smem <= 227 * 1024, "a chunk's working set does not fit");
+    static SmemLimit limit;
+    if (int rc = raise_smem_limit(limit, ssm_chunk_kernel<NP, TILES>, smem, "ssm_chunk")) return rc;
+    const dim3 grid(H, (P + TILES * 16 - 1) / (TILES * 16), num_requests);
+    ssm_chunk_kernel<NP, TILES><<<grid, kChunkThreads, smem, stream>>>((const __nv_bfloat16*)rows, stride, z, z_stride, db, al, sk, state, query_start_loc,
+                                                               state_slots, num_slots, out, H, G, P, N, few);
+    CIB_LAUNCH_CHECK("ssm_chunk");
+    return 0;
+}
+
+// Row tiles a CTA: as few as leave every CTA an SM of its own.
 template <int NP>
 static int launch_ssm_chunk(const void* rows, int stride, const float* z, int z_stride, AnyVec db, AnyVec al, AnyVec sk, float* state,
                             const int* query_start_loc, const int* state_slots, int num_slots, int num_requests, float* out, int H, int G, int P,
                             int N, int few, cudaStream_t stream) {
-    constexpr size_t smem = ssm_chunk_smem<NP>();
-    static_assert(smem <= 227 * 1024, "a chunk's working set does not fit");
-    static SmemLimit limit;
-    if (int rc = raise_smem_limit(limit, ssm_chunk_kernel<NP>, smem, "ssm_chunk")) return rc;
-    const dim3 grid(H, (P + kChunkRows - 1) / kChunkRows, num_requests);
-    ssm_chunk_kernel<NP><<<grid, kChunkThreads, smem, stream>>>((const __nv_bfloat16*)rows, stride, z, z_stride, db, al, sk, state, query_start_loc,
-                                                               state_slots, num_slots, out, H, G, P, N, few);
-    CIB_LAUNCH_CHECK("ssm_chunk");
-    return 0;
+    auto ctas = [&](int tiles) { return (long long)num_requests * H * ((P + tiles * 16 - 1) / (tiles * 16)); };
+#define CIB_SSM_TILES(TILES)                                                                                                             \
+    return launch_ssm_chunk_tiles<NP, TILES>(rows, stride, z, z_stride, db, al, sk, state, query_start_loc, state_slots, num_slots,          \
+                                             num_requests, out, H, G, P, N, few, stream)
+    if constexpr (NP >= 64)
+        if (ctas(1) <= 148) CIB_SSM_TILES(1);
+    if (ctas(2) <= 148) CIB_SSM_TILES(2);
+    CIB_SSM_TILES(4);
+#undef CIB_SSM_TILES
 }
 
 // rows [tokens][>= H P + 2 G N] `stride` apart; z float32 step-size logits [tokens][>= H] `z_stride` apart; dt_bias, a_log, skip [H];

@@ -128,6 +128,11 @@ class GeluFeedForward(SquaredReluFeedForward):
 
     accepts_lazy_norm = True       # the up projection can compute the norm of its input itself
 
+    def __init__(self, spec: PartSpec, **kw) -> None:
+        super().__init__(spec, **kw)
+        if self._bias_specs:
+            raise ValueError("gelu_tanh: biases are not built")
+
     def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
         y = self.up.forward(x)
         act = torch.empty_like(y)
