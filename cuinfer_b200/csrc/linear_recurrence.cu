@@ -224,10 +224,15 @@ lru_decode_kernel(const T* __restrict__ u, int u_stride, const T* __restrict__ w
     const T* wi = wr + (size_t)b * b;
     griddep_launch();
     // weights: not written by the kernel before this one
-    uint4 first_r = make_uint4(0, 0, 0, 0), first_i = first_r;
-    if (VEC && lane * 8 < b) {
-        first_r = *reinterpret_cast<const uint4*>(wr + lane * 8);
-        first_i = *reinterpret_cast<const uint4*>(wi + lane * 8);
+    constexpr int AHEAD = 4;
+    uint32_t first_r[AHEAD], first_i[AHEAD];
+    if constexpr (VEC) {
+#pragma unroll
+        for (int q = 0; q < AHEAD; ++q) {
+            const int k = q * 64 + lane * 2;
+            first_r[q] = k < b ? *reinterpret_cast<const uint32_t*>(wr + k) : 0u;
+            first_i[q] = k < b ? *reinterpret_cast<const uint32_t*>(wi + k) : 0u;
+        }
     }
     const float br = bias[c], bi = bias[C + c], rate = sp[c], yb = y_bias[c];
     griddep_wait();
@@ -245,34 +250,34 @@ lru_decode_kernel(const T* __restrict__ u, int u_stride, const T* __restrict__ w
             gate = to_f32(y[(size_t)mine * y_stride + c]);
         }
         __syncthreads();
-        for (int idx = threadIdx.x; idx < kLruTokens * b; idx += blockDim.x) {
-            const int tt = idx / b, k = idx - tt * b;
-            us[idx] = tt < count ? to_f32(u[(size_t)(tb + tt) * u_stride + (size_t)block * b + k]) : 0.f;
+        for (int k = threadIdx.x; k < b; k += blockDim.x) {
+            const T* src = u + (size_t)tb * u_stride + (size_t)block * b + k;
+            float x[kLruTokens];
+#pragma unroll
+            for (int tt = 0; tt < kLruTokens; ++tt) x[tt] = tt < count ? to_f32(src[(size_t)tt * u_stride]) : 0.f;
+#pragma unroll
+            for (int tt = 0; tt < kLruTokens; ++tt) us[tt * b + k] = x[tt];
         }
         __syncthreads();
         float v[2 * kLruTokens];                         // [token][Ra, Ri]
 #pragma unroll
         for (int i = 0; i < 2 * kLruTokens; ++i) v[i] = 0.f;
-        if constexpr (VEC) {                             // bfloat16, b a multiple of 8: 16 bytes of each row a lane
-            for (int k = lane * 8; k < b; k += 256) {
-                uint4 vr = first_r, vi = first_i;
-                if (k >= 256) {
-                    vr = *reinterpret_cast<const uint4*>(wr + k);
-                    vi = *reinterpret_cast<const uint4*>(wi + k);
-                }
-                const __nv_bfloat162* hr = reinterpret_cast<const __nv_bfloat162*>(&vr);
-                const __nv_bfloat162* hi = reinterpret_cast<const __nv_bfloat162*>(&vi);
+        if constexpr (VEC) {                             // bfloat16, b even: two neighbouring values a lane and load
+            auto pair = [&](int k, uint32_t vr, uint32_t vi) {
+                const float2 fr = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&vr));
+                const float2 fi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&vi));
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const float2 fr = __bfloat1622float2(hr[e]), fi = __bfloat1622float2(hi[e]);
-#pragma unroll
-                    for (int tt = 0; tt < kLruTokens; ++tt) {
-                        const float2 x = *reinterpret_cast<const float2*>(us + tt * b + k + 2 * e);
-                        v[2 * tt] = fmaf(fr.x, x.x, fmaf(fr.y, x.y, v[2 * tt]));
-                        v[2 * tt + 1] = fmaf(fi.x, x.x, fmaf(fi.y, x.y, v[2 * tt + 1]));
-                    }
+                for (int tt = 0; tt < kLruTokens; ++tt) {
+                    const float2 x = *reinterpret_cast<const float2*>(us + tt * b + k);
+                    v[2 * tt] = fmaf(fr.x, x.x, fmaf(fr.y, x.y, v[2 * tt]));
+                    v[2 * tt + 1] = fmaf(fi.x, x.x, fmaf(fi.y, x.y, v[2 * tt + 1]));
                 }
-            }
+            };
+#pragma unroll
+            for (int q = 0; q < AHEAD; ++q)
+                if (q * 64 + lane * 2 < b) pair(q * 64 + lane * 2, first_r[q], first_i[q]);
+            for (int k = AHEAD * 64 + lane * 2; k < b; k += 64)
+                pair(k, *reinterpret_cast<const uint32_t*>(wr + k), *reinterpret_cast<const uint32_t*>(wi + k));
         } else {
             for (int k = lane; k < b; k += 32) {
                 const float fr = to_f32(wr[k]), fi = to_f32(wi[k]);
@@ -371,7 +376,7 @@ extern "C" int cib_lru_decode(const void* u, int dtype, int u_stride, const void
     launch_pdl(lru_decode_kernel<T, VEC>, grid, dim3(kLruDecodeWarps * 32), smem, stream, pdl, (const T*)u, u_stride, (const T*)w, bias, sp, \
                (const T*)y, y_stride, y_bias, out_scale, state, state_slots, num_slots, (T*)out, C, b, num_tokens)
     if (dtype == kF32) CIB_LRU(float, false);
-    else if (dtype == kBF16 && b % 8 == 0 && (uintptr_t)w % 16 == 0) CIB_LRU(__nv_bfloat16, true);
+    else if (dtype == kBF16 && b % 2 == 0 && (uintptr_t)w % 4 == 0) CIB_LRU(__nv_bfloat16, true);
     else if (dtype == kBF16) CIB_LRU(__nv_bfloat16, false);
     else CIB_REQUIRE(false, "lru_decode: bad dtype %d", dtype);
 #undef CIB_LRU
